@@ -1,6 +1,7 @@
-"""ctypes binding of ``libquickdraw_b200.so`` (declarations: ``include/quickdraw_b200.h``).
+"""ctypes binding of ``libquickdraw_b200.so`` (declarations: ``include/quickdraw_b200.h``) and of
+``libquickdraw_b200_hybrid.so`` (``include/quickdraw_b200_hybrid.h``), the kernels of the bf16-weight models.
 
-The library is the only execution path of this package: if it cannot be loaded the
+Each library is the only execution path of this package: if it cannot be loaded the
 import of any operator raises, there is no PyTorch or CPU fallback.
 """
 
@@ -13,6 +14,7 @@ from pathlib import Path
 import torch
 
 LIB_PATH = Path(__file__).resolve().parent / "libquickdraw_b200.so"
+HYBRID_PATH = Path(__file__).resolve().parent / "libquickdraw_b200_hybrid.so"
 
 P, I, F, L = c_void_p, c_int, c_float, c_longlong
 
@@ -78,36 +80,69 @@ SIGNATURES = {
     "qd_seq_moe_combine_norm": [P, P, P, P, P, P, P, P, I, I, I, F, P],
 }
 
+# entry points of the second library (declarations: ``include/quickdraw_b200_hybrid.h``)
+HYBRID_SIGNATURES = {
+    "qd_set_chained_launches": [I],
+    "qd_linear": [P, L, I, P, P, L, I, I, I, I, I, P, P],
+    "qd_greedy": [P, I, P, P, P, P],
+    "qd_embed_norm": [P, P, I, P, P, P, P, I, I, F, I, P],
+    "qd_layer_norm_rows": [P, P, P, P, P, I, I, F, I, P],
+    "qd_sublayer_close": [P, P, L, P, P, P, P, P, P, L, P, I, P, P, P, I, I, F, I, P],
+    "qd_gla_prepare": [P, P, P, L, P, P, F, P, P, P, P, I, I, I, I, I, P],
+    "qd_channel_delta_prepare": [P, P, P, P, L, P, P, P, P, P, P, P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, I, P],
+    "qd_linear_recurrence": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
+    "qd_head_norm_gate": [P, P, P, L, P, I, I, I, F, I, I, P],
+    "qd_gla_step": [P, P, P, P, P, P, I, F, P, P, F, P, P, I, I, I, I, P],
+    "qd_channel_delta_step": [P, P, P, P, P, P, P, I, P, P, P, P, P, I, P, I, P, P, I, P, F, P, P, I, I, I, I, I, P],
+    "qd_window_attention": [P, P, P, P, L, P, P, P, I, P, F, F, P, P, I, I, P, I, P, P, I, I, I, I, I, I, P],
+    "qd_window_attention_step_floats": [I, I, I],
+    "qd_window_attention_step": [P, P, P, P, P, P, P, I, P, F, F, P, P, I, I, P, I, P, P, I, P, I, I, I, I, I, P],
+}
+HYBRID_LONG_RESULTS = {"qd_window_attention_step_floats"}
+
 LONG_RESULTS = {"qd_decode_workspace_bytes", "qd_program_bytes", "qd_exchange_bytes",
                 "qd_nvfp4_matmul_rows_scratch_bytes", "qd_seq_gdn_chunk_scratch_bytes",
                 "qd_nvfp4_expert_rows_scratch_bytes"}
 
 _lib = None
+_hybrid = None
 
 
 class LibraryMissing(RuntimeError):
     pass
 
 
+def _open(path: Path, target: str, signatures: dict, long_results: set) -> ctypes.CDLL:
+    if not path.exists():
+        raise LibraryMissing(
+            f"{path} not found: build it with `python -m quickdraw_b200.build{target}` "
+            "(this package has no fallback path)")
+    handle = ctypes.CDLL(str(path))
+    for name, argtypes in signatures.items():
+        fn = getattr(handle, name, None)
+        if fn is None:
+            continue
+        fn.argtypes = argtypes
+        fn.restype = c_longlong if name in long_results else c_int
+    handle.qd_error_string.argtypes = [c_int]
+    handle.qd_error_string.restype = c_char_p
+    return handle
+
+
 def lib() -> ctypes.CDLL:
     """Load the CUDA library once; raise loudly if it has not been built."""
     global _lib
     if _lib is None:
-        if not LIB_PATH.exists():
-            raise LibraryMissing(
-                f"{LIB_PATH} not found: build it with `python -m quickdraw_b200.build` "
-                "(this package has no fallback path)")
-        handle = ctypes.CDLL(str(LIB_PATH))
-        for name, argtypes in SIGNATURES.items():
-            fn = getattr(handle, name, None)
-            if fn is None:
-                continue
-            fn.argtypes = argtypes
-            fn.restype = c_longlong if name in LONG_RESULTS else c_int
-        handle.qd_error_string.argtypes = [c_int]
-        handle.qd_error_string.restype = c_char_p
-        _lib = handle
+        _lib = _open(LIB_PATH, "", SIGNATURES, LONG_RESULTS)
     return _lib
+
+
+def hybrid_lib() -> ctypes.CDLL:
+    """The library of the bf16-weight models, loaded on first use."""
+    global _hybrid
+    if _hybrid is None:
+        _hybrid = _open(HYBRID_PATH, " hybrid", HYBRID_SIGNATURES, HYBRID_LONG_RESULTS)
+    return _hybrid
 
 
 def exported_symbols() -> list[str]:
@@ -138,3 +173,9 @@ def check(code: int, name: str) -> None:
 
 def call(name: str, *args) -> None:
     check(getattr(lib(), name)(*args), name)
+
+
+def call_hybrid(name: str, *args) -> None:
+    code = getattr(hybrid_lib(), name)(*args)
+    if code != 0:
+        raise RuntimeError(f"{name} failed: {hybrid_lib().qd_error_string(code).decode()} (code {code})")

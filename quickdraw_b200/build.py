@@ -1,7 +1,9 @@
-"""Build the C-ABI CUDA library in-tree: ``python -m quickdraw_b200.build``.
+"""Build the C-ABI CUDA libraries in-tree: ``python -m quickdraw_b200.build [nvfp4|hybrid ...]``.
 
-Plain nvcc, one shared object (``quickdraw_b200/libquickdraw_b200.so``), sm_100a only,
-no link against libtorch: the host side passes raw device pointers through ctypes.
+Plain nvcc, shared objects for sm_100a only, no link against libtorch: the host side passes raw
+device pointers through ctypes.  Two libraries, so that a model only needs its own kernels
+compiled: ``libquickdraw_b200.so`` (NVFP4 / FP8 models) and ``libquickdraw_b200_hybrid.so``
+(bf16-weight models).  Without a name both are built.
 """
 
 from __future__ import annotations
@@ -14,37 +16,46 @@ from pathlib import Path
 PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 LIB = PKG / "libquickdraw_b200.so"
+HYBRID = PKG / "libquickdraw_b200_hybrid.so"
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-lineinfo", "-std=c++17",
          "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr"]
 
+COMMON = ("library",)
+HYBRID_SOURCES = ("linear", "residual", "linear_recurrence", "window_attention")
+HYBRID_HEADERS = ("common.cuh", "typed.cuh")
 
-def sources() -> list[Path]:
-    return sorted(CSRC.glob("*.cu"))
+
+def sources(target: str) -> list[Path]:
+    if target == "hybrid":
+        return [CSRC / f"{name}.cu" for name in COMMON + HYBRID_SOURCES]
+    return [path for path in sorted(CSRC.glob("*.cu")) if path.stem not in HYBRID_SOURCES]
 
 
-def stale() -> bool:
-    if not LIB.exists():
+def library(target: str) -> Path:
+    return {"nvfp4": LIB, "hybrid": HYBRID}[target]
+
+
+def stale(target: str = "nvfp4") -> bool:
+    lib = library(target)
+    if not lib.exists():
         return True
-    newest = max(p.stat().st_mtime for p in list(CSRC.glob("*.cu*")) +
-                 [PKG.parent / "include" / "quickdraw_b200.h"])
-    return newest > LIB.stat().st_mtime
+    headers = ([CSRC / name for name in HYBRID_HEADERS] if target == "hybrid" else sorted(CSRC.glob("*.cuh")))
+    headers += sorted((PKG.parent / "include").glob("*.h"))
+    return max(p.stat().st_mtime for p in sources(target) + headers) > lib.stat().st_mtime
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    if not force and not stale():
-        return LIB
-    objects = []
-    procs = []
+def build(force: bool = False, verbose: bool = False, targets=("nvfp4", "hybrid")) -> list[Path]:
+    """Compile what is out of date; every source of every requested library in parallel."""
+    wanted = [t for t in targets if force or stale(t)]
     build_dir = PKG / "build"
     build_dir.mkdir(exist_ok=True)
-    for src in sources():
-        obj = build_dir / (src.stem + ".o")
-        cmd = [NVCC, *FLAGS, "-c", str(src), "-o", str(obj)]
+    procs, objects = [], {t: [build_dir / (src.stem + ".o") for src in sources(t)] for t in wanted}
+    for src in dict.fromkeys(src for t in wanted for src in sources(t)):
+        cmd = [NVCC, *FLAGS, "-c", str(src), "-o", str(build_dir / (src.stem + ".o"))]
         if verbose:
             cmd.insert(1, "-Xptxas=-v")
         procs.append((src, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
-        objects.append(obj)
     failed = False
     for src, proc in procs:
         out, _ = proc.communicate()
@@ -53,9 +64,11 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         failed |= proc.returncode != 0
     if failed:
         raise RuntimeError("nvcc failed")
-    subprocess.run([NVCC, "-shared", "-o", str(LIB), *map(str, objects), "-lcudart"], check=True)
-    return LIB
+    for t in wanted:
+        subprocess.run([NVCC, "-shared", "-o", str(library(t)), *map(str, objects[t]), "-lcudart"], check=True)
+    return [library(t) for t in targets]
 
 
 if __name__ == "__main__":
-    print(build(force="--force" in sys.argv, verbose="-v" in sys.argv))
+    names = [a for a in sys.argv[1:] if not a.startswith("-")] or ["nvfp4", "hybrid"]
+    print(*build(force="--force" in sys.argv, verbose="-v" in sys.argv, targets=names), sep="\n")

@@ -1,0 +1,657 @@
+// Gated linear recurrences with one decay per head and key channel, state S [dim, vdim] per head in fp32:
+//   gated linear attention   S = diag(a) S + k v^T,                               o = S^T q
+//   channel-decay delta rule S = diag(g) S, u = beta (v - S^T k), S = S + k u^T,  o = S^T q
+// (gdn.cu has the delta rule with one decay per head.)  Everything that enters the recurrence is fp32.
+//
+// Prompt chunks: a prepare kernel (all tokens in parallel: short convolution, SiLU, unit norms, decays)
+// writes q, k, decay, v, beta as fp32 rows; linear_recurrence_kernel walks the tokens with the state in
+// registers.  A warp owns eight value columns; lane = (key group kl of eight, column pair cl): rows
+// 32 j + 4 kl + {0..3}, two columns, held as row pairs for the packed fp32 FMA.  Both read-outs of the
+// delta rule use the decayed state before the write, o = (gS)^T q + (k . q) u, so that one round of
+// shuffles carries both and the write is off the critical path.  Latency-bound: one warp per scheduler,
+// a dependent chain per token.
+// Decode: recurrence_step_kernel does everything between the projections and the output projection in
+// one launch: low-rank decay (and output gate), convolution, unit norms, recurrence, per-head RMS norm,
+// gate.  A cluster of blocks shares a head (32 value columns each) and adds its sums of squares over
+// distributed shared memory.  HBM-bound by the state.
+#include <cooperative_groups.h>
+
+#include "typed.cuh"
+
+namespace cg = cooperative_groups;
+
+namespace qd {
+namespace {
+
+constexpr float kUnitEps = 1e-6f;
+
+QD_DEVINL float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+QD_DEVINL float gla_decay(float z, float inv_tau) { return expf(log_sigmoid(z) * inv_tau); }
+QD_DEVINL float delta_decay(float z, float a_log) { return expf(-expf(a_log) * softplus_precise(z)); }
+
+// Convolution input history: ring of `taps` rows, position p in row p mod taps.  A step reads the rows of
+// the taps - 1 positions before it and writes its own, which is none of those.
+struct ConvSource {
+    const void* history;      // [taps, channels]
+    int taps, channels;
+};
+// sum over taps of w[j] * input(position - (taps - 1 - j)) of one channel; x: the channel's input at
+// chunk token t (row stride ld), older inputs from the history, zeros before position 0.
+template <typename T>
+QD_DEVINL float conv_at(const T* x, long long ld, int t, int position, const bf16* w, const ConvSource& src, int channel) {
+    float acc = 0.f;
+    for (int back = src.taps - 1; back >= 0; --back) {
+        const int p = position - back;
+        float v = 0.f;
+        if (back <= t) v = load_f(x + (long long)(t - back) * ld);
+        else if (p >= 0) v = load_f(reinterpret_cast<const T*>(src.history) + (size_t)(p % src.taps) * src.channels + channel);
+        acc = fmaf(v, ld_bf16(w + src.taps - 1 - back), acc);
+    }
+    return acc;
+}
+
+// ----------------------------------------------------------------------------------- prepare
+struct PrepareParams {
+    const void* q; const void* k; const void* v; long long ld;      // this chunk's projections, rows ld apart
+    const float* z; const bf16* z_bias;                             // decay logits [tokens, heads * dim], bias [heads * dim]
+    const void* beta; const bf16* a_log;                            // delta rule: [tokens] rows ld apart; [heads]
+    const bf16* q_taps; const bf16* k_taps; const bf16* v_taps; ConvSource conv;
+    float tau;
+    const int* position_ptr; int position;
+    float* oq; float* ok; float* og; float* ov; float* obeta; float* okq;
+    int heads, kv_heads, dim, vdim;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) gla_prepare_kernel(const __grid_constant__ PrepareParams p) {
+    chain_enter();
+    const size_t t = blockIdx.x;
+    const int keys = p.heads * p.dim, values = p.heads * p.vdim;
+    const T* q = reinterpret_cast<const T*>(p.q) + t * p.ld;
+    const T* k = reinterpret_cast<const T*>(p.k) + t * p.ld;
+    const T* v = reinterpret_cast<const T*>(p.v) + t * p.ld;
+    const float scale = 1.0f / sqrtf((float)p.dim), inv_tau = 1.0f / p.tau;
+    for (int i = threadIdx.x; i < keys; i += blockDim.x) {
+        p.oq[t * keys + i] = load_f(q + i) * scale;
+        p.ok[t * keys + i] = load_f(k + i);
+        p.og[t * keys + i] = gla_decay(p.z[t * keys + i] + ld_bf16(p.z_bias + i), inv_tau);
+    }
+    for (int i = threadIdx.x; i < values; i += blockDim.x) p.ov[t * values + i] = load_f(v + i);
+}
+
+constexpr int kMaxPerLane = 8;       // key channels per lane: dim <= 256
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constant__ PrepareParams p) {
+    chain_enter();
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int position = (p.position_ptr ? *p.position_ptr : p.position) + t;
+    const int keys = p.heads * p.dim, values = p.heads * p.vdim, kv_keys = p.kv_heads * p.dim;
+    const T* q = reinterpret_cast<const T*>(p.q);
+    const T* k = reinterpret_cast<const T*>(p.k);
+    const T* v = reinterpret_cast<const T*>(p.v);
+    const float scale = 1.0f / sqrtf((float)p.dim);
+    for (int h = warp; h < p.kv_heads; h += 8) {
+        float qv[kMaxPerLane], kv[kMaxPerLane], qq = 0.f, kk = 0.f, kq = 0.f;
+#pragma unroll
+        for (int i = 0; i < kMaxPerLane; ++i) {
+            const int d = i * 32 + lane, c = h * p.dim + d;
+            qv[i] = kv[i] = 0.f;
+            if (d < p.dim) {
+                qv[i] = silu_precise(conv_at(q + c, p.ld, t, position, p.q_taps + (size_t)c * p.conv.taps, p.conv, c));
+                kv[i] = silu_precise(conv_at(k + c, p.ld, t, position, p.k_taps + (size_t)c * p.conv.taps, p.conv, kv_keys + c));
+            }
+            qq = fmaf(qv[i], qv[i], qq);
+            kk = fmaf(kv[i], kv[i], kk);
+            kq = fmaf(qv[i], kv[i], kq);
+        }
+        qq = warp_sum(qq); kk = warp_sum(kk); kq = warp_sum(kq);
+        const float qs = scale / sqrtf(qq + kUnitEps), ks = 1.0f / sqrtf(kk + kUnitEps);
+#pragma unroll
+        for (int i = 0; i < kMaxPerLane; ++i) {
+            const int d = i * 32 + lane;
+            if (d < p.dim) {
+                p.oq[(size_t)t * kv_keys + h * p.dim + d] = qv[i] * qs;
+                p.ok[(size_t)t * kv_keys + h * p.dim + d] = kv[i] * ks;
+            }
+        }
+        if (lane == 0) p.okq[(size_t)t * p.kv_heads + h] = kq * qs * ks;
+    }
+    for (int c = threadIdx.x; c < values; c += 256)
+        p.ov[(size_t)t * values + c] = silu_precise(conv_at(v + c, p.ld, t, position, p.v_taps + (size_t)c * p.conv.taps, p.conv, 2 * kv_keys + c));
+    for (int c = threadIdx.x; c < keys; c += 256)
+        p.og[(size_t)t * keys + c] = delta_decay(p.z[(size_t)t * keys + c] + ld_bf16(p.z_bias + c), ld_bf16(p.a_log + c / p.dim));
+    const T* beta = reinterpret_cast<const T*>(p.beta) + (size_t)t * p.ld;
+    for (int h = threadIdx.x; h < p.heads; h += 256) p.obeta[(size_t)t * p.heads + h] = sigmoid_precise(load_f(beta + h));
+}
+
+// The chunk's last `taps` inputs into the history ring.
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_history_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long long ld, T* __restrict__ history,
+                    int taps, int kv_keys, int values, int tokens, const int* position_ptr, int position) {
+    chain_enter();
+    const int channels = 2 * kv_keys + values, back = blockIdx.y, t = tokens - 1 - back;
+    const int c = blockIdx.x * 256 + threadIdx.x;
+    if (t < 0 || c >= channels) return;
+    const int at = (position_ptr ? *position_ptr : position) + t;
+    const T* src = c < kv_keys ? q + c : (c < 2 * kv_keys ? k + (c - kv_keys) : v + (c - 2 * kv_keys));
+    history[(size_t)(at % taps) * channels + c] = src[(long long)t * ld];
+}
+
+// -------------------------------------------------------------------------------- recurrence
+typedef unsigned long long u64;
+QD_DEVINL u64 mul2(u64 a, u64 b) { u64 d; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
+QD_DEVINL u64 fma2(u64 a, u64 b, u64 c) { u64 d; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c)); return d; }
+QD_DEVINL u64 pack2(float lo, float hi) { return (u64)__float_as_uint(lo) | ((u64)__float_as_uint(hi) << 32); }
+QD_DEVINL float lo2(u64 v) { return __uint_as_float((uint32_t)v); }
+QD_DEVINL float hi2(u64 v) { return __uint_as_float((uint32_t)(v >> 32)); }
+
+QD_DEVINL void copy16(void* dst, const void* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+QD_DEVINL void copy4(void* dst, const void* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+QD_DEVINL void copies_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> QD_DEVINL void copies_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+constexpr int kRecThreads = 128, kRecCols = 32, kRecTile = 16;      // block: four warps x eight columns; tokens per staged tile
+
+struct RecurrenceParams {
+    const float* q; const float* k; const float* g; const float* v; const float* beta; const float* kq;
+    float* state; float* out;
+    int tokens, heads, kv_heads, dim, vdim, vectors;
+};
+
+// floats of one staged token: q, k, decay (padded to 32 J), v columns, beta, k . q (padded to 4)
+template <int J> constexpr int rec_token_floats() { return 3 * 32 * J + kRecCols + 4; }
+
+template <int J, bool DELTA>
+__global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __grid_constant__ RecurrenceParams p) {
+    chain_enter();
+    extern __shared__ __align__(16) float tiles[];
+    constexpr int kToken = rec_token_floats<J>(), kRow = 32 * J;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, kl = lane & 7, cl = lane >> 3;
+    const int head = blockIdx.x, kv = head / (p.heads / p.kv_heads), c0 = blockIdx.y * kRecCols;
+    const int col = c0 + warp * 8 + cl * 2;
+    const int dim = p.dim, vdim = p.vdim;
+    float* state = p.state + (size_t)head * dim * vdim;
+
+    for (int i = tid; i < 2 * kRecTile * kToken; i += kRecThreads) tiles[i] = 0.f;      // padding rows stay zero
+    u64 s[J][2][2];
+#pragma unroll
+    for (int j = 0; j < J; ++j)
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+                const int r = j * 32 + kl * 4 + h * 2;
+                const bool ok = col + c < vdim;
+                s[j][h][c] = pack2(ok && r < dim ? state[(size_t)r * vdim + col + c] : 0.f,
+                                   ok && r + 1 < dim ? state[(size_t)(r + 1) * vdim + col + c] : 0.f);
+            }
+    __syncthreads();
+
+    const int cols = min(kRecCols, vdim - c0);
+    auto stage = [&](int tile) {
+        float* base = tiles + (tile & 1) * kRecTile * kToken;
+        const int t0 = tile * kRecTile, count = min(kRecTile, p.tokens - t0);
+        if (p.vectors) {
+            const int kp = dim / 4, vp = cols / 4, per = 3 * kp + vp;
+            for (int i = tid; i < count * per; i += kRecThreads) {
+                const int tt = i / per, piece = i % per;
+                const size_t t = t0 + tt;
+                float* dst = base + tt * kToken;
+                if (piece < kp) copy16(dst + piece * 4, p.q + (t * p.kv_heads + kv) * dim + piece * 4);
+                else if (piece < 2 * kp) copy16(dst + kRow + (piece - kp) * 4, p.k + (t * p.kv_heads + kv) * dim + (piece - kp) * 4);
+                else if (piece < 3 * kp) copy16(dst + 2 * kRow + (piece - 2 * kp) * 4, p.g + (t * p.heads + head) * dim + (piece - 2 * kp) * 4);
+                else copy16(dst + 3 * kRow + (piece - 3 * kp) * 4, p.v + (t * p.heads + head) * vdim + c0 + (piece - 3 * kp) * 4);
+            }
+        } else {
+            const int per = 3 * dim + cols;
+            for (int i = tid; i < count * per; i += kRecThreads) {
+                const int tt = i / per, e = i % per;
+                const size_t t = t0 + tt;
+                float* dst = base + tt * kToken;
+                if (e < dim) copy4(dst + e, p.q + (t * p.kv_heads + kv) * dim + e);
+                else if (e < 2 * dim) copy4(dst + kRow + e - dim, p.k + (t * p.kv_heads + kv) * dim + e - dim);
+                else if (e < 3 * dim) copy4(dst + 2 * kRow + e - 2 * dim, p.g + (t * p.heads + head) * dim + e - 2 * dim);
+                else copy4(dst + 3 * kRow + e - 3 * dim, p.v + (t * p.heads + head) * vdim + c0 + e - 3 * dim);
+            }
+        }
+        if (DELTA && tid < count) {
+            float* dst = base + tid * kToken + 3 * kRow + kRecCols;
+            copy4(dst, p.beta + (size_t)(t0 + tid) * p.heads + head);
+            copy4(dst + 1, p.kq + (size_t)(t0 + tid) * p.kv_heads + kv);
+        }
+        copies_commit();
+    };
+
+    const int ntiles = (p.tokens + kRecTile - 1) / kRecTile;
+    stage(0);
+    for (int tile = 0; tile < ntiles; ++tile) {
+        if (tile + 1 < ntiles) { stage(tile + 1); copies_wait<1>(); } else { copies_wait<0>(); }
+        __syncthreads();
+        const float* base = tiles + (tile & 1) * kRecTile * kToken;
+        const int t0 = tile * kRecTile, count = min(kRecTile, p.tokens - t0);
+        ulonglong2 q[J], k[J], g[J];
+        auto fetch = [&](const float* token, ulonglong2 (&fq)[J], ulonglong2 (&fk)[J], ulonglong2 (&fg)[J]) {
+#pragma unroll
+            for (int j = 0; j < J; ++j) {
+                fg[j] = *reinterpret_cast<const ulonglong2*>(token + 2 * kRow + j * 32 + kl * 4);
+                fk[j] = *reinterpret_cast<const ulonglong2*>(token + kRow + j * 32 + kl * 4);
+                fq[j] = *reinterpret_cast<const ulonglong2*>(token + j * 32 + kl * 4);
+            }
+        };
+        constexpr bool kAhead = J <= 4;             // the next token's vectors in registers while this one is reduced
+        fetch(base, q, k, g);
+        for (int tt = 0; tt < count; ++tt) {
+            const float* token = base + tt * kToken;
+            if (!kAhead && tt) fetch(token, q, k, g);
+            const float2 v = *reinterpret_cast<const float2*>(token + 3 * kRow + warp * 8 + cl * 2);
+            u64 o[2] = {0ull, 0ull};
+            float out[2];
+            if (DELTA) {
+                const float2 bk = *reinterpret_cast<const float2*>(token + 3 * kRow + kRecCols);      // beta, k . q
+                u64 pr[2] = {0ull, 0ull};
+#pragma unroll
+                for (int j = 0; j < J; ++j)
+#pragma unroll
+                    for (int c = 0; c < 2; ++c) {
+                        s[j][0][c] = mul2(s[j][0][c], g[j].x);
+                        s[j][1][c] = mul2(s[j][1][c], g[j].y);
+                        pr[c] = fma2(s[j][0][c], k[j].x, pr[c]);
+                        o[c] = fma2(s[j][0][c], q[j].x, o[c]);
+                        pr[c] = fma2(s[j][1][c], k[j].y, pr[c]);
+                        o[c] = fma2(s[j][1][c], q[j].y, o[c]);
+                    }
+                float pred[2] = {lo2(pr[0]) + hi2(pr[0]), lo2(pr[1]) + hi2(pr[1])};
+                out[0] = lo2(o[0]) + hi2(o[0]);
+                out[1] = lo2(o[1]) + hi2(o[1]);
+                ulonglong2 nq[J], nk[J], ng[J];
+                if (kAhead && tt + 1 < count) fetch(token + kToken, nq, nk, ng);
+#pragma unroll
+                for (int x = 1; x < 8; x <<= 1) {
+                    pred[0] += __shfl_xor_sync(0xffffffffu, pred[0], x);
+                    pred[1] += __shfl_xor_sync(0xffffffffu, pred[1], x);
+                    out[0] += __shfl_xor_sync(0xffffffffu, out[0], x);
+                    out[1] += __shfl_xor_sync(0xffffffffu, out[1], x);
+                }
+                const float u0 = bk.x * (v.x - pred[0]), u1 = bk.x * (v.y - pred[1]);
+                out[0] = fmaf(u0, bk.y, out[0]);
+                out[1] = fmaf(u1, bk.y, out[1]);
+                const u64 uu[2] = {pack2(u0, u0), pack2(u1, u1)};
+#pragma unroll
+                for (int j = 0; j < J; ++j)
+#pragma unroll
+                    for (int c = 0; c < 2; ++c) {
+                        s[j][0][c] = fma2(k[j].x, uu[c], s[j][0][c]);
+                        s[j][1][c] = fma2(k[j].y, uu[c], s[j][1][c]);
+                    }
+                if (kAhead) {
+#pragma unroll
+                    for (int j = 0; j < J; ++j) { q[j] = nq[j]; k[j] = nk[j]; g[j] = ng[j]; }
+                }
+            } else {
+                const u64 vv[2] = {pack2(v.x, v.x), pack2(v.y, v.y)};
+                ulonglong2 nq[J], nk[J], ng[J];
+                if (kAhead && tt + 1 < count) fetch(token + kToken, nq, nk, ng);
+#pragma unroll
+                for (int j = 0; j < J; ++j)
+#pragma unroll
+                    for (int c = 0; c < 2; ++c) {
+                        s[j][0][c] = fma2(s[j][0][c], g[j].x, mul2(k[j].x, vv[c]));
+                        s[j][1][c] = fma2(s[j][1][c], g[j].y, mul2(k[j].y, vv[c]));
+                        o[c] = fma2(s[j][0][c], q[j].x, o[c]);
+                        o[c] = fma2(s[j][1][c], q[j].y, o[c]);
+                    }
+                out[0] = lo2(o[0]) + hi2(o[0]);
+                out[1] = lo2(o[1]) + hi2(o[1]);
+#pragma unroll
+                for (int x = 1; x < 8; x <<= 1) {
+                    out[0] += __shfl_xor_sync(0xffffffffu, out[0], x);
+                    out[1] += __shfl_xor_sync(0xffffffffu, out[1], x);
+                }
+                if (kAhead) {
+#pragma unroll
+                    for (int j = 0; j < J; ++j) { q[j] = nq[j]; k[j] = nk[j]; g[j] = ng[j]; }
+                }
+            }
+            if (kl == 0) {
+                float* dst = p.out + ((size_t)(t0 + tt) * p.heads + head) * vdim + col;
+                if (col < vdim) dst[0] = out[0];
+                if (col + 1 < vdim) dst[1] = out[1];
+            }
+        }
+        __syncthreads();                 // the buffer may be refilled
+    }
+#pragma unroll
+    for (int j = 0; j < J; ++j)
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+                const int r = j * 32 + kl * 4 + h * 2;
+                if (col + c < vdim) {
+                    if (r < dim) state[(size_t)r * vdim + col + c] = lo2(s[j][h][c]);
+                    if (r + 1 < dim) state[(size_t)(r + 1) * vdim + col + c] = hi2(s[j][h][c]);
+                }
+            }
+}
+
+template <int J, bool DELTA>
+int launch_recurrence(const RecurrenceParams& p, cudaStream_t stream) {
+    const size_t smem = 2ull * kRecTile * rec_token_floats<J>() * 4;
+    if (!allow_smem(linear_recurrence_kernel<J, DELTA>, smem)) return QD_ERR_LAUNCH;
+    return qd_launch(linear_recurrence_kernel<J, DELTA>, dim3(p.heads, (p.vdim + kRecCols - 1) / kRecCols), dim3(kRecThreads), smem,
+                     stream, 1, p);
+}
+template <bool DELTA>
+int recurrence(const RecurrenceParams& p, cudaStream_t stream) {
+    switch ((p.dim + 31) / 32) {
+        case 1: return launch_recurrence<1, DELTA>(p, stream);
+        case 2: return launch_recurrence<2, DELTA>(p, stream);
+        case 3: return launch_recurrence<3, DELTA>(p, stream);
+        case 4: return launch_recurrence<4, DELTA>(p, stream);
+        case 5: case 6: return launch_recurrence<6, DELTA>(p, stream);
+        case 7: case 8: return launch_recurrence<8, DELTA>(p, stream);
+        default: return QD_ERR_UNSUPPORTED;
+    }
+}
+
+// ------------------------------------------------------------------------ per-head norm, gate
+// out[t, h, :] = x / rms(x) * w * act(gate); act: 0 = SiLU, 1 = sigmoid.  A warp per (token, head).
+template <typename T>
+__global__ void __launch_bounds__(256)
+head_norm_gate_kernel(const float* __restrict__ x, const bf16* __restrict__ w, const T* __restrict__ gate, long long ld_gate,
+                      T* __restrict__ out, int tokens, int heads, int vdim, float eps, int act) {
+    chain_enter();
+    const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (item >= (long long)tokens * heads) return;
+    const long long t = item / heads;
+    const int h = (int)(item % heads);
+    const float* row = x + item * vdim;
+    float sq = 0.f;
+    for (int i = lane; i < vdim; i += 32) sq = fmaf(row[i], row[i], sq);
+    const float r = 1.0f / sqrtf(warp_sum(sq) / (float)vdim + eps);
+    const T* g = gate + t * ld_gate + (long long)h * vdim;
+    for (int i = lane; i < vdim; i += 32) {
+        const float gv = load_f(g + i);
+        store_f(out + item * vdim + i, row[i] * r * ld_bf16(w + i) * (act ? sigmoid_precise(gv) : silu_precise(gv)));
+    }
+}
+
+// ------------------------------------------------------------------------------- decode step
+struct StepParams {
+    const void* q; const void* k; const void* v;            // projections of the token
+    const void* low; const bf16* up; const bf16* up_bias; int rank;      // decay logits: up [heads * dim, rank] low + bias
+    const void* beta; const bf16* a_log;
+    const bf16* q_taps; const bf16* k_taps; const bf16* v_taps; int taps; void* history;
+    float tau;
+    const void* gate_low; const bf16* gate_up; int gate_rank;            // gate_up == NULL: gate_low is the gate itself
+    const bf16* norm; float eps;
+    const int* position_ptr; int position;
+    float* state; void* out;
+    int heads, kv_heads, dim, vdim;
+};
+
+constexpr int kStepThreads = 256, kStepGroups = 8;
+
+// dot(up[row, :rank], low) by the eight lanes of a group; every lane gets the sum
+QD_DEVINL float low_rank_dot(const bf16* up, const float* low, int rank, int sub) {
+    float acc = 0.f;
+    if (rank % 8 == 0) {
+        for (int r = sub * 8; r < rank; r += 64) {
+            float w[8];
+            unpack8(__ldg(reinterpret_cast<const uint4*>(up + r)), w);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) acc = fmaf(w[i], low[r + i], acc);
+        }
+    } else {
+        for (int r = sub; r < rank; r += 8) acc = fmaf(ld_bf16(up + r), low[r], acc);
+    }
+    return group_sum<8>(acc);
+}
+
+template <typename T, bool DELTA, int KPT>
+__global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const __grid_constant__ StepParams p) {
+    chain_enter();
+    extern __shared__ float low[];                 // rank + gate_rank
+    __shared__ float sq[256], sk[256], sg[256], sv[32], sgate[32], part[kStepGroups][33], red[33], squares[8];
+    cg::cluster_group cluster = cg::this_cluster();
+    cluster.barrier_arrive();                      // waited for before the first access to another block's memory
+    const int head = blockIdx.y, c0 = blockIdx.x * 32, tid = threadIdx.x, col = tid & 31, kg = tid >> 5;
+    const int dim = p.dim, vdim = p.vdim, kv = head / (p.heads / p.kv_heads), kv_keys = p.kv_heads * dim;
+    const bool col_ok = c0 + col < vdim;
+    float* tile = p.state + (size_t)head * dim * vdim + c0 + col;
+    float s[KPT];
+#pragma unroll
+    for (int j = 0; j < KPT; ++j) {
+        const int r = j * kStepGroups + kg;
+        s[j] = (r < dim && col_ok) ? tile[(size_t)r * vdim] : 0.f;
+    }
+    const T* lowv = reinterpret_cast<const T*>(p.low);
+    const T* gatev = reinterpret_cast<const T*>(p.gate_low);
+    for (int i = tid; i < p.rank; i += kStepThreads) low[i] = load_f(lowv + i);
+    if (p.gate_up) for (int i = tid; i < p.gate_rank; i += kStepThreads) low[p.rank + i] = load_f(gatev + i);
+    const T* q = reinterpret_cast<const T*>(p.q) + kv * dim;
+    const T* k = reinterpret_cast<const T*>(p.k) + kv * dim;
+    const T* v = reinterpret_cast<const T*>(p.v) + head * vdim + c0;
+    const float scale = 1.0f / sqrtf((float)dim);
+    const int position = p.position_ptr ? *p.position_ptr : p.position;
+    float qv = 0.f, kvv = 0.f;
+    if (DELTA) {
+        const ConvSource src = {p.history, p.taps, 2 * kv_keys + p.heads * vdim};
+        T* fresh = reinterpret_cast<T*>(p.history) + (size_t)(position % p.taps) * src.channels;
+        if (tid < dim) {
+            const int c = kv * dim + tid;
+            qv = silu_precise(conv_at(q + tid, 0, 0, position, p.q_taps + (size_t)c * p.taps, src, c));
+            kvv = silu_precise(conv_at(k + tid, 0, 0, position, p.k_taps + (size_t)c * p.taps, src, kv_keys + c));
+            if (blockIdx.x == 0 && head % (p.heads / p.kv_heads) == 0) { fresh[c] = q[tid]; fresh[kv_keys + c] = k[tid]; }
+        }
+        if (tid < 32 && col_ok) {
+            const int c = head * vdim + c0 + tid;
+            sv[tid] = silu_precise(conv_at(v + tid, 0, 0, position, p.v_taps + (size_t)c * p.taps, src, 2 * kv_keys + c));
+            fresh[2 * kv_keys + c] = v[tid];
+        }
+        const float qq = block_sum(qv * qv, red), kk = block_sum(kvv * kvv, red);
+        qv *= scale / sqrtf(qq + kUnitEps);
+        kvv *= 1.0f / sqrtf(kk + kUnitEps);
+    } else {
+        if (tid < dim) { qv = load_f(q + tid) * scale; kvv = load_f(k + tid); }
+        if (tid < 32 && col_ok) sv[tid] = load_f(v + tid);
+        __syncthreads();
+    }
+    if (tid < 256) { sq[tid] = qv; sk[tid] = kvv; }
+    // decay of the head's key channels, output gate of the block's columns: eight lanes per row
+    const int sub = tid & 7, group = tid >> 3;
+    for (int d = group; d < ((dim + 31) & ~31); d += 32) {
+        const int row = head * dim + min(d, dim - 1);
+        const float z = low_rank_dot(p.up + (size_t)row * p.rank, low, p.rank, sub) + ld_bf16(p.up_bias + row);
+        if (sub == 0 && d < dim) sg[d] = DELTA ? delta_decay(z, ld_bf16(p.a_log + head)) : gla_decay(z, 1.0f / p.tau);
+    }
+    {
+        const int c = head * vdim + min(c0 + group, vdim - 1);
+        const float gv = p.gate_up ? low_rank_dot(p.gate_up + (size_t)c * p.gate_rank, low + p.rank, p.gate_rank, sub) : load_f(gatev + c);
+        if (sub == 0) sgate[group] = DELTA ? sigmoid_precise(gv) : silu_precise(gv);
+    }
+    __syncthreads();
+
+    float pred = 0.f;
+#pragma unroll
+    for (int j = 0; j < KPT; ++j) {
+        const int r = j * kStepGroups + kg;
+        if (r < dim) {
+            s[j] *= sg[r];
+            if (DELTA) pred = fmaf(s[j], sk[r], pred);
+        }
+    }
+    float u = col_ok ? sv[col] : 0.f;
+    if (DELTA) {
+        part[kg][col] = pred;
+        __syncthreads();
+        float total = 0.f;
+#pragma unroll
+        for (int w = 0; w < kStepGroups; ++w) total += part[w][col];
+        u = sigmoid_precise(load_f(reinterpret_cast<const T*>(p.beta) + head)) * (u - total);
+        __syncthreads();
+    }
+    float o = 0.f;
+#pragma unroll
+    for (int j = 0; j < KPT; ++j) {
+        const int r = j * kStepGroups + kg;
+        if (r < dim) {
+            s[j] = fmaf(sk[r], u, s[j]);
+            o = fmaf(s[j], sq[r], o);
+            if (col_ok) tile[(size_t)r * vdim] = s[j];
+        }
+    }
+    part[kg][col] = o;
+    __syncthreads();
+    cluster.barrier_wait();
+    float value = 0.f;
+    if (kg == 0) {
+#pragma unroll
+        for (int w = 0; w < kStepGroups; ++w) value += part[w][col];
+        if (!col_ok) value = 0.f;
+        const float mine = warp_sum(value * value);
+        // this block's sum of squares into slot `rank` of every block of the head
+        if (col < (int)cluster.num_blocks()) *cluster.map_shared_rank(&squares[cluster.block_rank()], col) = mine;
+    }
+    cluster.sync();
+    if (kg == 0 && col_ok) {
+        float total = 0.f;
+        for (unsigned int b = 0; b < cluster.num_blocks(); ++b) total += squares[b];
+        const float r = 1.0f / sqrtf(total / (float)vdim + p.eps);
+        store_f(reinterpret_cast<T*>(p.out) + head * vdim + c0 + col, value * r * ld_bf16(p.norm + c0 + col) * sgate[col]);
+    }
+}
+
+template <typename T, bool DELTA, int KPT>
+int launch_step(const StepParams& p, cudaStream_t stream) {
+    const int slices = (p.vdim + 31) / 32;
+    if (slices > 8) return QD_ERR_UNSUPPORTED;
+    const size_t smem = (size_t)(p.rank + p.gate_rank) * 4 + 16;
+    if (!allow_smem(recurrence_step_kernel<T, DELTA, KPT>, smem)) return QD_ERR_UNSUPPORTED;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(slices, p.heads); cfg.blockDim = dim3(kStepThreads); cfg.dynamicSmemBytes = smem; cfg.stream = stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = slices; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr; cfg.numAttrs = qd_chain_switch() ? 2 : 1;
+    return cudaLaunchKernelEx(&cfg, recurrence_step_kernel<T, DELTA, KPT>, p) == cudaSuccess ? QD_OK : QD_ERR_LAUNCH;
+}
+template <typename T, bool DELTA>
+int step(const StepParams& p, cudaStream_t stream) {
+    if (p.dim <= 32) return launch_step<T, DELTA, 4>(p, stream);
+    if (p.dim <= 64) return launch_step<T, DELTA, 8>(p, stream);
+    if (p.dim <= 128) return launch_step<T, DELTA, 16>(p, stream);
+    if (p.dim <= 256) return launch_step<T, DELTA, 32>(p, stream);
+    return QD_ERR_UNSUPPORTED;
+}
+
+template <typename T, bool DELTA>
+int prepare(const PrepareParams& p, int tokens, cudaStream_t s) {
+    if (DELTA) return qd_launch(delta_prepare_kernel<T>, dim3(tokens), dim3(256), 0, s, 1, p);
+    return qd_launch(gla_prepare_kernel<T>, dim3(tokens), dim3(256), 0, s, 1, p);
+}
+template <typename T>
+int history(const void* q, const void* k, const void* v, long long ld, void* ring, int taps, int kv_keys, int values, int tokens,
+            const int* position_ptr, int position, cudaStream_t s) {
+    const int rows = tokens < taps ? tokens : taps;
+    return qd_launch(conv_history_kernel<T>, dim3((2 * kv_keys + values + 255) / 256, rows), dim3(256), 0, s, 1, (const T*)q, (const T*)k,
+                     (const T*)v, ld, (T*)ring, taps, kv_keys, values, tokens, position_ptr, position);
+}
+template <typename T>
+int norm_gate(const float* x, const void* w, const void* gate, long long ld, void* out, int tokens, int heads, int vdim, float eps,
+              int act, cudaStream_t s) {
+    return qd_launch(head_norm_gate_kernel<T>, dim3((unsigned)(((long long)tokens * heads + 7) / 8)), dim3(256), 0, s, 1, x, (const bf16*)w,
+                     (const T*)gate, ld, (T*)out, tokens, heads, vdim, eps, act);
+}
+
+}  // namespace
+}  // namespace qd
+
+extern "C" int qd_gla_prepare(const void* q, const void* k, const void* v, long long ld, const float* z, const void* z_bias,
+                              float tau, float* oq, float* ok, float* og, float* ov, int tokens, int heads, int dim, int vdim,
+                              int dtype, void* stream) {
+    QD_CHECK_ARG(q && k && v && z && z_bias && oq && ok && og && ov && tokens > 0 && heads > 0 && dim > 0 && vdim > 0 && tau > 0.f);
+    qd::PrepareParams p = {};
+    p.q = q; p.k = k; p.v = v; p.ld = ld; p.z = z; p.z_bias = (const bf16*)z_bias; p.tau = tau;
+    p.oq = oq; p.ok = ok; p.og = og; p.ov = ov; p.heads = heads; p.kv_heads = heads; p.dim = dim; p.vdim = vdim;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == QD_BF16) return qd::prepare<bf16, false>(p, tokens, s);
+    if (dtype == QD_F32) return qd::prepare<float, false>(p, tokens, s);
+    return QD_ERR_UNSUPPORTED;
+}
+
+extern "C" int qd_channel_delta_prepare(const void* q, const void* k, const void* v, const void* beta, long long ld, const float* z,
+                                        const void* z_bias, const void* a_log, const void* q_taps, const void* k_taps,
+                                        const void* v_taps, void* history, int taps, const int* position_ptr, int position,
+                                        float* oq, float* ok, float* og, float* ov, float* obeta, float* okq, int tokens, int heads,
+                                        int kv_heads, int dim, int vdim, int dtype, void* stream) {
+    QD_CHECK_ARG(q && k && v && beta && z && z_bias && a_log && q_taps && k_taps && v_taps && history && oq && ok && og && ov && obeta && okq);
+    QD_CHECK_ARG(tokens > 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && vdim > 0 && taps > 0 && position >= 0);
+    if (dim > 32 * qd::kMaxPerLane) return QD_ERR_UNSUPPORTED;
+    const int kv_keys = kv_heads * dim, values = heads * vdim;
+    qd::PrepareParams p = {q, k, v, ld, z, (const bf16*)z_bias, beta, (const bf16*)a_log, (const bf16*)q_taps, (const bf16*)k_taps,
+                           (const bf16*)v_taps, {history, taps, 2 * kv_keys + values}, 1.f, position_ptr, position, oq, ok, og, ov,
+                           obeta, okq, heads, kv_heads, dim, vdim};
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype != QD_BF16 && dtype != QD_F32) return QD_ERR_UNSUPPORTED;
+    const int rc = dtype == QD_BF16 ? qd::prepare<bf16, true>(p, tokens, s) : qd::prepare<float, true>(p, tokens, s);
+    if (rc != QD_OK) return rc;
+    return dtype == QD_BF16 ? qd::history<bf16>(q, k, v, ld, history, taps, kv_keys, values, tokens, position_ptr, position, s)
+                            : qd::history<float>(q, k, v, ld, history, taps, kv_keys, values, tokens, position_ptr, position, s);
+}
+
+extern "C" int qd_linear_recurrence(const float* q, const float* k, const float* g, const float* v, const float* beta, const float* kq,
+                                    float* state, float* out, int tokens, int heads, int kv_heads, int dim, int vdim, int delta,
+                                    void* stream) {
+    QD_CHECK_ARG(q && k && g && v && state && out && tokens > 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && vdim > 0);
+    QD_CHECK_ARG(!delta || (beta && kq));
+    const int vectors = dim % 4 == 0 && vdim % 4 == 0 && qd::aligned16(q) && qd::aligned16(k) && qd::aligned16(g) && qd::aligned16(v);
+    const qd::RecurrenceParams p = {q, k, g, v, beta, kq, state, out, tokens, heads, kv_heads, dim, vdim, vectors};
+    return delta ? qd::recurrence<true>(p, (cudaStream_t)stream) : qd::recurrence<false>(p, (cudaStream_t)stream);
+}
+
+extern "C" int qd_head_norm_gate(const float* x, const void* w, const void* gate, long long ld_gate, void* out, int tokens, int heads,
+                                 int vdim, float eps, int act, int dtype, void* stream) {
+    QD_CHECK_ARG(x && w && gate && out && tokens > 0 && heads > 0 && vdim > 0 && (act == 0 || act == 1));
+    if (dtype == QD_BF16) return qd::norm_gate<bf16>(x, w, gate, ld_gate, out, tokens, heads, vdim, eps, act, (cudaStream_t)stream);
+    if (dtype == QD_F32) return qd::norm_gate<float>(x, w, gate, ld_gate, out, tokens, heads, vdim, eps, act, (cudaStream_t)stream);
+    return QD_ERR_UNSUPPORTED;
+}
+
+extern "C" int qd_gla_step(const void* q, const void* k, const void* v, const void* low, const void* up, const void* up_bias, int rank,
+                           float tau, const void* gate, const void* norm, float eps, float* state, void* out, int heads, int dim,
+                           int vdim, int dtype, void* stream) {
+    QD_CHECK_ARG(q && k && v && low && up && up_bias && gate && norm && state && out && rank > 0 && heads > 0 && dim > 0 && vdim > 0 && tau > 0.f);
+    qd::StepParams p = {};
+    p.q = q; p.k = k; p.v = v; p.low = low; p.up = (const bf16*)up; p.up_bias = (const bf16*)up_bias; p.rank = rank; p.tau = tau;
+    p.gate_low = gate; p.norm = (const bf16*)norm; p.eps = eps; p.state = state; p.out = out;
+    p.heads = heads; p.kv_heads = heads; p.dim = dim; p.vdim = vdim; p.taps = 1;
+    if (dtype == QD_BF16) return qd::step<bf16, false>(p, (cudaStream_t)stream);
+    if (dtype == QD_F32) return qd::step<float, false>(p, (cudaStream_t)stream);
+    return QD_ERR_UNSUPPORTED;
+}
+
+extern "C" int qd_channel_delta_step(const void* q, const void* k, const void* v, const void* beta, const void* low, const void* up,
+                                     const void* up_bias, int rank, const void* a_log, const void* q_taps, const void* k_taps,
+                                     const void* v_taps, void* history, int taps, const int* position_ptr, int position,
+                                     const void* gate_low, const void* gate_up, int gate_rank, const void* norm, float eps,
+                                     float* state, void* out, int heads, int kv_heads, int dim, int vdim, int dtype, void* stream) {
+    QD_CHECK_ARG(q && k && v && beta && low && up && up_bias && a_log && q_taps && k_taps && v_taps && history && gate_low && gate_up && norm);
+    QD_CHECK_ARG(state && out && rank > 0 && gate_rank > 0 && taps > 0 && position >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0);
+    QD_CHECK_ARG(dim > 0 && vdim > 0);
+    const qd::StepParams p = {q, k, v, low, (const bf16*)up, (const bf16*)up_bias, rank, beta, (const bf16*)a_log, (const bf16*)q_taps,
+                              (const bf16*)k_taps, (const bf16*)v_taps, taps, history, 1.f, gate_low, (const bf16*)gate_up, gate_rank,
+                              (const bf16*)norm, eps, position_ptr, position, state, out, heads, kv_heads, dim, vdim};
+    if (dtype == QD_BF16) return qd::step<bf16, true>(p, (cudaStream_t)stream);
+    if (dtype == QD_F32) return qd::step<float, true>(p, (cudaStream_t)stream);
+    return QD_ERR_UNSUPPORTED;
+}

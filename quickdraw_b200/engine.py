@@ -12,8 +12,12 @@ Prompts run in chunks of ``prefill_chunk_size`` tokens through the sequence path
 (tensor-core products; the reference's default chunk is 128, here 2048 because larger chunks
 amortise the expert weights better) where the fused step applies, token by token otherwise.
 
+Which model design a checkpoint belongs to is looked up in ``registry.py``: it decides what holds
+the history and what advances it.  ``extend`` continues the current request by given tokens and
+returns the logits at chosen places (a replayed trace, a scored continuation).
+
 Backends: ``"b200"`` (default) runs the fused CUDA step where the checkpoint has the
-36B-A3B widths and the composed operator table otherwise; passing ``kernels=`` or
+36B-A3B widths (or is a bf16-weight hybrid) and the composed operator table otherwise; passing ``kernels=`` or
 ``step=`` gives the ``"custom"`` backend used by tests (no graph).  There is no CPU
 backend: on a CPU device only a caller-supplied ``step`` can run.
 """
@@ -24,33 +28,33 @@ from dataclasses import dataclass
 
 import torch
 
-from .state import DecodeState
-from .weights import Checkpoint
+from .registry import design_of, design_of_directory
+from .weights import Checkpoint, FezopelCheckpoint
 
 
 @dataclass
 class Snapshot:
-    """A request's history at one point: the token ids processed so far, the recurrent and
-    convolution tensors (copies), the position and the pending token.  The KV cache is not
-    copied: its rows below ``position`` stay valid as long as the engine only continues from a
-    restored snapshot or starts over (rows at or beyond the position are rewritten before they
-    are read).  Bound to the checkpoint and the execution settings it was taken under."""
+    """A request's history at one point: the token ids processed so far, copies of the tensors
+    the state calls its ``history`` (recurrent and convolution state; windowed key/value rings),
+    the position and the pending token.  A full-length KV cache is not copied: its rows below
+    ``position`` stay valid as long as the engine only continues from a restored snapshot or starts
+    over (rows at or beyond the position are rewritten before they are read).  Bound to the
+    checkpoint and the execution settings it was taken under."""
     tokens: tuple[int, ...]
     position: int
     pending_token: torch.Tensor | None
-    rec_state: torch.Tensor
-    conv_state: torch.Tensor
+    history: tuple[torch.Tensor, ...]
     binding: tuple
 
     def nbytes(self) -> int:
-        return self.rec_state.nbytes + self.conv_state.nbytes
+        return sum(t.nbytes for t in self.history)
 
 
 class Engine:
-    def __init__(self, ckpt: Checkpoint, max_context: int = 32768, device: str = "cuda",
+    def __init__(self, ckpt: Checkpoint | FezopelCheckpoint, max_context: int = 32768, device: str = "cuda",
                  backend: str | None = None, *, kernels: dict | None = None, step=None,
                  cuda_graph: bool = True, prefill_chunk_size: int = 2048,
-                 sequence_prefill: bool = True, _step_object=None):
+                 sequence_prefill: bool = True, dtype: torch.dtype = torch.bfloat16, _step_object=None):
         custom = kernels is not None or step is not None
         if backend is None:
             backend = "custom" if custom else "b200"
@@ -58,7 +62,10 @@ class Engine:
         assert kernels is None or step is None
         assert backend == "custom" or not custom
         assert max_context > 0 and prefill_chunk_size > 0
+        design = design_of(ckpt)
+        assert dtype in design.dtypes, f"{design.name} does not run in {dtype}"
         self.ckpt, self.max_context, self.device, self.backend = ckpt, max_context, device, backend
+        self.design, self.dtype = design, dtype
         self.prefill_chunk_size = prefill_chunk_size
         self.sequence_prefill = False      # set below where the chunked path applies
         self.chunk_prefill = None
@@ -75,7 +82,12 @@ class Engine:
             assert on_cuda, "the b200 backend needs a CUDA device; there is no CPU path"
             from . import fused
             from .kernels import bind_kernels
-            if kernels is None and fused.supports(ckpt):
+            if design.library == "hybrid":
+                assert kernels is None, "the operator table is for NVFP4 checkpoints"
+                from .hybrid import HybridModel
+                self.fused = self.step = self.chunk_prefill = HybridModel(ckpt, dtype)
+                self.sequence_prefill = sequence_prefill
+            elif kernels is None and fused.supports(ckpt):
                 self.fused = fused.FusedStep(ckpt)
                 self.step = self.fused
                 if sequence_prefill and all(fused.mixer_format(layer) in ("nvfp4", "fp8") for layer in ckpt.layers):
@@ -86,7 +98,7 @@ class Engine:
                 prepared = ([(1 + l.input_layernorm.float(), 1 + l.post_attention_layernorm.float())
                              for l in ckpt.layers], 1 + ckpt.final_norm.float())
                 self.step = bind_kernels(prepared=prepared, **(kernels or {}))["forward_step"]
-        self.state = DecodeState.allocate(ckpt.config, max_context, device)
+        self.state = design.allocate(ckpt.config, max_context, device, prefill_chunk_size, dtype)
         self.history: list[int] = []            # token ids processed since the last reset (prompt part; see _fold)
         self._decoded: list[torch.Tensor] = []  # tokens processed by decode steps, still on the device
         self._kv_tokens: list[int] = []         # the token sequence the cache rows [0, n) were computed from
@@ -106,9 +118,7 @@ class Engine:
         self._decode_input = torch.zeros((), dtype=torch.long, device=dev)
         self._device_position = torch.zeros((), dtype=torch.int32, device=dev)
         self._decode_output = torch.empty((), dtype=torch.long, device=dev)
-        scratch = DecodeState(torch.empty_like(self.state.kv_k), torch.empty_like(self.state.kv_v),
-                              torch.zeros_like(self.state.rec_state),
-                              torch.zeros_like(self.state.conv_state), 0)
+        scratch = self.state.blank()
         stream = torch.cuda.Stream(device=dev)
         stream.wait_stream(torch.cuda.current_stream(dev))
         with torch.cuda.stream(stream):
@@ -144,27 +154,59 @@ class Engine:
         self.reset()
         return self._extend(list(token_ids))
 
-    def _extend(self, token_ids: list[int]) -> torch.Tensor:
-        """Process ``token_ids`` after the current position; logits after the last one."""
-        start = self.state.position
+    def _extend(self, token_ids: list[int], want=None):
+        """Process ``token_ids`` after the current position: logits after the last one, or with ``want`` (ascending
+        places among the tokens) a list of the logits at those places."""
+        start, count = self.state.position, len(token_ids)
+        asked = [count - 1] if want is None else want
         tokens = torch.tensor(token_ids, dtype=torch.long, device=self.device)
-        logits = None
+        found: list[torch.Tensor] = []
         done = 0
-        if self.sequence_prefill and len(token_ids) > 1:
-            while done < len(token_ids) - 1:
-                stop = min(len(token_ids) - 1, done + self.prefill_chunk_size)
-                self.chunk_prefill.run(tokens[done:stop], start + done, self.state)
+        while done < count:
+            ahead = next((w for w in asked if w >= done), count)
+            # tokens that a chunk takes: a design whose chunks return logits takes all of them, otherwise those
+            # before the next wanted one
+            whole = self.sequence_prefill and self.design.chunk_logits
+            stop = min(count if whole else ahead, done + self.prefill_chunk_size)
+            if self.sequence_prefill and stop > done + (1 if whole else 0):
+                if whole:
+                    inside = [w - done for w in asked if done <= w < stop]
+                    rows = self.chunk_prefill.run(tokens[done:stop], start + done, self.state, inside)
+                    found += [] if rows is None else list(rows)
+                else:
+                    self.chunk_prefill.run(tokens[done:stop], start + done, self.state)
                 done = stop
-            self.state.position = start + done
-        for index, token in enumerate(tokens[done:], start=done):
-            if self.backend == "b200":
-                logits = self.step(self.ckpt, token, self.state.position, self.state,
-                                   logits=index == len(tokens) - 1)
+                self.state.position = start + done
+                continue
+            token, wanted = tokens[done], done == ahead
+            if self.graph is not None and wanted and self.design.chunk_logits:
+                logits = self._replay(token).clone()
+            elif self.backend == "b200":
+                logits = self.step(self.ckpt, token, self.state.position, self.state, logits=wanted)
             else:
                 logits = self.step(self.ckpt, token, self.state.position, self.state)
+            if wanted:
+                found.append(logits)
+            done += 1
             self.state.position += 1
         self._note([int(t) for t in token_ids])
-        return logits
+        return found[-1] if want is None else found
+
+    @torch.inference_mode()
+    def extend(self, token_ids: list[int], want=()) -> torch.Tensor:
+        """Continue the current request by ``token_ids``; fp32 logits [len(want), vocab] at the places ``want``
+        among them, in the order given.  ``reset`` starts a request."""
+        config = self.ckpt.config
+        assert 0 < len(token_ids) and self.state.position + len(token_ids) <= self.max_context, "context capacity reached"
+        assert all(0 <= t < config.vocab_size for t in token_ids), "token id outside the vocabulary"
+        assert all(0 <= w < len(token_ids) for w in want), "a wanted place lies outside the tokens"
+        self._fold()
+        self.pending_token = None
+        places = sorted(set(want))
+        rows = dict(zip(places, self._extend(list(token_ids), places)))
+        if not want:
+            return torch.empty((0, config.vocab_size), dtype=torch.float32, device=self.device)
+        return torch.stack([rows[w].float() for w in want])
 
     def _note(self, ids: list[int]) -> None:
         """Record tokens processed at the positions after ``history`` and what that did to the
@@ -194,8 +236,8 @@ class Engine:
         todo.md "Conversation reuse").  75 MB of copies for the 36B-A3B model, no KV copy."""
         self._fold()
         pending = None if self.pending_token is None else self.pending_token.clone()
-        return Snapshot(tuple(self.history), self.state.position, pending, self.state.rec_state.clone(),
-                        self.state.conv_state.clone(), self._binding())
+        return Snapshot(tuple(self.history), self.state.position, pending, tuple(t.clone() for t in self.state.history()),
+                        self._binding())
 
     @torch.inference_mode()
     def restore(self, snap: Snapshot) -> None:
@@ -205,14 +247,14 @@ class Engine:
         self._fold()
         assert snap.binding == self._binding(), "snapshot taken under another checkpoint or other settings"
         assert self._kv_covers(snap.tokens), "the cache rows of this snapshot have been overwritten"
-        self.state.rec_state.copy_(snap.rec_state)
-        self.state.conv_state.copy_(snap.conv_state)
+        for kept, copy in zip(self.state.history(), snap.history):
+            kept.copy_(copy)
         self.state.position = snap.position
         self.pending_token = None if snap.pending_token is None else snap.pending_token.clone()
         self.history = list(snap.tokens)
 
     def _kv_covers(self, tokens) -> bool:
-        return len(tokens) <= len(self._kv_tokens) and list(tokens) == self._kv_tokens[:len(tokens)]
+        return not self.state.keeps_every_row or len(tokens) <= len(self._kv_tokens) and list(tokens) == self._kv_tokens[:len(tokens)]
 
     @torch.inference_mode()
     def prefill_reuse(self, token_ids: list[int], snap: Snapshot | None = None) -> torch.Tensor:
@@ -238,13 +280,16 @@ class Engine:
 
     @classmethod
     def from_pretrained(cls, path: str, **kwargs) -> "Engine":
-        """Load a checkpoint directory (safetensors shards), merge the static FP8 scales of the
-        projections that share an activation, and build the engine (reference:
+        """Load a checkpoint directory of any registered design and build the engine (reference:
         quickdraw/engine/engine.py:85-90)."""
-        from .loader import load_checkpoint, merge_fp8_scales
-        ckpt = load_checkpoint(path, device=kwargs.get("device", "cuda"))
-        merge_fp8_scales(ckpt)
-        return cls(ckpt, **kwargs)
+        return cls(design_of_directory(path).load(path, kwargs.get("device", "cuda")), **kwargs)
+
+    def _replay(self, token: torch.Tensor) -> torch.Tensor:
+        """The captured step on ``token`` at the current position; its logits (overwritten by the next replay)."""
+        self._decode_input.copy_(token)
+        self._device_position.fill_(self.state.position)
+        self.graph.replay()
+        return self._decode_logits
 
     @torch.inference_mode()
     def decode_step(self) -> torch.Tensor:
@@ -259,9 +304,7 @@ class Engine:
             watchdog = getattr(self.step, "watchdog", None)
             if watchdog is not None:
                 watchdog.check()        # expert parallel: a lost peer raises here, before the launch
-            self._decode_input.copy_(self.pending_token)
-            self._device_position.fill_(self.state.position)
-            self.graph.replay()
+            self._replay(self.pending_token)
             self.pending_token = self._decode_output.clone()
         self.state.position += 1
         return self.pending_token

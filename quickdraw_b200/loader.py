@@ -21,12 +21,14 @@ from __future__ import annotations
 import json
 import re
 from contextlib import ExitStack
+from dataclasses import fields
 from pathlib import Path
 
 import torch
 
-from .weights import (Checkpoint, FP8Linear, FullAttnWeights, GDNWeights, LayerWeights, ModelConfig,
-                      MoEWeights, NVFP4Linear)
+from .weights import (ChannelDeltaConfig, ChannelDeltaWeights, Checkpoint, FezopelCheckpoint, FezopelConfig, FP8Linear,
+                      FullAttnWeights, GDNWeights, GeluMLPWeights, GLAConfig, GLAWeights, HybridLayerWeights, LayerWeights,
+                      ModelConfig, MoEWeights, NormWeights, NVFP4Linear, SublayerWeights, WindowAttnConfig, WindowAttnWeights)
 
 ROOT = "model.language_model."
 LAYER_NAME = re.compile(r"model\.language_model\.layers\.(\d+)\.")
@@ -46,8 +48,13 @@ class ShardReader:
     def __init__(self, directory: Path, stack: ExitStack):
         from safetensors import safe_open
         self.directory, self.stack, self._open = directory, stack, safe_open
-        self.weight_map: dict[str, str] = json.loads((directory / "model.safetensors.index.json").read_text())["weight_map"]
         self.handles: dict[str, object] = {}
+        index, single = directory / "model.safetensors.index.json", "model.safetensors"
+        if index.exists():
+            self.weight_map: dict[str, str] = json.loads(index.read_text())["weight_map"]
+        else:                    # one file, no index
+            self.handles[single] = stack.enter_context(safe_open(directory / single, framework="pt"))
+            self.weight_map = {name: single for name in self.handles[single].keys()}
 
     def __contains__(self, name: str) -> bool:
         return name in self.weight_map
@@ -270,3 +277,94 @@ def save_checkpoint(ckpt: Checkpoint, path: str | Path, shards: int = 2, text_co
     config = asdict(ckpt.config)
     theta = config.pop("rope_theta")
     (directory / "config.json").write_text(json.dumps({"text_config": dict(config, rope_parameters={"rope_theta": theta}, **(text_config or {}))}))
+
+
+# ------------------------------------------------------------------ bf16-weight hybrids
+# field of a mixer's container -> tensor name below "<layer>.mix."
+HYBRID_FIELDS = {
+    WindowAttnConfig: (WindowAttnWeights, {"q_norm": "q.norm", "k_norm": "k.norm"}),
+    GLAConfig: (GLAWeights, {"a2_b": "a2.b"}),
+    ChannelDeltaConfig: (ChannelDeltaWeights, {"q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv"}),
+}
+
+
+def hybrid_shapes(config: FezopelConfig, low_rank=lambda name: None) -> dict[str, tuple]:
+    """Every tensor name of the checkpoint and its shape; None where only the tensor knows it (the
+    inner size of the low-rank products, unless ``low_rank(name of the inner matrix)`` tells)."""
+    w = config.hidden_size
+    shapes: dict[str, tuple] = {"embed": (config.vocab_size, w), "head": (config.vocab_size, w)}
+
+    def norm(name):
+        shapes[name], shapes[name + ".b"] = (w,), (w,)
+
+    norm("final.norm")
+    for i, layer in enumerate(config.layers):
+        at, m = f"l{i}.", layer.mixer
+        mix, values = at + "mix.", m.heads * m.vdim
+        for which in (("1", "2") if layer.ff is not None else ("1",)):
+            norm(f"{at}norm{which}")
+            norm(f"{at}norm{which}b")
+            shapes[f"{at}rg{which}"], shapes[f"{at}rg{which}.b"] = (w, w), (w,)
+        if layer.ff is not None:
+            shapes[at + "mlp.up"], shapes[at + "mlp.down"] = (layer.ff, w), (w, layer.ff)
+        shapes[at + "dwa"] = (i + 2,)
+        keys = m.heads * m.dim
+        if isinstance(m, WindowAttnConfig):
+            kv_keys, kv_values = m.kv_heads * m.dim, m.kv_heads * m.vdim
+            own = {"q": (keys, w), "k": (kv_keys, w), "v": (kv_values, w), "q.norm": (keys,), "k.norm": (kv_keys,),
+                   "sink": (m.heads,), "g": (m.heads, w)}
+        elif isinstance(m, GLAConfig):
+            r = low_rank(mix + "a1")
+            own = {"q": (keys, w), "k": (keys, w), "v": (values, w), "g": (values, w), "norm": (m.vdim,), "a1": (r, w),
+                   "a2": (keys, r), "a2.b": (keys,)}
+        else:
+            kv_keys, r, rg = m.kv_heads * m.dim, low_rank(mix + "a1"), low_rank(mix + "g1")
+            own = {"q": (kv_keys, w), "k": (kv_keys, w), "v": (values, w), "q.conv": (kv_keys, m.conv),
+                   "k.conv": (kv_keys, m.conv), "v.conv": (values, m.conv), "b": (m.heads, w), "A_log": (m.heads,),
+                   "norm": (m.vdim,), "a1": (r, w), "a2": (keys, r), "dt_bias": (keys,), "g1": (rg, w), "g2": (values, rg)}
+        own["o"] = (w, values)
+        shapes.update({mix + name: shape for name, shape in own.items()})
+    return shapes
+
+
+def assemble_hybrid(config: FezopelConfig, get) -> FezopelCheckpoint:
+    """The containers from ``get(tensor name)``."""
+    norm = lambda name: NormWeights(get(name), get(name + ".b"))
+    around = lambda at, which: SublayerWeights(norm(f"{at}norm{which}"), get(f"{at}rg{which}"), get(f"{at}rg{which}.b"),
+                                               norm(f"{at}norm{which}b"))
+    layers = []
+    for i, layer in enumerate(config.layers):
+        at = f"l{i}."
+        container, renamed = HYBRID_FIELDS[type(layer.mixer)]
+        mixer = container(**{f.name: get(at + "mix." + renamed.get(f.name, f.name)) for f in fields(container)})
+        has_mlp = layer.ff is not None
+        layers.append(HybridLayerWeights(
+            idx=i, mixer=mixer, around_mixer=around(at, "1"), depth=get(at + "dwa"),
+            mlp=GeluMLPWeights(get(at + "mlp.up"), get(at + "mlp.down")) if has_mlp else None,
+            around_mlp=around(at, "2") if has_mlp else None))
+    return FezopelCheckpoint(config=config, embed_tokens=get("embed"), final_norm=norm("final.norm"), lm_head=get("head"),
+                             layers=layers)
+
+
+def load_hybrid_checkpoint(path: str | Path, device: str | torch.device = "cuda") -> FezopelCheckpoint:
+    """A directory with ``config.json`` and safetensors (one file, or shards with an index)."""
+    directory = Path(path)
+    config = FezopelConfig.from_json(directory / "config.json")
+    with ExitStack() as stack:
+        reader = ShardReader(directory, stack)
+        for name, shape in hybrid_shapes(config).items():
+            if name not in reader:
+                raise ValueError(f"{directory}: tensor {name} is missing")
+            found = tuple(reader._handle(name).get_slice(name).get_shape())
+            if len(found) != len(shape) or any(want is not None and have != want for have, want in zip(found, shape)):
+                raise ValueError(f"{directory}: tensor {name} has shape {found}, expected {shape}")
+        return assemble_hybrid(config, lambda name: reader.tensor(name).to(device=device, dtype=torch.bfloat16).contiguous())
+
+
+def save_hybrid_checkpoint(config: FezopelConfig, tensors: dict[str, torch.Tensor], path: str | Path) -> None:
+    """Write ``config.json`` and ``model.safetensors`` as ``load_hybrid_checkpoint`` reads them."""
+    from safetensors.torch import save_file
+    directory = Path(path)
+    directory.mkdir(parents=True, exist_ok=True)
+    (directory / "config.json").write_text(json.dumps(config.to_dict(), indent=1))
+    save_file({name: t.detach().cpu().contiguous().clone() for name, t in tensors.items()}, str(directory / "model.safetensors"))

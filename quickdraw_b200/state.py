@@ -5,11 +5,20 @@ Shapes (reference: quickdraw/engine/engine.py:43-59):
   rec_state   fp32 [linear_layers, value_heads, key_dim, value_dim]
   conv_state  bf16 [linear_layers, conv_channels, conv_width - 1], oldest tap first
 ``position`` counts processed tokens; the engine advances it, the step never does.
+
+``HybridState`` is the same for models whose layers have caches and states of different sizes:
+flat buffers with one view per layer, windowed key/value rings instead of a full-length cache.
 """
 
 from dataclasses import dataclass
 
 import torch
+
+
+def _same_request_buffers(state):
+    """A state of the same shapes whose histories are empty (the buffers of a warm-up run)."""
+    return (torch.empty_like(state.kv_k), torch.empty_like(state.kv_v), torch.zeros_like(state.rec_state),
+            torch.zeros_like(state.conv_state))
 
 
 @dataclass
@@ -23,6 +32,15 @@ class DecodeState:
     def memory_bytes(self) -> dict[str, int]:
         return {name: getattr(self, name).nbytes
                 for name in ("kv_k", "kv_v", "rec_state", "conv_state")}
+
+    keeps_every_row = True       # cache rows of processed positions stay until another request rewrites them
+
+    def blank(self) -> "DecodeState":
+        return DecodeState(*_same_request_buffers(self), 0)
+
+    def history(self) -> list[torch.Tensor]:
+        """What a snapshot copies: everything that later tokens of the request overwrite."""
+        return [self.rec_state, self.conv_state]
 
     @classmethod
     def allocate(cls, config, max_context: int, device) -> "DecodeState":
@@ -39,3 +57,61 @@ class DecodeState:
                 (linear, config.conv_channels, config.linear_conv_kernel_dim - 1),
                 dtype=torch.bfloat16, device=device),
             position=0)
+
+
+@dataclass
+class LayerHistory:
+    """One layer's views: ``k``, ``v`` [capacity, kv_heads, dim / vdim] (attention), ``rec`` fp32
+    [heads, dim, vdim], ``conv`` [taps, channels] (position p in row p mod taps)."""
+    k: torch.Tensor | None = None
+    v: torch.Tensor | None = None
+    rec: torch.Tensor | None = None
+    conv: torch.Tensor | None = None
+
+
+class HybridState:
+    """History of one request of a bf16-weight hybrid.  An attention layer keeps the last ``capacity``
+    positions, position p in row p mod capacity: the window plus the rows a prompt chunk of ``chunk``
+    tokens adds before its first token has attended.  Rows are only read for positions of the current
+    request, so a reset leaves them."""
+
+    keeps_every_row = False
+
+    def __init__(self, config, max_context: int, device, chunk: int = 2048, dtype: torch.dtype = torch.bfloat16):
+        self._args = (config, max_context, device, chunk, dtype)
+        self.position = 0
+        plans, sizes = [], {"kv_k": 0, "kv_v": 0, "rec_state": 0, "conv_state": 0}
+
+        def take(buffer: str, *shape: int):
+            start, count = sizes[buffer], 1
+            for n in shape:
+                count *= n
+            sizes[buffer] += -(-count // 64) * 64            # every view starts on a 128-byte boundary
+            return buffer, start, count, shape
+
+        for layer in config.layers:
+            m, plan = layer.mixer, {}
+            if hasattr(m, "window"):
+                capacity = min(max_context, m.window - 1 + chunk)
+                plan["k"] = take("kv_k", capacity, m.kv_heads, m.dim)
+                plan["v"] = take("kv_v", capacity, m.kv_heads, m.vdim)
+            else:
+                plan["rec"] = take("rec_state", m.heads, m.dim, m.vdim)
+                if hasattr(m, "conv"):
+                    plan["conv"] = take("conv_state", m.conv, 2 * m.kv_heads * m.dim + m.heads * m.vdim)
+            plans.append(plan)
+        for buffer, size in sizes.items():
+            fresh = torch.empty if buffer.startswith("kv") else torch.zeros
+            kind = torch.float32 if buffer == "rec_state" else dtype
+            setattr(self, buffer, fresh(size, dtype=kind, device=device))
+        self.layers = [LayerHistory(**{name: getattr(self, buffer)[start:start + count].view(shape)
+                                       for name, (buffer, start, count, shape) in plan.items()}) for plan in plans]
+
+    def blank(self) -> "HybridState":
+        return HybridState(*self._args)
+
+    def history(self) -> list[torch.Tensor]:
+        return [self.rec_state, self.conv_state, self.kv_k, self.kv_v]
+
+    def memory_bytes(self) -> dict[str, int]:
+        return {name: getattr(self, name).nbytes for name in ("kv_k", "kv_v", "rec_state", "conv_state")}

@@ -18,8 +18,8 @@ import zlib
 
 import torch
 
-from .weights import (Checkpoint, FP8Linear, FullAttnWeights, GDNWeights, LayerWeights, ModelConfig,
-                      MoEWeights, NVFP4Linear)
+from .weights import (ChannelDeltaConfig, Checkpoint, FezopelCheckpoint, FezopelConfig, FP8Linear, FullAttnWeights, GDNWeights, GLAConfig,
+                      HybridLayerConfig, LayerWeights, ModelConfig, MoEWeights, NVFP4Linear, WindowAttnConfig)
 
 BF16 = torch.bfloat16
 
@@ -199,3 +199,50 @@ def matvec_case(seed: int = 0, out: int = 1024, inp: int = 2048, device="cpu"):
     scales = (torch.randn(out, inp // 16).abs() * 0.05).clamp(max=448.0).to(torch.float8_e4m3fn)
     proj = NVFP4Linear(codes, scales, torch.tensor(1.0))
     return x.to(device), to_device(proj, device)
+
+
+# ------------------------------------------------------------------ bf16-weight hybrids
+def fezopel_config(num_layers: int = 12, vocab_size: int = 32768, *, hidden: int = 2048, ff: int | None = None,
+                   window: int = 1024, heads: int = 16, kv_heads: int = 4, dim: int = 128) -> FezopelConfig:
+    """Layers of the size of a real model: groups of gated linear attention, channel-decay delta rule and
+    windowed attention; the attention layers carry the feed-forward."""
+    gla = GLAConfig(heads=heads, dim=dim, vdim=dim, tau=16.0)
+    delta = ChannelDeltaConfig(heads=2 * heads, kv_heads=heads, dim=dim, vdim=dim, conv=4)
+    attn = WindowAttnConfig(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, window=window, rotary_dims=dim,
+                            rotary_base=1.0e6, scale=dim ** -0.5)
+    kinds = [HybridLayerConfig(gla, None), HybridLayerConfig(delta, None), HybridLayerConfig(attn, ff or 4 * hidden)]
+    return FezopelConfig(vocab_size=vocab_size, hidden_size=hidden, norm_eps=1e-6,
+                         layers=[kinds[i % 3] for i in range(num_layers)])
+
+
+def fezopel_tensors(config: FezopelConfig, seed: int = 0, device="cpu", rank: int = 16) -> dict[str, torch.Tensor]:
+    """Random tensors under the checkpoint's names: matrices with unit gain, norm weights near one, small
+    biases, decays spread over short and long memories."""
+    from .loader import hybrid_shapes
+    src, out = Source(seed, device), {}
+    for name, shape in hybrid_shapes(config, low_rank=lambda _: rank).items():
+        leaf = name.rsplit(".", 1)[-1]
+        if name == "embed":
+            out[name] = src.normal(name, *shape)
+        elif name.endswith(("dt_bias", "a2.b")):
+            out[name] = src.normal(name, *shape, std=1.5, mean=0.0 if leaf == "dt_bias" else 2.0)
+        elif leaf in ("A_log", "sink"):
+            out[name] = src.normal(name, *shape, std=0.7, mean=-1.0 if leaf == "A_log" else 0.0)
+        elif leaf == "dwa":
+            newest = torch.zeros(shape)
+            newest[-1] = 1.0
+            out[name] = (src.normal(name, *shape, std=0.2).float() + newest.to(src.device)).to(BF16)
+        elif leaf == "conv":
+            out[name] = src.normal(name, *shape, std=shape[1] ** -0.5)
+        elif leaf == "b":
+            out[name] = src.normal(name, *shape, std=0.1 if len(shape) == 1 else shape[1] ** -0.5)
+        elif "norm" in leaf:
+            out[name] = src.normal(name, *shape, std=0.1, mean=1.0)
+        else:
+            out[name] = src.normal(name, *shape, std=shape[-1] ** -0.5)
+    return out
+
+
+def make_fezopel(config: FezopelConfig, seed: int = 0, device="cpu", rank: int = 16) -> FezopelCheckpoint:
+    from .loader import assemble_hybrid
+    return assemble_hybrid(config, fezopel_tensors(config, seed, device, rank).__getitem__)

@@ -168,6 +168,194 @@ class Checkpoint:
     mtp: dict[str, torch.Tensor] = field(default_factory=dict)
 
 
+# ------------------------------------------------- bf16-weight hybrids (fp32 residual stream)
+@dataclass
+class WindowAttnConfig:
+    """Sliding-window attention with sinks; ``window`` counts the token itself."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    window: int
+    rotary_dims: int
+    rotary_base: float
+    scale: float
+
+
+@dataclass
+class GLAConfig:
+    """Gated linear attention; decay = sigmoid(z)^(1 / tau) per key channel."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+
+
+@dataclass
+class ChannelDeltaConfig:
+    """Delta rule with one decay per head and key channel, behind short convolutions."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+
+@dataclass
+class WindowAttnWeights:
+    """Names are the tensor names below ``<layer>.mix.``; all bf16."""
+    q: torch.Tensor
+    k: torch.Tensor
+    v: torch.Tensor
+    g: torch.Tensor
+    o: torch.Tensor
+    q_norm: torch.Tensor
+    k_norm: torch.Tensor
+    sink: torch.Tensor
+
+
+@dataclass
+class GLAWeights:
+    q: torch.Tensor
+    k: torch.Tensor
+    v: torch.Tensor
+    g: torch.Tensor
+    o: torch.Tensor
+    a1: torch.Tensor
+    a2: torch.Tensor
+    a2_b: torch.Tensor
+    norm: torch.Tensor
+
+
+@dataclass
+class ChannelDeltaWeights:
+    q: torch.Tensor
+    k: torch.Tensor
+    v: torch.Tensor
+    b: torch.Tensor
+    o: torch.Tensor
+    q_conv: torch.Tensor
+    k_conv: torch.Tensor
+    v_conv: torch.Tensor
+    A_log: torch.Tensor
+    dt_bias: torch.Tensor
+    a1: torch.Tensor
+    a2: torch.Tensor
+    g1: torch.Tensor
+    g2: torch.Tensor
+    norm: torch.Tensor
+
+
+@dataclass
+class NormWeights:
+    """Layer norm with weight and bias."""
+    w: torch.Tensor
+    b: torch.Tensor
+
+
+@dataclass
+class SublayerWeights:
+    """What surrounds a mixer or a feed-forward: the norm before it, the residual gate
+    (sigmoid(gate h + gate_b) on the result, h the normed input) and the norm after it."""
+    norm: NormWeights
+    gate: torch.Tensor
+    gate_b: torch.Tensor
+    post: NormWeights
+
+
+@dataclass
+class GeluMLPWeights:
+    up: torch.Tensor
+    down: torch.Tensor
+
+
+@dataclass
+class HybridLayerWeights:
+    idx: int
+    mixer: WindowAttnWeights | GLAWeights | ChannelDeltaWeights
+    around_mixer: SublayerWeights
+    mlp: GeluMLPWeights | None
+    around_mlp: SublayerWeights | None
+    depth: torch.Tensor          # weights of the depth average: embedding output, then every layer result
+
+
+@dataclass
+class HybridLayerConfig:
+    mixer: WindowAttnConfig | GLAConfig | ChannelDeltaConfig
+    ff: int | None
+
+
+@dataclass
+class FezopelConfig:
+    vocab_size: int
+    hidden_size: int
+    norm_eps: float
+    layers: list[HybridLayerConfig]
+
+    ARCHITECTURE = "Fezopel"
+
+    @classmethod
+    def from_json(cls, path: str | Path) -> "FezopelConfig":
+        return cls.from_dict(json.loads(Path(path).read_text()))
+
+    @classmethod
+    def from_dict(cls, data: dict) -> "FezopelConfig":
+        if data.get("architecture") != cls.ARCHITECTURE:
+            raise ValueError(f"not a {cls.ARCHITECTURE} configuration: {data.get('architecture')!r}")
+        layers = []
+        for index, entry in enumerate(data["layers"]):
+            m, kind = entry["mixer"], entry["type"]
+            if kind == "attention":
+                mixer = WindowAttnConfig(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"],
+                                         window=m["mask"]["size"], rotary_dims=m["rot"]["dims"],
+                                         rotary_base=float(m["rot"]["base"]), scale=float(m["scale"]))
+            elif kind == "gla":
+                mixer = GLAConfig(heads=m["heads"], dim=m["dim"], vdim=m["vdim"], tau=float(m["tau"]))
+            elif kind == "channel_delta":
+                mixer = ChannelDeltaConfig(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"],
+                                           conv=m["conv"])
+            else:
+                raise ValueError(f"layer {index}: unknown mixer {kind!r}")
+            kv_heads = getattr(mixer, "kv_heads", mixer.heads)
+            if mixer.heads % kv_heads:
+                raise ValueError(f"layer {index}: {mixer.heads} heads do not divide among {kv_heads} key/value heads")
+            mlp = entry["mlp"]
+            if mlp is not None and mlp["kind"] != "dense":
+                raise ValueError(f"layer {index}: unknown feed-forward {mlp['kind']!r}")
+            layers.append(HybridLayerConfig(mixer=mixer, ff=None if mlp is None else mlp["ff"]))
+        return cls(vocab_size=data["vocab"], hidden_size=data["width"], norm_eps=float(data["norm"]["eps"]), layers=layers)
+
+    def to_dict(self) -> dict:
+        """The ``config.json`` this configuration reads from."""
+        layers = []
+        for layer in self.layers:
+            m = layer.mixer
+            entry = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim}
+            if isinstance(m, WindowAttnConfig):
+                kind = "attention"
+                entry |= {"kv_heads": m.kv_heads, "mask": {"size": m.window}, "scale": m.scale,
+                          "rot": {"base": m.rotary_base, "dims": m.rotary_dims}}
+            elif isinstance(m, GLAConfig):
+                kind = "gla"
+                entry |= {"tau": m.tau}
+            else:
+                kind = "channel_delta"
+                entry |= {"kv_heads": m.kv_heads, "conv": m.conv}
+            layers.append({"type": kind, "mixer": entry,
+                           "mlp": None if layer.ff is None else {"kind": "dense", "ff": layer.ff}})
+        return {"architecture": self.ARCHITECTURE, "vocab": self.vocab_size, "width": self.hidden_size,
+                "norm": {"eps": self.norm_eps}, "layers": layers}
+
+
+@dataclass
+class FezopelCheckpoint:
+    config: FezopelConfig
+    embed_tokens: torch.Tensor
+    final_norm: NormWeights
+    lm_head: torch.Tensor
+    layers: list[HybridLayerWeights]
+
+
 CONTAINERS = {cls.__name__: cls for cls in (
     NVFP4Linear, FP8Linear, GDNWeights, FullAttnWeights, MoEWeights, LayerWeights,
     ModelConfig, Checkpoint)}
