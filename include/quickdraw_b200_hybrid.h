@@ -47,14 +47,14 @@ int qd_sublayer_close(const void* y, const void* gate, long long ld_gate, const 
     void* stream);
 
 /* fp32 operands of gated linear attention from a chunk's projections (rows ld apart): oq = q / sqrt(dim), ok = k,
- * ov = v, og = sigmoid(z + z_bias)^(1 / tau). */
+ * ov = v, og = sigmoid(z + z_bias)^(1 / tau) - 1.  og may be z. */
 int qd_gla_prepare(const void* q, const void* k, const void* v, long long ld, const float* z, const void* z_bias,
     float tau, float* oq, float* ok, float* og, float* ov, int tokens, int heads, int dim, int vdim, int dtype, void*
     stream);
 
 /* fp32 operands of the channel-decay delta rule: q, k, v through a causal convolution of `taps` taps (history ring
  * [taps, channels q | k | v], position p in row p mod taps; updated with the chunk's last inputs) and SiLU, q and k as
- * unit vectors per head (q also / sqrt(dim)), og = exp(-exp(a_log) softplus(z + z_bias)), obeta = sigmoid(beta),
+ * unit vectors per head (q also / sqrt(dim)), og = exp(-exp(a_log) softplus(z + z_bias)) - 1 (og may be z), obeta = sigmoid(beta),
  * okq = k . q.  The position of the chunk's first token is *position_ptr, or `position` if that is NULL. */
 int qd_channel_delta_prepare(const void* q, const void* k, const void* v, const void* beta, long long ld, const
     float* z, const void* z_bias, const void* a_log, const void* q_taps, const void* k_taps, const void* v_taps,
@@ -62,7 +62,7 @@ int qd_channel_delta_prepare(const void* q, const void* k, const void* v, const 
     float* obeta, float* okq, int tokens, int heads, int kv_heads, int dim, int vdim, int dtype, void* stream);
 
 /* The recurrence over a chunk; q, k [tokens, kv_heads, dim], g [tokens, heads, dim], v, out [tokens, heads, vdim], state
- * [heads, dim, vdim] fp32, updated in place.  delta = 0: S = diag(g) S + k v^T; 1: S = diag(g) S,
+ * [heads, dim, vdim] fp32, updated in place.  delta = 0: S = diag(1 + g) S + k v^T; 1: S = diag(1 + g) S,
  * u = beta (v - S^T k), S += k u^T; out = S^T q.  dim <= 256. */
 int qd_linear_recurrence(const float* q, const float* k, const float* g, const float* v, const float* beta, const
     float* kq, float* state, float* out, int tokens, int heads, int kv_heads, int dim, int vdim, int delta, void*

@@ -26,8 +26,10 @@ namespace {
 constexpr float kUnitEps = 1e-6f;
 
 QD_DEVINL float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
-QD_DEVINL float gla_decay(float z, float inv_tau) { return expf(log_sigmoid(z) * inv_tau); }
-QD_DEVINL float delta_decay(float z, float a_log) { return expf(-expf(a_log) * softplus_precise(z)); }
+// Decays are carried as decay - 1, S + S (decay - 1) in one FMA: a slow channel's decay is so close to one
+// that its own rounding, the same at every token, would add up over a long sequence.
+QD_DEVINL float gla_decay_less_one(float z, float inv_tau) { return expm1f(log_sigmoid(z) * inv_tau); }
+QD_DEVINL float delta_decay_less_one(float z, float a_log) { return expm1f(-expf(a_log) * softplus_precise(z)); }
 
 // Convolution input history: ring of `taps` rows, position p in row p mod taps.  A step reads the rows of
 // the taps - 1 positions before it and writes its own, which is none of those.
@@ -74,7 +76,7 @@ __global__ void __launch_bounds__(256) gla_prepare_kernel(const __grid_constant_
     for (int i = threadIdx.x; i < keys; i += blockDim.x) {
         p.oq[t * keys + i] = load_f(q + i) * scale;
         p.ok[t * keys + i] = load_f(k + i);
-        p.og[t * keys + i] = gla_decay(p.z[t * keys + i] + ld_bf16(p.z_bias + i), inv_tau);
+        p.og[t * keys + i] = gla_decay_less_one(p.z[t * keys + i] + ld_bf16(p.z_bias + i), inv_tau);
     }
     for (int i = threadIdx.x; i < values; i += blockDim.x) p.ov[t * values + i] = load_f(v + i);
 }
@@ -120,7 +122,7 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constan
     for (int c = threadIdx.x; c < values; c += 256)
         p.ov[(size_t)t * values + c] = silu_precise(conv_at(v + c, p.ld, t, position, p.v_taps + (size_t)c * p.conv.taps, p.conv, 2 * kv_keys + c));
     for (int c = threadIdx.x; c < keys; c += 256)
-        p.og[(size_t)t * keys + c] = delta_decay(p.z[(size_t)t * keys + c] + ld_bf16(p.z_bias + c), ld_bf16(p.a_log + c / p.dim));
+        p.og[(size_t)t * keys + c] = delta_decay_less_one(p.z[(size_t)t * keys + c] + ld_bf16(p.z_bias + c), ld_bf16(p.a_log + c / p.dim));
     const T* beta = reinterpret_cast<const T*>(p.beta) + (size_t)t * p.ld;
     for (int h = threadIdx.x; h < p.heads; h += 256) p.obeta[(size_t)t * p.heads + h] = sigmoid_precise(load_f(beta + h));
 }
@@ -141,7 +143,6 @@ conv_history_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* _
 
 // -------------------------------------------------------------------------------- recurrence
 typedef unsigned long long u64;
-QD_DEVINL u64 mul2(u64 a, u64 b) { u64 d; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
 QD_DEVINL u64 fma2(u64 a, u64 b, u64 c) { u64 d; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c)); return d; }
 QD_DEVINL u64 pack2(float lo, float hi) { return (u64)__float_as_uint(lo) | ((u64)__float_as_uint(hi) << 32); }
 QD_DEVINL float lo2(u64 v) { return __uint_as_float((uint32_t)v); }
@@ -259,8 +260,8 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
                 for (int j = 0; j < J; ++j)
 #pragma unroll
                     for (int c = 0; c < 2; ++c) {
-                        s[j][0][c] = mul2(s[j][0][c], g[j].x);
-                        s[j][1][c] = mul2(s[j][1][c], g[j].y);
+                        s[j][0][c] = fma2(s[j][0][c], g[j].x, s[j][0][c]);
+                        s[j][1][c] = fma2(s[j][1][c], g[j].y, s[j][1][c]);
                         pr[c] = fma2(s[j][0][c], k[j].x, pr[c]);
                         o[c] = fma2(s[j][0][c], q[j].x, o[c]);
                         pr[c] = fma2(s[j][1][c], k[j].y, pr[c]);
@@ -301,8 +302,8 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
                 for (int j = 0; j < J; ++j)
 #pragma unroll
                     for (int c = 0; c < 2; ++c) {
-                        s[j][0][c] = fma2(s[j][0][c], g[j].x, mul2(k[j].x, vv[c]));
-                        s[j][1][c] = fma2(s[j][1][c], g[j].y, mul2(k[j].y, vv[c]));
+                        s[j][0][c] = fma2(k[j].x, vv[c], fma2(s[j][0][c], g[j].x, s[j][0][c]));
+                        s[j][1][c] = fma2(k[j].y, vv[c], fma2(s[j][1][c], g[j].y, s[j][1][c]));
                         o[c] = fma2(s[j][0][c], q[j].x, o[c]);
                         o[c] = fma2(s[j][1][c], q[j].y, o[c]);
                     }
@@ -470,7 +471,7 @@ __global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const __g
     for (int d = group; d < ((dim + 31) & ~31); d += 32) {
         const int row = head * dim + min(d, dim - 1);
         const float z = low_rank_dot(p.up + (size_t)row * p.rank, low, p.rank, sub) + ld_bf16(p.up_bias + row);
-        if (sub == 0 && d < dim) sg[d] = DELTA ? delta_decay(z, ld_bf16(p.a_log + head)) : gla_decay(z, 1.0f / p.tau);
+        if (sub == 0 && d < dim) sg[d] = DELTA ? delta_decay_less_one(z, ld_bf16(p.a_log + head)) : gla_decay_less_one(z, 1.0f / p.tau);
     }
     {
         const int c = head * vdim + min(c0 + group, vdim - 1);
@@ -484,7 +485,7 @@ __global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const __g
     for (int j = 0; j < KPT; ++j) {
         const int r = j * kStepGroups + kg;
         if (r < dim) {
-            s[j] *= sg[r];
+            s[j] = fmaf(s[j], sg[r], s[j]);
             if (DELTA) pred = fmaf(s[j], sk[r], pred);
         }
     }
