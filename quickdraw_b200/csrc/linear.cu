@@ -4,8 +4,8 @@
 //   linear_umma_kernel  many token rows, bf16 x: tcgen05.mma kind::f16, both operands by tiled TMA
 //                       (128-byte swizzle), accumulators in tensor memory.  Tensor-bound.
 //   linear_rows_kernel  up to eight token rows: a warp streams whole weight rows (16-byte loads, the
-//                       first 1024 inputs of each row requested before the wait for the preceding
-//                       kernel), the token rows in shared memory as fp32.  HBM-bound.
+//                       first inputs of each row - up to 4096 - requested before the wait for the
+//                       preceding kernel), the token rows in shared memory as fp32.  HBM-bound.
 //   linear_tile_kernel  any shape and alignment, and fp32 x with many rows: 64 x 64 tiles on the FMA pipe.
 #include <cuda.h>
 
@@ -15,12 +15,15 @@ namespace qd {
 namespace {
 
 // ------------------------------------------------------------------------------ few token rows
-constexpr int kRowsChunk = 1024;              // inputs staged at a time: four 16-byte pieces per lane and weight row
+// Inputs staged at a time: sixteen 16-byte pieces of weights per lane while one or two token rows leave the registers
+// and the shared memory for it.
+constexpr int rows_chunk(int R, int NR) { return (R <= 2 ? 4096 : (R == 4 ? 2048 : 1024)) / NR; }
 
 template <typename TX, typename TY, int R, int NR>
 __global__ void __launch_bounds__(256)
 linear_rows_kernel(const TX* __restrict__ x, long long ldx, const bf16* __restrict__ w, TY* __restrict__ y,
                    long long ldy, int tokens, int rows, int width, int gelu_cols) {
+    constexpr int kRowsChunk = rows_chunk(R, NR);
     __shared__ __align__(16) float xs[R][kRowsChunk];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int n0 = (blockIdx.x * 8 + warp) * NR;

@@ -5,11 +5,10 @@
 //
 // Prompt chunks: a prepare kernel (all tokens in parallel: short convolution, SiLU, unit norms, decays)
 // writes q, k, decay, v, beta as fp32 rows; linear_recurrence_kernel walks the tokens with the state in
-// registers.  A warp owns eight value columns; lane = (key group kl of eight, column pair cl): rows
-// 32 j + 4 kl + {0..3}, two columns, held as row pairs for the packed fp32 FMA.  Both read-outs of the
-// delta rule use the decayed state before the write, o = (gS)^T q + (k . q) u, so that one round of
-// shuffles carries both and the write is off the critical path.  Latency-bound: one warp per scheduler,
-// a dependent chain per token.
+// registers.  A warp owns eight value columns; a lane a group of key rows and a few columns, held as row
+// pairs for the packed fp32 FMA.  Both read-outs of the delta rule use the decayed state before the
+// write, o = (gS)^T q + (k . q) u, so that the second one hides in the first one's shuffles.
+// Latency-bound: one warp per scheduler, a dependent chain per token.
 // Decode: recurrence_step_kernel does everything between the projections and the output projection in
 // one launch: low-rank decay (and output gate), convolution, unit norms, recurrence, per-head RMS norm,
 // gate.  A cluster of blocks shares a head (32 value columns each) and adds its sums of squares over
@@ -29,7 +28,7 @@ QD_DEVINL float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf
 // Decays are carried as decay - 1, S + S (decay - 1) in one FMA: a slow channel's decay is so close to one
 // that its own rounding, the same at every token, would add up over a long sequence.
 QD_DEVINL float gla_decay_less_one(float z, float inv_tau) { return expm1f(log_sigmoid(z) * inv_tau); }
-QD_DEVINL float delta_decay_less_one(float z, float a_log) { return expm1f(-expf(a_log) * softplus_precise(z)); }
+QD_DEVINL float delta_decay_less_one(float z, float rate) { return expm1f(-rate * softplus_precise(z)); }      // rate = exp(A_log)
 
 // Convolution input history: ring of `taps` rows, position p in row p mod taps.  A step reads the rows of
 // the taps - 1 positions before it and writes its own, which is none of those.
@@ -61,7 +60,7 @@ struct PrepareParams {
     float tau;
     const int* position_ptr; int position;
     float* oq; float* ok; float* og; float* ov; float* obeta; float* okq;
-    int heads, kv_heads, dim, vdim;
+    int tokens, heads, kv_heads, dim, vdim;
 };
 
 template <typename T>
@@ -82,49 +81,132 @@ __global__ void __launch_bounds__(256) gla_prepare_kernel(const __grid_constant_
 }
 
 constexpr int kMaxPerLane = 8;       // key channels per lane: dim <= 256
+constexpr int kPrepareTokens = 8;    // tokens a block walks with the convolution's window in registers
 
-template <typename T>
+// The window of one channel: `back` of token t is the input of the position `back` before it.
+// TAPS == 0: any number, every input read again for every token.
+template <typename T, int TAPS> struct ConvWindow {
+    float w[TAPS ? TAPS : 1], x[TAPS ? TAPS : 1];
+    // before the first of the block's tokens, t: loads the taps and the inputs of t - TAPS + 1 .. t - 1
+    QD_DEVINL void open(const T* row0, long long ld, int t, int position, const bf16* taps, const ConvSource& src, int channel) {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j] = ld_bf16(taps + j);
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j) {
+            const int back = TAPS - j, at = t - back, p = position - back;      // becomes x[j - 1] when t's input arrives
+            x[j] = at >= 0 ? load_f(row0 + (long long)at * ld)
+                           : (p >= 0 ? load_f(reinterpret_cast<const T*>(src.history) + (size_t)(p % src.taps) * src.channels + channel) : 0.f);
+        }
+    }
+    QD_DEVINL float next(const T* row0, long long ld, int t, int position, const bf16* taps, const ConvSource& src, int channel) {
+        if (TAPS == 0) return conv_at(row0 + (long long)t * ld, ld, t, position, taps, src, channel);
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j) x[j - 1] = x[j];
+        x[TAPS ? TAPS - 1 : 0] = load_f(row0 + (long long)t * ld);
+        float acc = 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) acc = fmaf(x[j], w[j], acc);
+        return acc;
+    }
+};
+
+// blockIdx.y: groups of eight key/value heads (a warp each), then groups of 256 value channels, then
+// groups of 256 decay channels (the first of these also the step sizes).
+template <typename T, int TAPS>
 __global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constant__ PrepareParams p) {
     chain_enter();
-    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int position = (p.position_ptr ? *p.position_ptr : p.position) + t;
+    const int t0 = blockIdx.x * kPrepareTokens, t1 = min(t0 + kPrepareTokens, p.tokens), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int base = p.position_ptr ? *p.position_ptr : p.position;
     const int keys = p.heads * p.dim, values = p.heads * p.vdim, kv_keys = p.kv_heads * p.dim;
-    const T* q = reinterpret_cast<const T*>(p.q);
-    const T* k = reinterpret_cast<const T*>(p.k);
-    const T* v = reinterpret_cast<const T*>(p.v);
-    const float scale = 1.0f / sqrtf((float)p.dim);
-    for (int h = warp; h < p.kv_heads; h += 8) {
-        float qv[kMaxPerLane], kv[kMaxPerLane], qq = 0.f, kk = 0.f, kq = 0.f;
+    const int head_groups = (p.kv_heads + 7) / 8, value_groups = (values + 255) / 256;
+    int group = blockIdx.y;
+    if (group < head_groups) {
+        const T* q = reinterpret_cast<const T*>(p.q);
+        const T* k = reinterpret_cast<const T*>(p.k);
+        const float scale = 1.0f / sqrtf((float)p.dim);
+        const int h = group * 8 + warp;
+        if (h >= p.kv_heads) return;
+        ConvWindow<T, TAPS> wq[kMaxPerLane / 2], wk[kMaxPerLane / 2];
+        const bool windows = p.dim <= 32 * (kMaxPerLane / 2);      // wider heads read their inputs again
+        if (windows)
 #pragma unroll
-        for (int i = 0; i < kMaxPerLane; ++i) {
-            const int d = i * 32 + lane, c = h * p.dim + d;
-            qv[i] = kv[i] = 0.f;
-            if (d < p.dim) {
-                qv[i] = silu_precise(conv_at(q + c, p.ld, t, position, p.q_taps + (size_t)c * p.conv.taps, p.conv, c));
-                kv[i] = silu_precise(conv_at(k + c, p.ld, t, position, p.k_taps + (size_t)c * p.conv.taps, p.conv, kv_keys + c));
+            for (int i = 0; i < kMaxPerLane / 2; ++i) {
+                const int d = i * 32 + lane, c = h * p.dim + d;
+                if (d < p.dim) {
+                    wq[i].open(q + c, p.ld, t0, base + t0, p.q_taps + (size_t)c * p.conv.taps, p.conv, c);
+                    wk[i].open(k + c, p.ld, t0, base + t0, p.k_taps + (size_t)c * p.conv.taps, p.conv, kv_keys + c);
+                }
             }
-            qq = fmaf(qv[i], qv[i], qq);
-            kk = fmaf(kv[i], kv[i], kk);
-            kq = fmaf(qv[i], kv[i], kq);
-        }
-        qq = warp_sum(qq); kk = warp_sum(kk); kq = warp_sum(kq);
-        const float qs = scale / sqrtf(qq + kUnitEps), ks = 1.0f / sqrtf(kk + kUnitEps);
+        for (int t = t0; t < t1; ++t) {
+            float qv[kMaxPerLane], kv[kMaxPerLane], qq = 0.f, kk = 0.f, kq = 0.f;
 #pragma unroll
-        for (int i = 0; i < kMaxPerLane; ++i) {
-            const int d = i * 32 + lane;
-            if (d < p.dim) {
-                p.oq[(size_t)t * kv_keys + h * p.dim + d] = qv[i] * qs;
-                p.ok[(size_t)t * kv_keys + h * p.dim + d] = kv[i] * ks;
+            for (int i = 0; i < kMaxPerLane; ++i) {
+                const int d = i * 32 + lane, c = h * p.dim + d;
+                qv[i] = kv[i] = 0.f;
+                if (d < p.dim) {
+                    const bf16* qt = p.q_taps + (size_t)c * p.conv.taps;
+                    const bf16* kt = p.k_taps + (size_t)c * p.conv.taps;
+                    if (windows && i < kMaxPerLane / 2) {
+                        qv[i] = wq[i % (kMaxPerLane / 2)].next(q + c, p.ld, t, base + t, qt, p.conv, c);
+                        kv[i] = wk[i % (kMaxPerLane / 2)].next(k + c, p.ld, t, base + t, kt, p.conv, kv_keys + c);
+                    } else {
+                        qv[i] = conv_at(q + c + (long long)t * p.ld, p.ld, t, base + t, qt, p.conv, c);
+                        kv[i] = conv_at(k + c + (long long)t * p.ld, p.ld, t, base + t, kt, p.conv, kv_keys + c);
+                    }
+                    qv[i] = silu_precise(qv[i]);
+                    kv[i] = silu_precise(kv[i]);
+                }
+                qq = fmaf(qv[i], qv[i], qq);
+                kk = fmaf(kv[i], kv[i], kk);
+                kq = fmaf(qv[i], kv[i], kq);
             }
+            qq = warp_sum(qq); kk = warp_sum(kk); kq = warp_sum(kq);
+            const float qs = scale / sqrtf(qq + kUnitEps), ks = 1.0f / sqrtf(kk + kUnitEps);
+            const size_t at = (size_t)t * kv_keys + h * p.dim;
+#pragma unroll
+            for (int i = 0; i < kMaxPerLane; ++i) {
+                const int d = i * 32 + lane;
+                if (d < p.dim) { p.oq[at + d] = qv[i] * qs; p.ok[at + d] = kv[i] * ks; }
+            }
+            if (lane == 0) p.okq[(size_t)t * p.kv_heads + h] = kq * qs * ks;
         }
-        if (lane == 0) p.okq[(size_t)t * p.kv_heads + h] = kq * qs * ks;
+        return;
     }
-    for (int c = threadIdx.x; c < values; c += 256)
-        p.ov[(size_t)t * values + c] = silu_precise(conv_at(v + c, p.ld, t, position, p.v_taps + (size_t)c * p.conv.taps, p.conv, 2 * kv_keys + c));
-    for (int c = threadIdx.x; c < keys; c += 256)
-        p.og[(size_t)t * keys + c] = delta_decay_less_one(p.z[(size_t)t * keys + c] + ld_bf16(p.z_bias + c), ld_bf16(p.a_log + c / p.dim));
-    const T* beta = reinterpret_cast<const T*>(p.beta) + (size_t)t * p.ld;
-    for (int h = threadIdx.x; h < p.heads; h += 256) p.obeta[(size_t)t * p.heads + h] = sigmoid_precise(load_f(beta + h));
+    group -= head_groups;
+    if (group < value_groups) {
+        const int c = group * 256 + threadIdx.x, channel = 2 * kv_keys + c;
+        if (c >= values) return;
+        const T* v = reinterpret_cast<const T*>(p.v) + c;
+        const bf16* taps = p.v_taps + (size_t)c * p.conv.taps;
+        ConvWindow<T, TAPS> w;
+        w.open(v, p.ld, t0, base + t0, taps, p.conv, channel);
+        for (int t = t0; t < t1; ++t) p.ov[(size_t)t * values + c] = silu_precise(w.next(v, p.ld, t, base + t, taps, p.conv, channel));
+        return;
+    }
+    group -= value_groups;
+    const int c = group * 256 + threadIdx.x;
+    if (c < keys) {
+        const float bias = ld_bf16(p.z_bias + c), rate = expf(ld_bf16(p.a_log + c / p.dim));
+#pragma unroll 4
+        for (int t = t0; t < t1; ++t) p.og[(size_t)t * keys + c] = delta_decay_less_one(p.z[(size_t)t * keys + c] + bias, rate);
+    }
+    if (group == 0)
+        for (int i = threadIdx.x; i < (t1 - t0) * p.heads; i += 256) {
+            const int t = t0 + i / p.heads, h = i % p.heads;
+            p.obeta[(size_t)t * p.heads + h] = sigmoid_precise(load_f(reinterpret_cast<const T*>(p.beta) + (long long)t * p.ld + h));
+        }
+}
+
+template <typename T>
+int launch_delta_prepare(const PrepareParams& p, cudaStream_t s) {
+    const int groups = (p.kv_heads + 7) / 8 + (p.heads * p.vdim + 255) / 256 + (p.heads * p.dim + 255) / 256;
+    const dim3 grid((p.tokens + kPrepareTokens - 1) / kPrepareTokens, groups);
+    switch (p.conv.taps) {
+        case 2: return qd_launch(delta_prepare_kernel<T, 2>, grid, dim3(256), 0, s, 1, p);
+        case 3: return qd_launch(delta_prepare_kernel<T, 3>, grid, dim3(256), 0, s, 1, p);
+        case 4: return qd_launch(delta_prepare_kernel<T, 4>, grid, dim3(256), 0, s, 1, p);
+        default: return qd_launch(delta_prepare_kernel<T, 0>, grid, dim3(256), 0, s, 1, p);
+    }
 }
 
 // The chunk's last `taps` inputs into the history ring.
@@ -165,60 +247,81 @@ struct RecurrenceParams {
     int tokens, heads, kv_heads, dim, vdim, vectors;
 };
 
-// floats of one staged token: q, k, decay (padded to 32 J), v columns, beta, k . q (padded to 4)
-template <int J> constexpr int rec_token_floats() { return 3 * 32 * J + kRecCols + 4; }
+// floats of one staged token: q, k, decay - 1 (padded to `row`), v columns, beta, k . q (padded to 4)
+constexpr int rec_token_floats(int row) { return 3 * row + kRecCols + 4; }
 
-template <int J, bool DELTA>
+// A token's vectors, this lane's rows.
+template <int J> struct RecVectors { ulonglong2 q[J], k[J], g[J]; };
+
+// Sums over the KL lanes of a key group; every lane ends up with the sum of ONE of its CC columns (the
+// column index is returned), so that a round moves half of what the round before it did.
+template <int KL, int CC>
+QD_DEVINL int reduce_columns(const float (&v)[CC], int kl, float& total) {
+    if (CC == 2) {
+        const bool odd = kl & 1;
+        total = (odd ? v[1] : v[0]) + __shfl_xor_sync(0xffffffffu, odd ? v[0] : v[1], 1);
+#pragma unroll
+        for (int x = 2; x < KL; x <<= 1) total += __shfl_xor_sync(0xffffffffu, total, x);
+        return kl & 1;
+    }
+    const bool upper = kl & 1, odd = kl & 2;
+    float a = upper ? v[CC - 2] : v[0], b = upper ? v[CC - 1] : v[1];
+    a += __shfl_xor_sync(0xffffffffu, upper ? v[0] : v[CC - 2], 1);
+    b += __shfl_xor_sync(0xffffffffu, upper ? v[1] : v[CC - 1], 1);
+    total = (odd ? b : a) + __shfl_xor_sync(0xffffffffu, odd ? a : b, 2);
+#pragma unroll
+    for (int x = 4; x < KL; x <<= 1) total += __shfl_xor_sync(0xffffffffu, total, x);
+    return (upper ? 2 : 0) + (odd ? 1 : 0);
+}
+
+// KL lanes share a column's keys (rows 4 KL j + 4 kl + {0..3}), a lane holds CC = KL / 4 columns: more
+// columns per lane mean fewer shared-memory reads per state element, fewer lanes per column fewer rounds
+// of shuffles in the delta rule's dependent chain.
+template <int KL, int J, bool DELTA>
 __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __grid_constant__ RecurrenceParams p) {
     chain_enter();
     extern __shared__ __align__(16) float tiles[];
-    constexpr int kToken = rec_token_floats<J>(), kRow = 32 * J;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, kl = lane & 7, cl = lane >> 3;
+    constexpr int CC = KL / 4, kRow = 4 * KL * J, kToken = rec_token_floats(kRow);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, kl = lane % KL, cl = lane / KL;
     const int head = blockIdx.x, kv = head / (p.heads / p.kv_heads), c0 = blockIdx.y * kRecCols;
-    const int col = c0 + warp * 8 + cl * 2;
+    const int local = warp * 8 + cl * CC, col = c0 + local;
     const int dim = p.dim, vdim = p.vdim;
     float* state = p.state + (size_t)head * dim * vdim;
 
     for (int i = tid; i < 2 * kRecTile * kToken; i += kRecThreads) tiles[i] = 0.f;      // padding rows stay zero
-    u64 s[J][2][2];
+    u64 s[J][2][CC];
 #pragma unroll
     for (int j = 0; j < J; ++j)
 #pragma unroll
         for (int h = 0; h < 2; ++h)
 #pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                const int r = j * 32 + kl * 4 + h * 2;
+            for (int c = 0; c < CC; ++c) {
+                const int r = j * 4 * KL + kl * 4 + h * 2;
                 const bool ok = col + c < vdim;
                 s[j][h][c] = pack2(ok && r < dim ? state[(size_t)r * vdim + col + c] : 0.f,
                                    ok && r + 1 < dim ? state[(size_t)(r + 1) * vdim + col + c] : 0.f);
             }
     __syncthreads();
 
-    const int cols = min(kRecCols, vdim - c0);
+    // a thread copies the same piece of every token of a tile
+    const int cols = min(kRecCols, vdim - c0), unit = p.vectors ? 4 : 1;
+    const int kp = dim / unit, per = 3 * kp + cols / unit;
     auto stage = [&](int tile) {
-        float* base = tiles + (tile & 1) * kRecTile * kToken;
         const int t0 = tile * kRecTile, count = min(kRecTile, p.tokens - t0);
-        if (p.vectors) {
-            const int kp = dim / 4, vp = cols / 4, per = 3 * kp + vp;
-            for (int i = tid; i < count * per; i += kRecThreads) {
-                const int tt = i / per, piece = i % per;
-                const size_t t = t0 + tt;
-                float* dst = base + tt * kToken;
-                if (piece < kp) copy16(dst + piece * 4, p.q + (t * p.kv_heads + kv) * dim + piece * 4);
-                else if (piece < 2 * kp) copy16(dst + kRow + (piece - kp) * 4, p.k + (t * p.kv_heads + kv) * dim + (piece - kp) * 4);
-                else if (piece < 3 * kp) copy16(dst + 2 * kRow + (piece - 2 * kp) * 4, p.g + (t * p.heads + head) * dim + (piece - 2 * kp) * 4);
-                else copy16(dst + 3 * kRow + (piece - 3 * kp) * 4, p.v + (t * p.heads + head) * vdim + c0 + (piece - 3 * kp) * 4);
-            }
-        } else {
-            const int per = 3 * dim + cols;
-            for (int i = tid; i < count * per; i += kRecThreads) {
-                const int tt = i / per, e = i % per;
-                const size_t t = t0 + tt;
-                float* dst = base + tt * kToken;
-                if (e < dim) copy4(dst + e, p.q + (t * p.kv_heads + kv) * dim + e);
-                else if (e < 2 * dim) copy4(dst + kRow + e - dim, p.k + (t * p.kv_heads + kv) * dim + e - dim);
-                else if (e < 3 * dim) copy4(dst + 2 * kRow + e - 2 * dim, p.g + (t * p.heads + head) * dim + e - 2 * dim);
-                else copy4(dst + 3 * kRow + e - 3 * dim, p.v + (t * p.heads + head) * vdim + c0 + e - 3 * dim);
+        float* base = tiles + (tile & 1) * kRecTile * kToken;
+        for (int piece = tid; piece < per; piece += kRecThreads) {
+            const int which = piece / kp, e = (which < 3 ? piece - which * kp : piece - 3 * kp) * unit;
+            const float* src;
+            float* dst = base + (which < 3 ? which : 3) * kRow + e;
+            size_t stride;
+            if (which < 2) { stride = (size_t)p.kv_heads * dim; src = (which ? p.k : p.q) + t0 * stride + (size_t)kv * dim + e; }
+            else if (which == 2) { stride = (size_t)p.heads * dim; src = p.g + t0 * stride + (size_t)head * dim + e; }
+            else { stride = (size_t)p.heads * vdim; src = p.v + t0 * stride + (size_t)head * vdim + c0 + e; }
+            if (p.vectors) {
+#pragma unroll 4
+                for (int tt = 0; tt < count; ++tt, src += stride, dst += kToken) copy16(dst, src);
+            } else {
+                for (int tt = 0; tt < count; ++tt, src += stride, dst += kToken) copy4(dst, src);
             }
         }
         if (DELTA && tid < count) {
@@ -228,103 +331,107 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
         }
         copies_commit();
     };
+    auto fetch = [&](const float* token, RecVectors<J>& f) {
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+            f.g[j] = *reinterpret_cast<const ulonglong2*>(token + 2 * kRow + j * 4 * KL + kl * 4);
+            f.k[j] = *reinterpret_cast<const ulonglong2*>(token + kRow + j * 4 * KL + kl * 4);
+            f.q[j] = *reinterpret_cast<const ulonglong2*>(token + j * 4 * KL + kl * 4);
+        }
+    };
+    float* out = p.out + (size_t)head * vdim;
+    const size_t out_stride = (size_t)p.heads * vdim;
+    auto advance = [&](const RecVectors<J>& f, const float* token) {
+        float v[CC], o[CC], u[CC];
+#pragma unroll
+        for (int c = 0; c < CC; ++c) v[c] = token[3 * kRow + local + c];
+        u64 oa[CC], ob[CC];
+#pragma unroll
+        for (int c = 0; c < CC; ++c) oa[c] = ob[c] = 0ull;
+        float kq = 0.f;
+        if (DELTA) {
+            const float2 bk = *reinterpret_cast<const float2*>(token + 3 * kRow + kRecCols);      // beta, k . q
+            kq = bk.y;
+            u64 pa[CC], pb[CC];
+            float pred[CC];
+#pragma unroll
+            for (int c = 0; c < CC; ++c) pa[c] = pb[c] = 0ull;
+#pragma unroll
+            for (int j = 0; j < J; ++j)
+#pragma unroll
+                for (int c = 0; c < CC; ++c) {
+                    s[j][0][c] = fma2(s[j][0][c], f.g[j].x, s[j][0][c]);
+                    s[j][1][c] = fma2(s[j][1][c], f.g[j].y, s[j][1][c]);
+                    pa[c] = fma2(s[j][0][c], f.k[j].x, pa[c]);
+                    pb[c] = fma2(s[j][1][c], f.k[j].y, pb[c]);
+                }
+#pragma unroll
+            for (int c = 0; c < CC; ++c) pred[c] = (lo2(pa[c]) + hi2(pa[c])) + (lo2(pb[c]) + hi2(pb[c]));
+#pragma unroll
+            for (int x = 1; x < KL; x <<= 1)
+#pragma unroll
+                for (int c = 0; c < CC; ++c) pred[c] += __shfl_xor_sync(0xffffffffu, pred[c], x);
+#pragma unroll
+            for (int j = 0; j < J; ++j)               // fills the shuffles' latency
+#pragma unroll
+                for (int c = 0; c < CC; ++c) {
+                    oa[c] = fma2(s[j][0][c], f.q[j].x, oa[c]);
+                    ob[c] = fma2(s[j][1][c], f.q[j].y, ob[c]);
+                }
+#pragma unroll
+            for (int c = 0; c < CC; ++c) u[c] = bk.x * (v[c] - pred[c]);
+#pragma unroll
+            for (int j = 0; j < J; ++j)
+#pragma unroll
+                for (int c = 0; c < CC; ++c) {
+                    const u64 uu = pack2(u[c], u[c]);
+                    s[j][0][c] = fma2(f.k[j].x, uu, s[j][0][c]);
+                    s[j][1][c] = fma2(f.k[j].y, uu, s[j][1][c]);
+                }
+        } else {
+#pragma unroll
+            for (int c = 0; c < CC; ++c) {
+                const u64 vv = pack2(v[c], v[c]);
+#pragma unroll
+                for (int j = 0; j < J; ++j) {
+                    s[j][0][c] = fma2(f.k[j].x, vv, fma2(s[j][0][c], f.g[j].x, s[j][0][c]));
+                    s[j][1][c] = fma2(f.k[j].y, vv, fma2(s[j][1][c], f.g[j].y, s[j][1][c]));
+                    oa[c] = fma2(s[j][0][c], f.q[j].x, oa[c]);
+                    ob[c] = fma2(s[j][1][c], f.q[j].y, ob[c]);
+                }
+            }
+        }
+#pragma unroll
+        for (int c = 0; c < CC; ++c) o[c] = (lo2(oa[c]) + hi2(oa[c])) + (lo2(ob[c]) + hi2(ob[c]));
+        float total;
+        const int mine = reduce_columns<KL, CC>(o, kl, total);
+        if (DELTA) {
+            float um = u[0];
+#pragma unroll
+            for (int c = 1; c < CC; ++c) um = mine == c ? u[c] : um;
+            total = fmaf(um, kq, total);
+        }
+        if (kl < CC && col + mine < vdim) out[col + mine] = total;
+        out += out_stride;
+    };
 
     const int ntiles = (p.tokens + kRecTile - 1) / kRecTile;
     stage(0);
     for (int tile = 0; tile < ntiles; ++tile) {
         if (tile + 1 < ntiles) { stage(tile + 1); copies_wait<1>(); } else { copies_wait<0>(); }
         __syncthreads();
-        const float* base = tiles + (tile & 1) * kRecTile * kToken;
-        const int t0 = tile * kRecTile, count = min(kRecTile, p.tokens - t0);
-        ulonglong2 q[J], k[J], g[J];
-        auto fetch = [&](const float* token, ulonglong2 (&fq)[J], ulonglong2 (&fk)[J], ulonglong2 (&fg)[J]) {
-#pragma unroll
-            for (int j = 0; j < J; ++j) {
-                fg[j] = *reinterpret_cast<const ulonglong2*>(token + 2 * kRow + j * 32 + kl * 4);
-                fk[j] = *reinterpret_cast<const ulonglong2*>(token + kRow + j * 32 + kl * 4);
-                fq[j] = *reinterpret_cast<const ulonglong2*>(token + j * 32 + kl * 4);
-            }
-        };
-        constexpr bool kAhead = J <= 4;             // the next token's vectors in registers while this one is reduced
-        fetch(base, q, k, g);
-        for (int tt = 0; tt < count; ++tt) {
-            const float* token = base + tt * kToken;
-            if (!kAhead && tt) fetch(token, q, k, g);
-            const float2 v = *reinterpret_cast<const float2*>(token + 3 * kRow + warp * 8 + cl * 2);
-            u64 o[2] = {0ull, 0ull};
-            float out[2];
-            if (DELTA) {
-                const float2 bk = *reinterpret_cast<const float2*>(token + 3 * kRow + kRecCols);      // beta, k . q
-                u64 pr[2] = {0ull, 0ull};
-#pragma unroll
-                for (int j = 0; j < J; ++j)
-#pragma unroll
-                    for (int c = 0; c < 2; ++c) {
-                        s[j][0][c] = fma2(s[j][0][c], g[j].x, s[j][0][c]);
-                        s[j][1][c] = fma2(s[j][1][c], g[j].y, s[j][1][c]);
-                        pr[c] = fma2(s[j][0][c], k[j].x, pr[c]);
-                        o[c] = fma2(s[j][0][c], q[j].x, o[c]);
-                        pr[c] = fma2(s[j][1][c], k[j].y, pr[c]);
-                        o[c] = fma2(s[j][1][c], q[j].y, o[c]);
-                    }
-                float pred[2] = {lo2(pr[0]) + hi2(pr[0]), lo2(pr[1]) + hi2(pr[1])};
-                out[0] = lo2(o[0]) + hi2(o[0]);
-                out[1] = lo2(o[1]) + hi2(o[1]);
-                ulonglong2 nq[J], nk[J], ng[J];
-                if (kAhead && tt + 1 < count) fetch(token + kToken, nq, nk, ng);
-#pragma unroll
-                for (int x = 1; x < 8; x <<= 1) {
-                    pred[0] += __shfl_xor_sync(0xffffffffu, pred[0], x);
-                    pred[1] += __shfl_xor_sync(0xffffffffu, pred[1], x);
-                    out[0] += __shfl_xor_sync(0xffffffffu, out[0], x);
-                    out[1] += __shfl_xor_sync(0xffffffffu, out[1], x);
-                }
-                const float u0 = bk.x * (v.x - pred[0]), u1 = bk.x * (v.y - pred[1]);
-                out[0] = fmaf(u0, bk.y, out[0]);
-                out[1] = fmaf(u1, bk.y, out[1]);
-                const u64 uu[2] = {pack2(u0, u0), pack2(u1, u1)};
-#pragma unroll
-                for (int j = 0; j < J; ++j)
-#pragma unroll
-                    for (int c = 0; c < 2; ++c) {
-                        s[j][0][c] = fma2(k[j].x, uu[c], s[j][0][c]);
-                        s[j][1][c] = fma2(k[j].y, uu[c], s[j][1][c]);
-                    }
-                if (kAhead) {
-#pragma unroll
-                    for (int j = 0; j < J; ++j) { q[j] = nq[j]; k[j] = nk[j]; g[j] = ng[j]; }
-                }
-            } else {
-                const u64 vv[2] = {pack2(v.x, v.x), pack2(v.y, v.y)};
-                ulonglong2 nq[J], nk[J], ng[J];
-                if (kAhead && tt + 1 < count) fetch(token + kToken, nq, nk, ng);
-#pragma unroll
-                for (int j = 0; j < J; ++j)
-#pragma unroll
-                    for (int c = 0; c < 2; ++c) {
-                        s[j][0][c] = fma2(k[j].x, vv[c], fma2(s[j][0][c], g[j].x, s[j][0][c]));
-                        s[j][1][c] = fma2(k[j].y, vv[c], fma2(s[j][1][c], g[j].y, s[j][1][c]));
-                        o[c] = fma2(s[j][0][c], q[j].x, o[c]);
-                        o[c] = fma2(s[j][1][c], q[j].y, o[c]);
-                    }
-                out[0] = lo2(o[0]) + hi2(o[0]);
-                out[1] = lo2(o[1]) + hi2(o[1]);
-#pragma unroll
-                for (int x = 1; x < 8; x <<= 1) {
-                    out[0] += __shfl_xor_sync(0xffffffffu, out[0], x);
-                    out[1] += __shfl_xor_sync(0xffffffffu, out[1], x);
-                }
-                if (kAhead) {
-#pragma unroll
-                    for (int j = 0; j < J; ++j) { q[j] = nq[j]; k[j] = nk[j]; g[j] = ng[j]; }
-                }
-            }
-            if (kl == 0) {
-                float* dst = p.out + ((size_t)(t0 + tt) * p.heads + head) * vdim + col;
-                if (col < vdim) dst[0] = out[0];
-                if (col + 1 < vdim) dst[1] = out[1];
-            }
+        const float* token = tiles + (tile & 1) * kRecTile * kToken;
+        const int count = min(kRecTile, p.tokens - tile * kRecTile);
+        RecVectors<J> even, odd;                     // the next token's vectors are read while this one is reduced
+        fetch(token, even);
+        int tt = 0;
+        for (; tt + 2 <= count; tt += 2, token += 2 * kToken) {
+            fetch(token + kToken, odd);
+            advance(even, token);
+            if (tt + 2 < count) fetch(token + 2 * kToken, even);
+            advance(odd, token + kToken);
         }
+        if (tt < count) advance(even, token);
         __syncthreads();                 // the buffer may be refilled
     }
 #pragma unroll
@@ -332,8 +439,8 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
 #pragma unroll
         for (int h = 0; h < 2; ++h)
 #pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                const int r = j * 32 + kl * 4 + h * 2;
+            for (int c = 0; c < CC; ++c) {
+                const int r = j * 4 * KL + kl * 4 + h * 2;
                 if (col + c < vdim) {
                     if (r < dim) state[(size_t)r * vdim + col + c] = lo2(s[j][h][c]);
                     if (r + 1 < dim) state[(size_t)(r + 1) * vdim + col + c] = hi2(s[j][h][c]);
@@ -341,24 +448,29 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
             }
 }
 
-template <int J, bool DELTA>
+template <int KL, int J, bool DELTA>
 int launch_recurrence(const RecurrenceParams& p, cudaStream_t stream) {
-    const size_t smem = 2ull * kRecTile * rec_token_floats<J>() * 4;
-    if (!allow_smem(linear_recurrence_kernel<J, DELTA>, smem)) return QD_ERR_LAUNCH;
-    return qd_launch(linear_recurrence_kernel<J, DELTA>, dim3(p.heads, (p.vdim + kRecCols - 1) / kRecCols), dim3(kRecThreads), smem,
+    const size_t smem = 2ull * kRecTile * rec_token_floats(4 * KL * J) * 4;
+    if (!allow_smem(linear_recurrence_kernel<KL, J, DELTA>, smem)) return QD_ERR_LAUNCH;
+    return qd_launch(linear_recurrence_kernel<KL, J, DELTA>, dim3(p.heads, (p.vdim + kRecCols - 1) / kRecCols), dim3(kRecThreads), smem,
                      stream, 1, p);
 }
 template <bool DELTA>
 int recurrence(const RecurrenceParams& p, cudaStream_t stream) {
-    switch ((p.dim + 31) / 32) {
-        case 1: return launch_recurrence<1, DELTA>(p, stream);
-        case 2: return launch_recurrence<2, DELTA>(p, stream);
-        case 3: return launch_recurrence<3, DELTA>(p, stream);
-        case 4: return launch_recurrence<4, DELTA>(p, stream);
-        case 5: case 6: return launch_recurrence<6, DELTA>(p, stream);
-        case 7: case 8: return launch_recurrence<8, DELTA>(p, stream);
-        default: return QD_ERR_UNSUPPORTED;
+    if (DELTA) {
+        if (p.dim <= 32) return launch_recurrence<8, 1, true>(p, stream);
+        if (p.dim <= 64) return launch_recurrence<8, 2, true>(p, stream);
+        if (p.dim <= 96) return launch_recurrence<8, 3, true>(p, stream);
+        if (p.dim <= 128) return launch_recurrence<8, 4, true>(p, stream);
+        if (p.dim <= 192) return launch_recurrence<16, 3, true>(p, stream);
+        if (p.dim <= 256) return launch_recurrence<16, 4, true>(p, stream);
+        return QD_ERR_UNSUPPORTED;
     }
+    if (p.dim <= 64) return launch_recurrence<16, 1, false>(p, stream);
+    if (p.dim <= 128) return launch_recurrence<16, 2, false>(p, stream);
+    if (p.dim <= 192) return launch_recurrence<16, 3, false>(p, stream);
+    if (p.dim <= 256) return launch_recurrence<16, 4, false>(p, stream);
+    return QD_ERR_UNSUPPORTED;
 }
 
 // ------------------------------------------------------------------------ per-head norm, gate
@@ -416,23 +528,28 @@ QD_DEVINL float low_rank_dot(const bf16* up, const float* low, int rank, int sub
     return group_sum<8>(acc);
 }
 
+// ask for `bytes` from p on (one 128-byte line per thread and round) to be in L2 soon
+QD_DEVINL void prefetch_span(const void* p, size_t bytes) {
+    for (size_t at = (size_t)threadIdx.x * 128; at < bytes; at += (size_t)blockDim.x * 128)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(p) + at));
+}
+
 template <typename T, bool DELTA, int KPT>
 __global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const __grid_constant__ StepParams p) {
-    chain_enter();
-    extern __shared__ float low[];                 // rank + gate_rank
-    __shared__ float sq[256], sk[256], sg[256], sv[32], sgate[32], part[kStepGroups][33], red[33], squares[8];
-    cg::cluster_group cluster = cg::this_cluster();
-    cluster.barrier_arrive();                      // waited for before the first access to another block's memory
     const int head = blockIdx.y, c0 = blockIdx.x * 32, tid = threadIdx.x, col = tid & 31, kg = tid >> 5;
     const int dim = p.dim, vdim = p.vdim, kv = head / (p.heads / p.kv_heads), kv_keys = p.kv_heads * dim;
+    grid_launch_dependents();
+    // the state tile (one line per key row) and the head's constant matrices are on their way while the kernel before this one ends
+    if (tid < dim) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.state + ((size_t)head * dim + tid) * vdim + c0));
+    prefetch_span(p.up + (size_t)head * dim * p.rank, (size_t)dim * p.rank * sizeof(bf16));
+    if (p.gate_up) prefetch_span(p.gate_up + ((size_t)head * vdim + c0) * p.gate_rank, (size_t)min(32, vdim - c0) * p.gate_rank * sizeof(bf16));
+    grid_dependency_wait();
+    extern __shared__ float low[];                 // rank + gate_rank
+    __shared__ float sq[256], sk[256], sg[256], sv[32], sgate[32], part[kStepGroups][33], norms[2][kStepGroups], squares[8];
+    cg::cluster_group cluster = cg::this_cluster();
+    cluster.barrier_arrive();                      // waited for before the first access to another block's memory
     const bool col_ok = c0 + col < vdim;
     float* tile = p.state + (size_t)head * dim * vdim + c0 + col;
-    float s[KPT];
-#pragma unroll
-    for (int j = 0; j < KPT; ++j) {
-        const int r = j * kStepGroups + kg;
-        s[j] = (r < dim && col_ok) ? tile[(size_t)r * vdim] : 0.f;
-    }
     const T* lowv = reinterpret_cast<const T*>(p.low);
     const T* gatev = reinterpret_cast<const T*>(p.gate_low);
     for (int i = tid; i < p.rank; i += kStepThreads) low[i] = load_f(lowv + i);
@@ -441,42 +558,57 @@ __global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const __g
     const T* k = reinterpret_cast<const T*>(p.k) + kv * dim;
     const T* v = reinterpret_cast<const T*>(p.v) + head * vdim + c0;
     const float scale = 1.0f / sqrtf((float)dim);
-    const int position = p.position_ptr ? *p.position_ptr : p.position;
-    float qv = 0.f, kvv = 0.f;
+    float qv = 0.f, kvv = 0.f, beta = 0.f, rate = 0.f;
     if (DELTA) {
+        const int position = p.position_ptr ? *p.position_ptr : p.position;
         const ConvSource src = {p.history, p.taps, 2 * kv_keys + p.heads * vdim};
         T* fresh = reinterpret_cast<T*>(p.history) + (size_t)(position % p.taps) * src.channels;
+        beta = sigmoid_precise(load_f(reinterpret_cast<const T*>(p.beta) + head));
+        rate = expf(ld_bf16(p.a_log + head));
         if (tid < dim) {
             const int c = kv * dim + tid;
             qv = silu_precise(conv_at(q + tid, 0, 0, position, p.q_taps + (size_t)c * p.taps, src, c));
             kvv = silu_precise(conv_at(k + tid, 0, 0, position, p.k_taps + (size_t)c * p.taps, src, kv_keys + c));
             if (blockIdx.x == 0 && head % (p.heads / p.kv_heads) == 0) { fresh[c] = q[tid]; fresh[kv_keys + c] = k[tid]; }
         }
-        if (tid < 32 && col_ok) {
-            const int c = head * vdim + c0 + tid;
-            sv[tid] = silu_precise(conv_at(v + tid, 0, 0, position, p.v_taps + (size_t)c * p.taps, src, 2 * kv_keys + c));
-            fresh[2 * kv_keys + c] = v[tid];
+        if (kg == kStepGroups - 1 && col_ok) {
+            const int c = head * vdim + c0 + col;
+            sv[col] = silu_precise(conv_at(v + col, 0, 0, position, p.v_taps + (size_t)c * p.taps, src, 2 * kv_keys + c));
+            fresh[2 * kv_keys + c] = v[col];
         }
-        const float qq = block_sum(qv * qv, red), kk = block_sum(kvv * kvv, red);
-        qv *= scale / sqrtf(qq + kUnitEps);
-        kvv *= 1.0f / sqrtf(kk + kUnitEps);
+        const float qq = warp_sum(qv * qv), kk = warp_sum(kvv * kvv);
+        if (col == 0) { norms[0][kg] = qq; norms[1][kg] = kk; }
     } else {
         if (tid < dim) { qv = load_f(q + tid) * scale; kvv = load_f(k + tid); }
-        if (tid < 32 && col_ok) sv[tid] = load_f(v + tid);
-        __syncthreads();
+        if (kg == kStepGroups - 1 && col_ok) sv[col] = load_f(v + col);
     }
-    if (tid < 256) { sq[tid] = qv; sk[tid] = kvv; }
+    sq[tid] = qv; sk[tid] = kvv;                   // not yet unit vectors in the delta rule: their factors join the sums below
+    float s[KPT];
+#pragma unroll
+    for (int j = 0; j < KPT; ++j) {
+        const int r = j * kStepGroups + kg;
+        s[j] = (r < dim && col_ok) ? tile[(size_t)r * vdim] : 0.f;
+    }
+    __syncthreads();
     // decay of the head's key channels, output gate of the block's columns: eight lanes per row
     const int sub = tid & 7, group = tid >> 3;
     for (int d = group; d < ((dim + 31) & ~31); d += 32) {
         const int row = head * dim + min(d, dim - 1);
         const float z = low_rank_dot(p.up + (size_t)row * p.rank, low, p.rank, sub) + ld_bf16(p.up_bias + row);
-        if (sub == 0 && d < dim) sg[d] = DELTA ? delta_decay_less_one(z, ld_bf16(p.a_log + head)) : gla_decay_less_one(z, 1.0f / p.tau);
+        if (sub == 0 && d < dim) sg[d] = DELTA ? delta_decay_less_one(z, rate) : gla_decay_less_one(z, 1.0f / p.tau);
     }
     {
         const int c = head * vdim + min(c0 + group, vdim - 1);
         const float gv = p.gate_up ? low_rank_dot(p.gate_up + (size_t)c * p.gate_rank, low + p.rank, p.gate_rank, sub) : load_f(gatev + c);
         if (sub == 0) sgate[group] = DELTA ? sigmoid_precise(gv) : silu_precise(gv);
+    }
+    float qs = 1.f, ks = 1.f;
+    if (DELTA) {
+        float qq = 0.f, kk = 0.f;
+#pragma unroll
+        for (int w = 0; w < kStepGroups; ++w) { qq += norms[0][w]; kk += norms[1][w]; }
+        qs = scale / sqrtf(qq + kUnitEps);
+        ks = 1.0f / sqrtf(kk + kUnitEps);
     }
     __syncthreads();
 
@@ -486,7 +618,7 @@ __global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const __g
         const int r = j * kStepGroups + kg;
         if (r < dim) {
             s[j] = fmaf(s[j], sg[r], s[j]);
-            if (DELTA) pred = fmaf(s[j], sk[r], pred);
+            if (DELTA) pred = fmaf(s[j], sk[r] * ks, pred);
         }
     }
     float u = col_ok ? sv[col] : 0.f;
@@ -496,7 +628,7 @@ __global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const __g
         float total = 0.f;
 #pragma unroll
         for (int w = 0; w < kStepGroups; ++w) total += part[w][col];
-        u = sigmoid_precise(load_f(reinterpret_cast<const T*>(p.beta) + head)) * (u - total);
+        u = beta * (u - total);
         __syncthreads();
     }
     float o = 0.f;
@@ -504,8 +636,8 @@ __global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const __g
     for (int j = 0; j < KPT; ++j) {
         const int r = j * kStepGroups + kg;
         if (r < dim) {
-            s[j] = fmaf(sk[r], u, s[j]);
-            o = fmaf(s[j], sq[r], o);
+            s[j] = fmaf(sk[r] * ks, u, s[j]);
+            o = fmaf(s[j], sq[r] * qs, o);
             if (col_ok) tile[(size_t)r * vdim] = s[j];
         }
     }
@@ -557,7 +689,7 @@ int step(const StepParams& p, cudaStream_t stream) {
 
 template <typename T, bool DELTA>
 int prepare(const PrepareParams& p, int tokens, cudaStream_t s) {
-    if (DELTA) return qd_launch(delta_prepare_kernel<T>, dim3(tokens), dim3(256), 0, s, 1, p);
+    if (DELTA) return launch_delta_prepare<T>(p, s);
     return qd_launch(gla_prepare_kernel<T>, dim3(tokens), dim3(256), 0, s, 1, p);
 }
 template <typename T>
@@ -583,7 +715,7 @@ extern "C" int qd_gla_prepare(const void* q, const void* k, const void* v, long 
     QD_CHECK_ARG(q && k && v && z && z_bias && oq && ok && og && ov && tokens > 0 && heads > 0 && dim > 0 && vdim > 0 && tau > 0.f);
     qd::PrepareParams p = {};
     p.q = q; p.k = k; p.v = v; p.ld = ld; p.z = z; p.z_bias = (const bf16*)z_bias; p.tau = tau;
-    p.oq = oq; p.ok = ok; p.og = og; p.ov = ov; p.heads = heads; p.kv_heads = heads; p.dim = dim; p.vdim = vdim;
+    p.oq = oq; p.ok = ok; p.og = og; p.ov = ov; p.tokens = tokens; p.heads = heads; p.kv_heads = heads; p.dim = dim; p.vdim = vdim;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == QD_BF16) return qd::prepare<bf16, false>(p, tokens, s);
     if (dtype == QD_F32) return qd::prepare<float, false>(p, tokens, s);
@@ -601,7 +733,7 @@ extern "C" int qd_channel_delta_prepare(const void* q, const void* k, const void
     const int kv_keys = kv_heads * dim, values = heads * vdim;
     qd::PrepareParams p = {q, k, v, ld, z, (const bf16*)z_bias, beta, (const bf16*)a_log, (const bf16*)q_taps, (const bf16*)k_taps,
                            (const bf16*)v_taps, {history, taps, 2 * kv_keys + values}, 1.f, position_ptr, position, oq, ok, og, ov,
-                           obeta, okq, heads, kv_heads, dim, vdim};
+                           obeta, okq, tokens, heads, kv_heads, dim, vdim};
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype != QD_BF16 && dtype != QD_F32) return QD_ERR_UNSUPPORTED;
     const int rc = dtype == QD_BF16 ? qd::prepare<bf16, true>(p, tokens, s) : qd::prepare<float, true>(p, tokens, s);

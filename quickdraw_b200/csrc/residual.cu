@@ -104,6 +104,102 @@ sublayer_close_kernel(const __grid_constant__ CloseParams p) {
     if (p.next_w) norm_out(row, width, p.eps, p.next_w, p.next_b, reinterpret_cast<T*>(p.normed) + at, red);
 }
 
+// The same for widths that split evenly: every thread keeps VPT groups of four consecutive elements in
+// registers, the sums over earlier results are formed before the first reduction, and mean and deviation
+// come out of ONE exchange: equal counts merge as mean = average of the means, M2 = sum of the M2 + count
+// times the squared distances of the means.
+QD_DEVINL void merged_moments(const float* v, int count, int width, float eps, float2* stats, float& mean, float& rstd) {
+    float m = 0.f, m2 = 0.f;
+    for (int i = 0; i < count; ++i) m += v[i];
+    m /= (float)count;
+    for (int i = 0; i < count; ++i) { const float d = v[i] - m; m2 = fmaf(d, d, m2); }
+    float n = (float)count;
+#pragma unroll
+    for (int x = 1; x < 32; x <<= 1) {
+        const float om = __shfl_xor_sync(0xffffffffu, m, x), o2 = __shfl_xor_sync(0xffffffffu, m2, x);
+        const float d = om - m;
+        m2 = m2 + o2 + d * d * (0.5f * n);
+        m = 0.5f * (m + om);
+        n *= 2.f;
+    }
+    const int warps = blockDim.x >> 5;
+    if ((threadIdx.x & 31) == 0) stats[threadIdx.x >> 5] = make_float2(m, m2);
+    __syncthreads();
+    float sum = 0.f, sq = 0.f;
+    for (int w = 0; w < warps; ++w) sum += stats[w].x;
+    mean = sum / (float)warps;
+    for (int w = 0; w < warps; ++w) { const float d = stats[w].x - mean; sq += stats[w].y + n * d * d; }
+    rstd = 1.0f / sqrtf(sq / (float)width + eps);
+}
+
+template <typename T, int VPT>
+__global__ void __launch_bounds__(kMaxThreads)
+sublayer_close_vec_kernel(const __grid_constant__ CloseParams p) {
+    chain_enter();
+    __shared__ float2 stats[2][kMaxThreads / 32];
+    const int width = p.width, threads = blockDim.x;
+    const size_t t = blockIdx.x, at = t * width;
+    const T* y = reinterpret_cast<const T*>(p.y) + at;
+    const T* gate = reinterpret_cast<const T*>(p.gate) + t * p.ld_gate;
+    float z[4 * VPT], x[4 * VPT], mix[4 * VPT];
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int i = (threadIdx.x + k * threads) * 4;
+        const float4 yv = load4(y + i), gv = load4(gate + i), bv = load4(p.gate_bias + i), xv = load4(p.x_in + at + i);
+        const float ya[4] = {yv.x, yv.y, yv.z, yv.w}, ga[4] = {gv.x + bv.x, gv.y + bv.y, gv.z + bv.z, gv.w + bv.w};
+        const float xa[4] = {xv.x, xv.y, xv.z, xv.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) { z[4 * k + e] = ya[e] * sigmoid_precise(ga[e]); x[4 * k + e] = xa[e]; mix[4 * k + e] = 0.f; }
+    }
+    for (int j0 = 0; j0 < p.older; j0 += 4) {
+        float4 r[4][VPT];
+        float c[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+            c[q] = j0 + q < p.older ? ld_bf16(p.depth + j0 + q) : 0.f;
+            const float* result = p.results + (size_t)min(j0 + q, p.older - 1) * p.result_stride + at;
+#pragma unroll
+            for (int k = 0; k < VPT; ++k) r[q][k] = load4(result + (threadIdx.x + k * threads) * 4);
+        }
+#pragma unroll
+        for (int q = 0; q < 4; ++q)
+#pragma unroll
+            for (int k = 0; k < VPT; ++k) {
+                mix[4 * k] = fmaf(r[q][k].x, c[q], mix[4 * k]); mix[4 * k + 1] = fmaf(r[q][k].y, c[q], mix[4 * k + 1]);
+                mix[4 * k + 2] = fmaf(r[q][k].z, c[q], mix[4 * k + 2]); mix[4 * k + 3] = fmaf(r[q][k].w, c[q], mix[4 * k + 3]);
+            }
+    }
+    float mean, rstd;
+    merged_moments(z, 4 * VPT, width, p.eps, stats[0], mean, rstd);
+    const float newest = p.older >= 0 ? ld_bf16(p.depth + p.older) : 1.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int i = (threadIdx.x + k * threads) * 4;
+        const float4 wv = load4(p.post_w + i), bv = load4(p.post_b + i);
+        const float wa[4] = {wv.x, wv.y, wv.z, wv.w}, ba[4] = {bv.x, bv.y, bv.z, bv.w};
+        float* v = z + 4 * k;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[e] = x[4 * k + e] + ((v[e] - mean) * rstd * wa[e] + ba[e]);
+        if (p.older >= 0) {
+            store4(p.results + (size_t)p.older * p.result_stride + at + i, make_float4(v[0], v[1], v[2], v[3]));
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[e] = fmaf(v[e], newest, mix[4 * k + e]);
+        }
+        store4(p.x_out + at + i, make_float4(v[0], v[1], v[2], v[3]));
+    }
+    if (!p.next_w) return;
+    merged_moments(z, 4 * VPT, width, p.eps, stats[1], mean, rstd);
+    T* normed = reinterpret_cast<T*>(p.normed) + at;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int i = (threadIdx.x + k * threads) * 4;
+        const float4 wv = load4(p.next_w + i), bv = load4(p.next_b + i);
+        const float* v = z + 4 * k;
+        store4(normed + i, make_float4((v[0] - mean) * rstd * wv.x + bv.x, (v[1] - mean) * rstd * wv.y + bv.y,
+                                       (v[2] - mean) * rstd * wv.z + bv.z, (v[3] - mean) * rstd * wv.w + bv.w));
+    }
+}
+
 int row_threads(int width) {
     int threads = (width / 4 + 31) / 32 * 32;
     return threads < 64 ? 64 : (threads > kMaxThreads ? kMaxThreads : threads);
@@ -126,6 +222,19 @@ int norm_rows(const float* x, const int* index, const void* w, const void* b, vo
 }
 template <typename T>
 int close(const CloseParams& p, int tokens, cudaStream_t s) {
+    // groups of four per thread: few tokens want many threads, many tokens more work per thread
+    const int quads = p.width / 4;
+    const auto fits = [&](int vpt) { return quads % (32 * vpt) == 0 && quads / vpt <= kMaxThreads; };
+    const auto at16 = [](const void* a) { return aligned16(a); };
+    const bool vectors = p.width % 4 == 0 && p.ld_gate % 8 == 0 && p.result_stride % 4 == 0 && at16(p.y) && at16(p.gate) && at16(p.gate_bias) &&
+                         at16(p.post_w) && at16(p.post_b) && at16(p.x_in) && at16(p.x_out) && at16(p.results) && at16(p.next_w) &&
+                         at16(p.next_b) && at16(p.normed);
+    if (vectors) {
+        if (fits(1) && (tokens < 64 || quads <= 256)) return qd_launch(sublayer_close_vec_kernel<T, 1>, dim3(tokens), dim3(quads), 0, s, 1, p);
+        if (fits(2)) return qd_launch(sublayer_close_vec_kernel<T, 2>, dim3(tokens), dim3(quads / 2), 0, s, 1, p);
+        if (fits(4)) return qd_launch(sublayer_close_vec_kernel<T, 4>, dim3(tokens), dim3(quads / 4), 0, s, 1, p);
+        if (fits(1)) return qd_launch(sublayer_close_vec_kernel<T, 1>, dim3(tokens), dim3(quads), 0, s, 1, p);
+    }
     const size_t smem = (size_t)p.width * 4;
     if (!allow_smem(sublayer_close_kernel<T>, smem)) return QD_ERR_UNSUPPORTED;
     return qd_launch(sublayer_close_kernel<T>, dim3(tokens), dim3(row_threads(p.width)), smem, s, 1, p);

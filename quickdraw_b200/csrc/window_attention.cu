@@ -4,8 +4,8 @@
 // sequence's cache does not grow with its length.
 //
 // Prompt chunks: attn_prepare_kernel (norm, rotation, ring rows) and attn_flash_kernel (mma.sync m16n8k16;
-// 64 packed (token, head of the group) rows per block, key tiles of 64 through two cp.async buffers, only
-// the tiles a row of the block can see; probabilities as two bf16 pieces).  attn_rows_kernel covers fp32
+// 64 or 128 packed (token, head of the group) rows per block, key tiles of 64 through two cp.async buffers,
+// only the tiles a row of the block can see; probabilities as two bf16 pieces).  attn_rows_kernel covers fp32
 // and shapes without 16-byte rows.  Decode: attn_step_kernel, one launch: norm and rotation in every
 // block, blocks = (key/value head, split of the window), the last block of a head merges.
 #include "typed.cuh"
@@ -122,7 +122,7 @@ __global__ void __launch_bounds__(256) attn_rows_kernel(const __grid_constant__ 
 }
 
 // ------------------------------------------------------------------------------- tensor cores
-constexpr int kFlashRows = 64, kFlashKeys = 64, kFlashThreads = 128;
+constexpr int kFlashKeys = 64;
 constexpr float kLog2e = 1.4426950408889634f;
 
 QD_DEVINL void mma_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -148,11 +148,11 @@ QD_DEVINL uint32_t pack_pair(float lo, float hi) {
 
 // dim, vdim multiples of eight, vdim <= DV (a multiple of sixteen).  Shared rows are padded to an odd
 // number of 16-byte pieces: the eight rows an ldmatrix phase touches fall into different banks.
-template <int DV>
-__global__ void __launch_bounds__(kFlashThreads) attn_flash_kernel(const __grid_constant__ AttnParams p) {
+template <int DV, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32) attn_flash_kernel(const __grid_constant__ AttnParams p) {
     chain_enter();
     extern __shared__ __align__(16) bf16 tiles[];
-    constexpr int kVRow = DV + 8;
+    constexpr int kVRow = DV + 8, kFlashRows = WARPS * 16, kFlashThreads = WARPS * 32;
     const int dk = (p.dim + 15) & ~15, krow = dk + 8;
     bf16* qs = tiles;
     bf16* ks = qs + kFlashRows * krow;
@@ -318,6 +318,20 @@ QD_DEVINL float dot_rows(const float* q, const T* k, int n) {
 }
 
 template <typename T>
+QD_DEVINL void dot_rows2(const float* q0, const float* q1, const T* k, int n, float& d0, float& d1) {
+    if ((n & 3) != 0) { d0 = dot_rows(q0, k, n); d1 = dot_rows(q1, k, n); return; }
+    float a0[4] = {0.f, 0.f, 0.f, 0.f}, a1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+    for (int d = 0; d < n; d += 4) {
+        const float4 kv = load4(k + d), x = load4(q0 + d), y = load4(q1 + d);
+        a0[0] = fmaf(x.x, kv.x, a0[0]); a0[1] = fmaf(x.y, kv.y, a0[1]); a0[2] = fmaf(x.z, kv.z, a0[2]); a0[3] = fmaf(x.w, kv.w, a0[3]);
+        a1[0] = fmaf(y.x, kv.x, a1[0]); a1[1] = fmaf(y.y, kv.y, a1[1]); a1[2] = fmaf(y.z, kv.z, a1[2]); a1[3] = fmaf(y.w, kv.w, a1[3]);
+    }
+    d0 = (a0[0] + a0[1]) + (a0[2] + a0[3]);
+    d1 = (a1[0] + a1[1]) + (a1[2] + a1[3]);
+}
+
+template <typename T>
 static size_t step_smem(int share, int dim, int vdim, int rot) {
     const int dp = (dim + kPad + 3) / 4 * 4, vp = (vdim + 3) / 4 * 4;
     return sizeof(float) * ((size_t)share * dp + (size_t)share * vp + share * (kStepKeys + 4) + 8 + rot) +
@@ -395,9 +409,21 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
             }
         }
         __syncthreads();
-        for (int i = tid; i < share * kStepKeys; i += kStepThreads) {
-            const int h = i / kStepKeys, r = i % kStepKeys;
-            score[i] = r < count ? dot_rows(qs + h * dp, ks + r * dp, dim) * p.scale : -INFINITY;
+        {       // a thread's key against two heads at a time
+            constexpr int kGroups = kStepThreads / kStepKeys;
+            const int r = tid % kStepKeys;
+            for (int h = tid / kStepKeys; h < share; h += 2 * kGroups) {
+                const int h2 = h + kGroups;
+                float d0 = -INFINITY, d1 = -INFINITY;
+                if (r < count) {
+                    if (h2 < share) dot_rows2(qs + h * dp, qs + h2 * dp, ks + r * dp, dim, d0, d1);
+                    else d0 = dot_rows(qs + h * dp, ks + r * dp, dim);
+                    d0 *= p.scale;
+                    d1 *= p.scale;
+                }
+                score[h * kStepKeys + r] = d0;
+                if (h2 < share) score[h2 * kStepKeys + r] = d1;
+            }
         }
         __syncthreads();
         for (int h = warp; h < share; h += kStepThreads / 32) {
@@ -417,23 +443,41 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
             }
         }
         __syncthreads();
-        for (int i = tid; i < share * vdim; i += kStepThreads) {
-            const int h = i / vdim, c = i % vdim;
-            float a = acc[h * vp + c] * stat[h * 4 + 2];
-            const float* w = score + h * kStepKeys;
-            for (int r = 0; r < count; ++r) a = fmaf(w[r], load_f(vs + r * vp + c), a);
-            acc[h * vp + c] = a;
+        if (quads) {
+            for (int i = tid; i < share * (vdim / 4); i += kStepThreads) {
+                const int h = i / (vdim / 4), c = i % (vdim / 4) * 4;
+                const float keep = stat[h * 4 + 2];
+                float4 a = load4(acc + h * vp + c);
+                a.x *= keep; a.y *= keep; a.z *= keep; a.w *= keep;
+                const float* w = score + h * kStepKeys;
+#pragma unroll 4
+                for (int r = 0; r < count; ++r) {
+                    const float4 v4 = load4(vs + r * vp + c);
+                    a.x = fmaf(w[r], v4.x, a.x); a.y = fmaf(w[r], v4.y, a.y); a.z = fmaf(w[r], v4.z, a.z); a.w = fmaf(w[r], v4.w, a.w);
+                }
+                store4(acc + h * vp + c, a);
+            }
+        } else {
+            for (int i = tid; i < share * vdim; i += kStepThreads) {
+                const int h = i / vdim, c = i % vdim;
+                float a = acc[h * vp + c] * stat[h * 4 + 2];
+                const float* w = score + h * kStepKeys;
+                for (int r = 0; r < count; ++r) a = fmaf(w[r], load_f(vs + r * vp + c), a);
+                acc[h * vp + c] = a;
+            }
         }
         __syncthreads();
     }
 
-    // partial results [head][split][vdim + 2]; the last split of this key/value head to arrive merges them
-    const int stride = vdim + 2;
-    for (int i = tid; i < share * stride; i += kStepThreads) {
-        const int h = i / stride, c = i % stride;
-        const float x = c < vdim ? acc[h * vp + c] : stat[h * 4 + (c - vdim)];
-        sp.partial[((size_t)(g * share + h) * sp.splits + split) * stride + c] = x;
+    // partial results: (maximum, denominator) [head][split], then sums [head][split][vdim]; the last split of this
+    // key/value head to arrive merges them
+    float2* stats = reinterpret_cast<float2*>(sp.partial) + (size_t)g * share * sp.splits;
+    float* sums = sp.partial + 2 * (size_t)p.heads * sp.splits + (size_t)g * share * sp.splits * vdim;
+    for (int i = tid; i < share * vdim; i += kStepThreads) {
+        const int h = i / vdim, c = i % vdim;
+        sums[((size_t)h * sp.splits + split) * vdim + c] = acc[h * vp + c];
     }
+    for (int h = tid; h < share; h += kStepThreads) stats[h * sp.splits + split] = make_float2(stat[h * 4], stat[h * 4 + 1]);
     __threadfence();
     __syncthreads();
     if (tid == 0) last = atomicAdd(sp.counters + g, 1u) == (unsigned)active - 1u;
@@ -441,30 +485,50 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
     if (!last) return;
     __threadfence();
     if (tid == 0) sp.counters[g] = 0u;
-    for (int i = tid; i < share * vdim; i += kStepThreads) {
-        const int h = i / vdim, c = i % vdim, head = g * share + h;
-        const float* rows = sp.partial + (size_t)head * sp.splits * stride;
+    // factor of every split (sink, denominator and gate included) into the score rows, then the weighted sums
+    for (int h = warp; h < share; h += kStepThreads / 32) {
+        const int head = g * share + h;
         const float sink = ld_bf16(p.sink + head);
-        float top = sink;
-        for (int s = 0; s < active; ++s) top = fmaxf(top, __ldcg(rows + (size_t)s * stride + vdim));
-        float sum = expf(sink - top), o = 0.f;
-        for (int s = 0; s < active; ++s) {
-            const float f = expf(__ldcg(rows + (size_t)s * stride + vdim) - top);
-            sum = fmaf(__ldcg(rows + (size_t)s * stride + vdim + 1), f, sum);
-            o = fmaf(__ldcg(rows + (size_t)s * stride + c), f, o);
+        float2 mine[kStepKeys / 32];
+        float top = sink, sum = 0.f;
+#pragma unroll
+        for (int i = 0; i < kStepKeys / 32; ++i) {
+            const int s = i * 32 + lane;
+            mine[i] = s < active ? __ldcg(stats + h * sp.splits + s) : make_float2(-INFINITY, 0.f);
+            top = fmaxf(top, mine[i].x);
         }
-        const float gate = sigmoid_precise(load_f(reinterpret_cast<const T*>(p.gate) + head));
-        store_f(reinterpret_cast<T*>(p.out) + head * vdim + c, o / sum * gate);
+        top = warp_max(top);
+#pragma unroll
+        for (int i = 0; i < kStepKeys / 32; ++i) { mine[i].x = expf(mine[i].x - top); sum = fmaf(mine[i].y, mine[i].x, sum); }
+        const float f = sigmoid_precise(load_f(reinterpret_cast<const T*>(p.gate) + head)) / (warp_sum(sum) + expf(sink - top));
+#pragma unroll
+        for (int i = 0; i < kStepKeys / 32; ++i) score[h * kStepKeys + i * 32 + lane] = mine[i].x * f;
+    }
+    __syncthreads();
+    for (int i = tid; i < share * vdim; i += kStepThreads) {
+        const int h = i / vdim, c = i % vdim;
+        const float* rows = sums + (size_t)h * sp.splits * vdim + c;
+        float o = 0.f;
+#pragma unroll 8
+        for (int s = 0; s < active; ++s) o = fmaf(__ldcg(rows + (size_t)s * vdim), score[h * kStepKeys + s], o);
+        store_f(reinterpret_cast<T*>(p.out) + (g * share + h) * vdim + c, o);
     }
 }
 
+template <int DV, int WARPS>
+int launch_flash_rows(const AttnParams& p, long long rows, cudaStream_t s) {
+    const int krow = ((p.dim + 15) & ~15) + 8;
+    const size_t smem = sizeof(bf16) * ((size_t)(WARPS * 16 + 2 * kFlashKeys) * krow + 2ull * kFlashKeys * (DV + 8));
+    if (!allow_smem(attn_flash_kernel<DV, WARPS>, smem)) return QD_ERR_UNSUPPORTED;
+    const dim3 grid((unsigned)((rows + WARPS * 16 - 1) / (WARPS * 16)), p.kv_heads);
+    return qd_launch(attn_flash_kernel<DV, WARPS>, grid, dim3(WARPS * 32), smem, s, 1, p);
+}
 template <int DV>
 int launch_flash(const AttnParams& p, cudaStream_t s) {
-    const int krow = ((p.dim + 15) & ~15) + 8;
-    const size_t smem = sizeof(bf16) * ((size_t)(kFlashRows + 2 * kFlashKeys) * krow + 2ull * kFlashKeys * (DV + 8));
-    if (!allow_smem(attn_flash_kernel<DV>, smem)) return QD_ERR_UNSUPPORTED;
     const long long rows = (long long)p.tokens * (p.heads / p.kv_heads);
-    return qd_launch(attn_flash_kernel<DV>, dim3((unsigned)((rows + kFlashRows - 1) / kFlashRows), p.kv_heads), dim3(kFlashThreads), smem, s, 1, p);
+    // 128 rows share a key tile once such blocks fill the GPU
+    if (rows * p.kv_heads >= 128ll * device_sms()) return launch_flash_rows<DV, 8>(p, rows, s);
+    return launch_flash_rows<DV, 4>(p, rows, s);
 }
 template <typename T>
 int chunk(const AttnParams& p, cudaStream_t s) {
@@ -522,7 +586,7 @@ extern "C" int qd_window_attention_step(const void* q, const void* k, const void
                                         void* k_cache, void* v_cache, int capacity, int window, const int* position_ptr, int position,
                                         float* partial, unsigned int* counters, int splits, void* out, int heads, int kv_heads,
                                         int dim, int vdim, int dtype, void* stream) {
-    QD_ATTN_ARGS_OK(partial && counters && splits > 0);
+    QD_ATTN_ARGS_OK(partial && counters && splits > 0 && splits <= qd::kStepKeys);
     const qd::AttnStep sp = {{q, k, v, gate, 0, (const bf16*)q_norm, (const bf16*)k_norm, freq, rot, (const bf16*)sink, scale, eps, k_cache,
                               v_cache, capacity, window, position_ptr, position, nullptr, out, 1, heads, kv_heads, dim, vdim},
                              partial, counters, splits};

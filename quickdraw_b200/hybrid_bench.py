@@ -249,9 +249,11 @@ class Cases:
         own = [lambda r=r: call_hybrid("qd_sublayer_close", ptr(y), ptr(gate), width, ptr(vec), ptr(vec), ptr(vec), ptr(stream), ptr(stream),
                                        ptr(r), r.stride(0), ptr(depth), older, ptr(vec), ptr(vec), ptr(normed), tokens, width, 1e-6, 0,
                                        stream_of(y)) for r in results for _ in range(4)]
-        gamma, res, new = self.rnd(width, dtype=F32), self.rnd(tokens, width), self.rnd(tokens, width)
-        like = lambda: call("qd_seq_add_rms_norm", ptr(y), ptr(res), ptr(gamma), ptr(normed), ptr(new), tokens, width, 1e-6, stream_of(y))
-        self.pair(f"sublayer_close_kernel {tokens} x {width}, {older} earlier results", (own, nbytes), "seq_add_norm", ([like] * 8, tokens * width * 8))
+        gamma = self.rnd(width, dtype=F32)
+        four = [[self.rnd(tokens, width) for _ in range(4)] for _ in range(sets_for(tokens * width * 8))]
+        like = [lambda f=f: call("qd_seq_add_rms_norm", ptr(f[0]), ptr(f[1]), ptr(gamma), ptr(f[2]), ptr(f[3]), tokens, width, 1e-6, stream_of(y))
+                for f in four]
+        self.pair(f"sublayer_close_kernel {tokens} x {width}, {older} earlier results", (own, nbytes), "seq_add_norm", (like, tokens * width * 8))
 
 
 def step_bytes(engine, position: int) -> float:
