@@ -54,16 +54,17 @@ int qd_gla_prepare(const void* q, const void* k, const void* v, long long ld, co
 
 /* fp32 operands of the channel-decay delta rule: q, k, v through a causal convolution of `taps` taps (history ring
  * [taps, channels q | k | v], position p in row p mod taps; updated with the chunk's last inputs) and SiLU, q and k as
- * unit vectors per head (q also / sqrt(dim)), og = exp(-exp(a_log) softplus(z + z_bias)) - 1 (og may be z), obeta = sigmoid(beta),
- * okq = k . q.  The position of the chunk's first token is *position_ptr, or `position` if that is NULL. */
+ * not yet unit vectors: oscales [tokens, kv_heads, 3] = the factors that make k and
+ * q unit vectors (q's also / sqrt(dim)) and k . q of the results, og = exp(-exp(a_log) softplus(z + z_bias)) - 1 (og may be z), obeta = sigmoid(beta).
+ * The position of the chunk's first token is *position_ptr, or `position` if that is NULL. */
 int qd_channel_delta_prepare(const void* q, const void* k, const void* v, const void* beta, long long ld, const
     float* z, const void* z_bias, const void* a_log, const void* q_taps, const void* k_taps, const void* v_taps,
     void* history, int taps, const int* position_ptr, int position, float* oq, float* ok, float* og, float* ov,
-    float* obeta, float* okq, int tokens, int heads, int kv_heads, int dim, int vdim, int dtype, void* stream);
+    float* obeta, float* oscales, int tokens, int heads, int kv_heads, int dim, int vdim, int dtype, void* stream);
 
 /* The recurrence over a chunk; q, k [tokens, kv_heads, dim], g [tokens, heads, dim], v, out [tokens, heads, vdim], state
  * [heads, dim, vdim] fp32, updated in place.  delta = 0: S = diag(1 + g) S + k v^T; 1: S = diag(1 + g) S,
- * u = beta (v - S^T k), S += k u^T; out = S^T q.  dim <= 256. */
+ * u = beta (v - S^T k), S += k u^T, with k and q times their scales; out = S^T q.  dim <= 256. */
 int qd_linear_recurrence(const float* q, const float* k, const float* g, const float* v, const float* beta, const
     float* kq, float* state, float* out, int tokens, int heads, int kv_heads, int dim, int vdim, int delta, void*
     stream);

@@ -15,9 +15,9 @@ namespace qd {
 namespace {
 
 // ------------------------------------------------------------------------------ few token rows
-// Inputs staged at a time: sixteen 16-byte pieces of weights per lane while one or two token rows leave the registers
-// and the shared memory for it.
-constexpr int rows_chunk(int R, int NR) { return (R <= 2 ? 4096 : (R == 4 ? 2048 : 1024)) / NR; }
+// Inputs staged at a time.  One weight row per warp (few rows: one or two blocks per SM): up to sixteen 16-byte
+// pieces per lane in flight; two rows per warp: eight, and more blocks.
+constexpr int rows_chunk(int R, int NR) { return NR == 2 ? 1024 : (R <= 2 ? 4096 : (R == 4 ? 2048 : 1024)); }
 
 template <typename TX, typename TY, int R, int NR>
 __global__ void __launch_bounds__(256)

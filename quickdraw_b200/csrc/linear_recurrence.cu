@@ -3,8 +3,8 @@
 //   channel-decay delta rule S = diag(g) S, u = beta (v - S^T k), S = S + k u^T,  o = S^T q
 // (gdn.cu has the delta rule with one decay per head.)  Everything that enters the recurrence is fp32.
 //
-// Prompt chunks: a prepare kernel (all tokens in parallel: short convolution, SiLU, unit norms, decays)
-// writes q, k, decay, v, beta as fp32 rows; linear_recurrence_kernel walks the tokens with the state in
+// Prompt chunks: a prepare kernel (all tokens in parallel: short convolution, SiLU, decays) writes q, k,
+// decay, v, beta as fp32 rows, unit_scales_kernel the factors that make q and k unit vectors; linear_recurrence_kernel walks the tokens with the state in
 // registers.  A warp owns eight value columns; a lane a group of key rows and a few columns, held as row
 // pairs for the packed fp32 FMA.  Both read-outs of the delta rule use the decayed state before the
 // write, o = (gS)^T q + (k . q) u, so that the second one hides in the first one's shuffles.
@@ -59,7 +59,7 @@ struct PrepareParams {
     const bf16* q_taps; const bf16* k_taps; const bf16* v_taps; ConvSource conv;
     float tau;
     const int* position_ptr; int position;
-    float* oq; float* ok; float* og; float* ov; float* obeta; float* okq;
+    float* oq; float* ok; float* og; float* ov; float* obeta; float* oscales;
     int tokens, heads, kv_heads, dim, vdim;
 };
 
@@ -80,133 +80,106 @@ __global__ void __launch_bounds__(256) gla_prepare_kernel(const __grid_constant_
     for (int i = threadIdx.x; i < values; i += blockDim.x) p.ov[t * values + i] = load_f(v + i);
 }
 
-constexpr int kMaxPerLane = 8;       // key channels per lane: dim <= 256
-constexpr int kPrepareTokens = 8;    // tokens a block walks with the convolution's window in registers
+constexpr int kPrepareTokens = 8;    // tokens of one channel per thread, all their inputs requested at once
 
-// The window of one channel: `back` of token t is the input of the position `back` before it.
-// TAPS == 0: any number, every input read again for every token.
-template <typename T, int TAPS> struct ConvWindow {
-    float w[TAPS ? TAPS : 1], x[TAPS ? TAPS : 1];
-    // before the first of the block's tokens, t: loads the taps and the inputs of t - TAPS + 1 .. t - 1
-    QD_DEVINL void open(const T* row0, long long ld, int t, int position, const bf16* taps, const ConvSource& src, int channel) {
-#pragma unroll
-        for (int j = 0; j < TAPS; ++j) w[j] = ld_bf16(taps + j);
-#pragma unroll
-        for (int j = 1; j < TAPS; ++j) {
-            const int back = TAPS - j, at = t - back, p = position - back;      // becomes x[j - 1] when t's input arrives
-            x[j] = at >= 0 ? load_f(row0 + (long long)at * ld)
-                           : (p >= 0 ? load_f(reinterpret_cast<const T*>(src.history) + (size_t)(p % src.taps) * src.channels + channel) : 0.f);
-        }
-    }
-    QD_DEVINL float next(const T* row0, long long ld, int t, int position, const bf16* taps, const ConvSource& src, int channel) {
-        if (TAPS == 0) return conv_at(row0 + (long long)t * ld, ld, t, position, taps, src, channel);
-#pragma unroll
-        for (int j = 1; j < TAPS; ++j) x[j - 1] = x[j];
-        x[TAPS ? TAPS - 1 : 0] = load_f(row0 + (long long)t * ld);
-        float acc = 0.f;
-#pragma unroll
-        for (int j = 0; j < TAPS; ++j) acc = fmaf(x[j], w[j], acc);
-        return acc;
-    }
-};
-
-// blockIdx.y: groups of eight key/value heads (a warp each), then groups of 256 value channels, then
-// groups of 256 decay channels (the first of these also the step sizes).
+// blockIdx.y: groups of 256 convolution channels (q | k | v), then groups of 256 decay channels (the
+// first of these also the step sizes).  TAPS == 0: any number of taps.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256) delta_prepare_kernel(const __grid_constant__ PrepareParams p) {
     chain_enter();
-    const int t0 = blockIdx.x * kPrepareTokens, t1 = min(t0 + kPrepareTokens, p.tokens), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = blockIdx.x * kPrepareTokens, count = min(kPrepareTokens, p.tokens - t0);
     const int base = p.position_ptr ? *p.position_ptr : p.position;
-    const int keys = p.heads * p.dim, values = p.heads * p.vdim, kv_keys = p.kv_heads * p.dim;
-    const int head_groups = (p.kv_heads + 7) / 8, value_groups = (values + 255) / 256;
+    const int keys = p.heads * p.dim, values = p.heads * p.vdim, kv_keys = p.kv_heads * p.dim, channels = 2 * kv_keys + values;
+    const int conv_groups = (channels + 255) / 256;
     int group = blockIdx.y;
-    if (group < head_groups) {
-        const T* q = reinterpret_cast<const T*>(p.q);
-        const T* k = reinterpret_cast<const T*>(p.k);
-        const float scale = 1.0f / sqrtf((float)p.dim);
-        const int h = group * 8 + warp;
-        if (h >= p.kv_heads) return;
-        ConvWindow<T, TAPS> wq[kMaxPerLane / 2], wk[kMaxPerLane / 2];
-        const bool windows = p.dim <= 32 * (kMaxPerLane / 2);      // wider heads read their inputs again
-        if (windows)
+    if (group < conv_groups) {
+        const int channel = group * 256 + threadIdx.x;
+        if (channel >= channels) return;
+        const int which = channel < kv_keys ? 0 : (channel < 2 * kv_keys ? 1 : 2), c = channel - which * kv_keys;
+        const T* x = reinterpret_cast<const T*>(which == 0 ? p.q : (which == 1 ? p.k : p.v)) + c;
+        const bf16* taps = (which == 0 ? p.q_taps : (which == 1 ? p.k_taps : p.v_taps)) + (size_t)c * p.conv.taps;
+        float* out = which == 0 ? p.oq : (which == 1 ? p.ok : p.ov);
+        const int width = which == 2 ? values : kv_keys;
+        out += (size_t)t0 * width + c;
+        if (TAPS == 0) {
+            for (int i = 0; i < count; ++i)
+                out[(size_t)i * width] = silu_precise(conv_at(x + (long long)(t0 + i) * p.ld, p.ld, t0 + i, base + t0 + i, taps, p.conv, channel));
+            return;
+        }
+        constexpr int kBack = TAPS ? TAPS - 1 : 0;
+        float w[kBack + 1], in[kBack + kPrepareTokens];
 #pragma unroll
-            for (int i = 0; i < kMaxPerLane / 2; ++i) {
-                const int d = i * 32 + lane, c = h * p.dim + d;
-                if (d < p.dim) {
-                    wq[i].open(q + c, p.ld, t0, base + t0, p.q_taps + (size_t)c * p.conv.taps, p.conv, c);
-                    wk[i].open(k + c, p.ld, t0, base + t0, p.k_taps + (size_t)c * p.conv.taps, p.conv, kv_keys + c);
-                }
-            }
-        for (int t = t0; t < t1; ++t) {
-            float qv[kMaxPerLane], kv[kMaxPerLane], qq = 0.f, kk = 0.f, kq = 0.f;
+        for (int j = 0; j <= kBack; ++j) w[j] = ld_bf16(taps + j);
 #pragma unroll
-            for (int i = 0; i < kMaxPerLane; ++i) {
-                const int d = i * 32 + lane, c = h * p.dim + d;
-                qv[i] = kv[i] = 0.f;
-                if (d < p.dim) {
-                    const bf16* qt = p.q_taps + (size_t)c * p.conv.taps;
-                    const bf16* kt = p.k_taps + (size_t)c * p.conv.taps;
-                    if (windows && i < kMaxPerLane / 2) {
-                        qv[i] = wq[i % (kMaxPerLane / 2)].next(q + c, p.ld, t, base + t, qt, p.conv, c);
-                        kv[i] = wk[i % (kMaxPerLane / 2)].next(k + c, p.ld, t, base + t, kt, p.conv, kv_keys + c);
-                    } else {
-                        qv[i] = conv_at(q + c + (long long)t * p.ld, p.ld, t, base + t, qt, p.conv, c);
-                        kv[i] = conv_at(k + c + (long long)t * p.ld, p.ld, t, base + t, kt, p.conv, kv_keys + c);
-                    }
-                    qv[i] = silu_precise(qv[i]);
-                    kv[i] = silu_precise(kv[i]);
-                }
-                qq = fmaf(qv[i], qv[i], qq);
-                kk = fmaf(kv[i], kv[i], kk);
-                kq = fmaf(qv[i], kv[i], kq);
-            }
-            qq = warp_sum(qq); kk = warp_sum(kk); kq = warp_sum(kq);
-            const float qs = scale / sqrtf(qq + kUnitEps), ks = 1.0f / sqrtf(kk + kUnitEps);
-            const size_t at = (size_t)t * kv_keys + h * p.dim;
+        for (int j = 0; j < kBack + kPrepareTokens; ++j) {
+            const int t = t0 + j - kBack, at = base + t;
+            in[j] = 0.f;
+            if (t >= 0) { if (t < p.tokens) in[j] = load_f(x + (long long)t * p.ld); }
+            else if (at >= 0) in[j] = load_f(reinterpret_cast<const T*>(p.conv.history) + (size_t)(at % p.conv.taps) * channels + channel);
+        }
 #pragma unroll
-            for (int i = 0; i < kMaxPerLane; ++i) {
-                const int d = i * 32 + lane;
-                if (d < p.dim) { p.oq[at + d] = qv[i] * qs; p.ok[at + d] = kv[i] * ks; }
-            }
-            if (lane == 0) p.okq[(size_t)t * p.kv_heads + h] = kq * qs * ks;
+        for (int i = 0; i < kPrepareTokens; ++i) {
+            float acc = 0.f;
+#pragma unroll
+            for (int j = 0; j <= kBack; ++j) acc = fmaf(in[i + j], w[j], acc);
+            if (i < count) out[(size_t)i * width] = silu_precise(acc);
         }
         return;
     }
-    group -= head_groups;
-    if (group < value_groups) {
-        const int c = group * 256 + threadIdx.x, channel = 2 * kv_keys + c;
-        if (c >= values) return;
-        const T* v = reinterpret_cast<const T*>(p.v) + c;
-        const bf16* taps = p.v_taps + (size_t)c * p.conv.taps;
-        ConvWindow<T, TAPS> w;
-        w.open(v, p.ld, t0, base + t0, taps, p.conv, channel);
-        for (int t = t0; t < t1; ++t) p.ov[(size_t)t * values + c] = silu_precise(w.next(v, p.ld, t, base + t, taps, p.conv, channel));
-        return;
-    }
-    group -= value_groups;
+    group -= conv_groups;
     const int c = group * 256 + threadIdx.x;
     if (c < keys) {
         const float bias = ld_bf16(p.z_bias + c), rate = expf(ld_bf16(p.a_log + c / p.dim));
-#pragma unroll 4
-        for (int t = t0; t < t1; ++t) p.og[(size_t)t * keys + c] = delta_decay_less_one(p.z[(size_t)t * keys + c] + bias, rate);
+        float z[kPrepareTokens];
+#pragma unroll
+        for (int i = 0; i < kPrepareTokens; ++i) z[i] = i < count ? p.z[(size_t)(t0 + i) * keys + c] : 0.f;
+#pragma unroll
+        for (int i = 0; i < kPrepareTokens; ++i)
+            if (i < count) p.og[(size_t)(t0 + i) * keys + c] = delta_decay_less_one(z[i] + bias, rate);
     }
     if (group == 0)
-        for (int i = threadIdx.x; i < (t1 - t0) * p.heads; i += 256) {
+        for (int i = threadIdx.x; i < count * p.heads; i += 256) {
             const int t = t0 + i / p.heads, h = i % p.heads;
             p.obeta[(size_t)t * p.heads + h] = sigmoid_precise(load_f(reinterpret_cast<const T*>(p.beta) + (long long)t * p.ld + h));
         }
 }
 
+// Per token and key/value head: the factors that make k and q unit vectors (q's with 1 / sqrt(dim)) and
+// k . q of the results.  A warp each.
+__global__ void __launch_bounds__(256)
+unit_scales_kernel(const float* __restrict__ q, const float* __restrict__ k, float* __restrict__ scales, long long rows, int dim) {
+    chain_enter();
+    const long long row = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (row >= rows) return;
+    float qq = 0.f, kk = 0.f, kq = 0.f;
+    for (int d = lane; d < dim; d += 32) {
+        const float a = q[row * dim + d], b = k[row * dim + d];
+        qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); kq = fmaf(a, b, kq);
+    }
+    qq = warp_sum(qq); kk = warp_sum(kk); kq = warp_sum(kq);
+    if (lane == 0) {
+        const float ks = 1.0f / sqrtf(kk + kUnitEps), qs = 1.0f / (sqrtf(qq + kUnitEps) * sqrtf((float)dim));
+        scales[row * 3] = ks;
+        scales[row * 3 + 1] = qs;
+        scales[row * 3 + 2] = kq * ks * qs;
+    }
+}
+
 template <typename T>
 int launch_delta_prepare(const PrepareParams& p, cudaStream_t s) {
-    const int groups = (p.kv_heads + 7) / 8 + (p.heads * p.vdim + 255) / 256 + (p.heads * p.dim + 255) / 256;
+    const int groups = (2 * p.kv_heads * p.dim + p.heads * p.vdim + 255) / 256 + (p.heads * p.dim + 255) / 256;
     const dim3 grid((p.tokens + kPrepareTokens - 1) / kPrepareTokens, groups);
+    int rc;
     switch (p.conv.taps) {
-        case 2: return qd_launch(delta_prepare_kernel<T, 2>, grid, dim3(256), 0, s, 1, p);
-        case 3: return qd_launch(delta_prepare_kernel<T, 3>, grid, dim3(256), 0, s, 1, p);
-        case 4: return qd_launch(delta_prepare_kernel<T, 4>, grid, dim3(256), 0, s, 1, p);
-        default: return qd_launch(delta_prepare_kernel<T, 0>, grid, dim3(256), 0, s, 1, p);
+        case 2: rc = qd_launch(delta_prepare_kernel<T, 2>, grid, dim3(256), 0, s, 1, p); break;
+        case 3: rc = qd_launch(delta_prepare_kernel<T, 3>, grid, dim3(256), 0, s, 1, p); break;
+        case 4: rc = qd_launch(delta_prepare_kernel<T, 4>, grid, dim3(256), 0, s, 1, p); break;
+        default: rc = qd_launch(delta_prepare_kernel<T, 0>, grid, dim3(256), 0, s, 1, p); break;
     }
+    if (rc != QD_OK) return rc;
+    const long long rows = (long long)p.tokens * p.kv_heads;
+    return qd_launch(unit_scales_kernel, dim3((unsigned)((rows + 7) / 8)), dim3(256), 0, s, 1, p.oq, p.ok, p.oscales, rows, p.dim);
 }
 
 // The chunk's last `taps` inputs into the history ring.
@@ -242,36 +215,31 @@ template <int N> QD_DEVINL void copies_wait() { asm volatile("cp.async.wait_grou
 constexpr int kRecThreads = 128, kRecCols = 32, kRecTile = 16;      // block: four warps x eight columns; tokens per staged tile
 
 struct RecurrenceParams {
-    const float* q; const float* k; const float* g; const float* v; const float* beta; const float* kq;
+    const float* q; const float* k; const float* g; const float* v; const float* beta;
+    const float* scales;          // delta rule: per token and key/value head the factors that make k and q unit vectors (q's / sqrt(dim)), k . q of the unit vectors
     float* state; float* out;
     int tokens, heads, kv_heads, dim, vdim, vectors;
 };
 
-// floats of one staged token: q, k, decay - 1 (padded to `row`), v columns, beta, k . q (padded to 4)
+// floats of one staged token: q, k, decay - 1 (padded to `row`), v columns, step size and the three scales
 constexpr int rec_token_floats(int row) { return 3 * row + kRecCols + 4; }
 
 // A token's vectors, this lane's rows.
 template <int J> struct RecVectors { ulonglong2 q[J], k[J], g[J]; };
 
-// Sums over the KL lanes of a key group; every lane ends up with the sum of ONE of its CC columns (the
-// column index is returned), so that a round moves half of what the round before it did.
-template <int KL, int CC>
-QD_DEVINL int reduce_columns(const float (&v)[CC], int kl, float& total) {
-    if (CC == 2) {
-        const bool odd = kl & 1;
-        total = (odd ? v[1] : v[0]) + __shfl_xor_sync(0xffffffffu, odd ? v[0] : v[1], 1);
+// Four tokens' read-outs of CC = KL / 4 columns, summed over the KL lanes of a key group: KL values over KL
+// lanes, so every round exchanges half of what is left and lane kl ends up with value kl (token kl / CC,
+// column kl % CC).
+template <int KL>
+QD_DEVINL float scatter_sum(float (&v)[KL], int kl) {
 #pragma unroll
-        for (int x = 2; x < KL; x <<= 1) total += __shfl_xor_sync(0xffffffffu, total, x);
-        return kl & 1;
+    for (int x = KL / 2; x >= 1; x >>= 1) {
+        const bool upper = kl & x;
+#pragma unroll
+        for (int i = 0; i < x; ++i)
+            v[i] = (upper ? v[i + x] : v[i]) + __shfl_xor_sync(0xffffffffu, upper ? v[i] : v[i + x], x);
     }
-    const bool upper = kl & 1, odd = kl & 2;
-    float a = upper ? v[CC - 2] : v[0], b = upper ? v[CC - 1] : v[1];
-    a += __shfl_xor_sync(0xffffffffu, upper ? v[0] : v[CC - 2], 1);
-    b += __shfl_xor_sync(0xffffffffu, upper ? v[1] : v[CC - 1], 1);
-    total = (odd ? b : a) + __shfl_xor_sync(0xffffffffu, odd ? a : b, 2);
-#pragma unroll
-    for (int x = 4; x < KL; x <<= 1) total += __shfl_xor_sync(0xffffffffu, total, x);
-    return (upper ? 2 : 0) + (odd ? 1 : 0);
+    return v[0];
 }
 
 // KL lanes share a column's keys (rows 4 KL j + 4 kl + {0..3}), a lane holds CC = KL / 4 columns: more
@@ -327,7 +295,7 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
         if (DELTA && tid < count) {
             float* dst = base + tid * kToken + 3 * kRow + kRecCols;
             copy4(dst, p.beta + (size_t)(t0 + tid) * p.heads + head);
-            copy4(dst + 1, p.kq + (size_t)(t0 + tid) * p.kv_heads + kv);
+            for (int i = 0; i < 3; ++i) copy4(dst + 1 + i, p.scales + ((size_t)(t0 + tid) * p.kv_heads + kv) * 3 + i);
         }
         copies_commit();
     };
@@ -341,17 +309,16 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
     };
     float* out = p.out + (size_t)head * vdim;
     const size_t out_stride = (size_t)p.heads * vdim;
-    auto advance = [&](const RecVectors<J>& f, const float* token) {
-        float v[CC], o[CC], u[CC];
-#pragma unroll
-        for (int c = 0; c < CC; ++c) v[c] = token[3 * kRow + local + c];
+    // one token; o: the read-outs of this lane's rows
+    auto advance = [&](const RecVectors<J>& f, const float* token, float* o) {
+        float v[CC];
+        if (CC == 2) { const float2 x = *reinterpret_cast<const float2*>(token + 3 * kRow + local); v[0] = x.x; v[1] = x.y; }
+        else { const float4 x = *reinterpret_cast<const float4*>(token + 3 * kRow + local); v[0] = x.x; v[1] = x.y; v[CC - 2] = x.z; v[CC - 1] = x.w; }
         u64 oa[CC], ob[CC];
 #pragma unroll
         for (int c = 0; c < CC; ++c) oa[c] = ob[c] = 0ull;
-        float kq = 0.f;
         if (DELTA) {
-            const float2 bk = *reinterpret_cast<const float2*>(token + 3 * kRow + kRecCols);      // beta, k . q
-            kq = bk.y;
+            const float4 w = *reinterpret_cast<const float4*>(token + 3 * kRow + kRecCols);      // step size, scale of k, of q, k . q
             u64 pa[CC], pb[CC];
             float pred[CC];
 #pragma unroll
@@ -379,15 +346,16 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
                     ob[c] = fma2(s[j][1][c], f.q[j].y, ob[c]);
                 }
 #pragma unroll
-            for (int c = 0; c < CC; ++c) u[c] = bk.x * (v[c] - pred[c]);
+            for (int c = 0; c < CC; ++c) {
+                const float u = w.x * fmaf(-w.y, pred[c], v[c]), ku = w.y * u;
+                const u64 uu = pack2(ku, ku);
 #pragma unroll
-            for (int j = 0; j < J; ++j)
-#pragma unroll
-                for (int c = 0; c < CC; ++c) {
-                    const u64 uu = pack2(u[c], u[c]);
+                for (int j = 0; j < J; ++j) {
                     s[j][0][c] = fma2(f.k[j].x, uu, s[j][0][c]);
                     s[j][1][c] = fma2(f.k[j].y, uu, s[j][1][c]);
                 }
+                o[c] = fmaf(w.z, (lo2(oa[c]) + hi2(oa[c])) + (lo2(ob[c]) + hi2(ob[c])), kl == 0 ? u * w.w : 0.f);
+            }
         } else {
 #pragma unroll
             for (int c = 0; c < CC; ++c) {
@@ -399,20 +367,9 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
                     oa[c] = fma2(s[j][0][c], f.q[j].x, oa[c]);
                     ob[c] = fma2(s[j][1][c], f.q[j].y, ob[c]);
                 }
+                o[c] = (lo2(oa[c]) + hi2(oa[c])) + (lo2(ob[c]) + hi2(ob[c]));
             }
         }
-#pragma unroll
-        for (int c = 0; c < CC; ++c) o[c] = (lo2(oa[c]) + hi2(oa[c])) + (lo2(ob[c]) + hi2(ob[c]));
-        float total;
-        const int mine = reduce_columns<KL, CC>(o, kl, total);
-        if (DELTA) {
-            float um = u[0];
-#pragma unroll
-            for (int c = 1; c < CC; ++c) um = mine == c ? u[c] : um;
-            total = fmaf(um, kq, total);
-        }
-        if (kl < CC && col + mine < vdim) out[col + mine] = total;
-        out += out_stride;
     };
 
     const int ntiles = (p.tokens + kRecTile - 1) / kRecTile;
@@ -424,14 +381,23 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
         const int count = min(kRecTile, p.tokens - tile * kRecTile);
         RecVectors<J> even, odd;                     // the next token's vectors are read while this one is reduced
         fetch(token, even);
-        int tt = 0;
-        for (; tt + 2 <= count; tt += 2, token += 2 * kToken) {
-            fetch(token + kToken, odd);
-            advance(even, token);
+        for (int tt = 0; tt < count; tt += 4, token += 4 * kToken) {
+            float o[KL];
+#pragma unroll
+            for (int i = 0; i < KL; ++i) o[i] = 0.f;
+            if (tt + 1 < count) fetch(token + kToken, odd);
+            advance(even, token, o);
             if (tt + 2 < count) fetch(token + 2 * kToken, even);
-            advance(odd, token + kToken);
+            if (tt + 1 < count) advance(odd, token + kToken, o + CC);
+            if (tt + 3 < count) fetch(token + 3 * kToken, odd);
+            if (tt + 2 < count) advance(even, token + 2 * kToken, o + 2 * CC);
+            if (tt + 4 < count) fetch(token + 4 * kToken, even);
+            if (tt + 3 < count) advance(odd, token + 3 * kToken, o + 3 * CC);
+            const float mine = scatter_sum<KL>(o, kl);
+            const int t = kl / CC, c = kl % CC;
+            if (tt + t < count && col + c < vdim) out[t * out_stride + col + c] = mine;
+            out += 4 * out_stride;
         }
-        if (tt < count) advance(even, token);
         __syncthreads();                 // the buffer may be refilled
     }
 #pragma unroll
@@ -725,15 +691,14 @@ extern "C" int qd_gla_prepare(const void* q, const void* k, const void* v, long 
 extern "C" int qd_channel_delta_prepare(const void* q, const void* k, const void* v, const void* beta, long long ld, const float* z,
                                         const void* z_bias, const void* a_log, const void* q_taps, const void* k_taps,
                                         const void* v_taps, void* history, int taps, const int* position_ptr, int position,
-                                        float* oq, float* ok, float* og, float* ov, float* obeta, float* okq, int tokens, int heads,
+                                        float* oq, float* ok, float* og, float* ov, float* obeta, float* oscales, int tokens, int heads,
                                         int kv_heads, int dim, int vdim, int dtype, void* stream) {
-    QD_CHECK_ARG(q && k && v && beta && z && z_bias && a_log && q_taps && k_taps && v_taps && history && oq && ok && og && ov && obeta && okq);
+    QD_CHECK_ARG(q && k && v && beta && z && z_bias && a_log && q_taps && k_taps && v_taps && history && oq && ok && og && ov && obeta && oscales);
     QD_CHECK_ARG(tokens > 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && vdim > 0 && taps > 0 && position >= 0);
-    if (dim > 32 * qd::kMaxPerLane) return QD_ERR_UNSUPPORTED;
     const int kv_keys = kv_heads * dim, values = heads * vdim;
     qd::PrepareParams p = {q, k, v, ld, z, (const bf16*)z_bias, beta, (const bf16*)a_log, (const bf16*)q_taps, (const bf16*)k_taps,
                            (const bf16*)v_taps, {history, taps, 2 * kv_keys + values}, 1.f, position_ptr, position, oq, ok, og, ov,
-                           obeta, okq, tokens, heads, kv_heads, dim, vdim};
+                           obeta, oscales, tokens, heads, kv_heads, dim, vdim};
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype != QD_BF16 && dtype != QD_F32) return QD_ERR_UNSUPPORTED;
     const int rc = dtype == QD_BF16 ? qd::prepare<bf16, true>(p, tokens, s) : qd::prepare<float, true>(p, tokens, s);
@@ -742,13 +707,13 @@ extern "C" int qd_channel_delta_prepare(const void* q, const void* k, const void
                             : qd::history<float>(q, k, v, ld, history, taps, kv_keys, values, tokens, position_ptr, position, s);
 }
 
-extern "C" int qd_linear_recurrence(const float* q, const float* k, const float* g, const float* v, const float* beta, const float* kq,
-                                    float* state, float* out, int tokens, int heads, int kv_heads, int dim, int vdim, int delta,
+extern "C" int qd_linear_recurrence(const float* q, const float* k, const float* g, const float* v, const float* beta,
+                                    const float* scales, float* state, float* out, int tokens, int heads, int kv_heads, int dim, int vdim, int delta,
                                     void* stream) {
     QD_CHECK_ARG(q && k && g && v && state && out && tokens > 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && vdim > 0);
-    QD_CHECK_ARG(!delta || (beta && kq));
+    QD_CHECK_ARG(!delta || (beta && scales));
     const int vectors = dim % 4 == 0 && vdim % 4 == 0 && qd::aligned16(q) && qd::aligned16(k) && qd::aligned16(g) && qd::aligned16(v);
-    const qd::RecurrenceParams p = {q, k, g, v, beta, kq, state, out, tokens, heads, kv_heads, dim, vdim, vectors};
+    const qd::RecurrenceParams p = {q, k, g, v, beta, scales, state, out, tokens, heads, kv_heads, dim, vdim, vectors};
     return delta ? qd::recurrence<true>(p, (cudaStream_t)stream) : qd::recurrence<false>(p, (cudaStream_t)stream);
 }
 

@@ -299,43 +299,51 @@ __global__ void __launch_bounds__(WARPS * 32) attn_flash_kernel(const __grid_con
 }
 
 // ------------------------------------------------------------------------------------- decode
-constexpr int kStepKeys = 64, kStepThreads = 256, kPad = 4;
+constexpr int kStepKeys = 64, kStepThreads = 256;
 
 struct AttnStep { AttnParams a; float* partial; unsigned int* counters; int splits; };
 
-template <typename T>
-QD_DEVINL float dot_rows(const float* q, const T* k, int n) {
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    if ((n & 3) == 0) {
-        for (int d = 0; d < n; d += 4) {
-            const float4 a = load4(q + d), b = load4(k + d);
-            acc[0] = fmaf(a.x, b.x, acc[0]); acc[1] = fmaf(a.y, b.y, acc[1]); acc[2] = fmaf(a.z, b.z, acc[2]); acc[3] = fmaf(a.w, b.w, acc[3]);
-        }
-    } else {
-        for (int d = 0; d < n; ++d) acc[d & 3] = fmaf(q[d], load_f(k + d), acc[d & 3]);
-    }
-    return (acc[0] + acc[1]) + (acc[2] + acc[3]);
+// Elements of a shared row of n elements: 16-byte pieces, an odd number of them (rows read side by side
+// then start in different banks).
+template <typename T> __host__ __device__ constexpr int step_row(int n) {
+    const int e = 16 / (int)sizeof(T), pieces = (n + e - 1) / e;
+    return (pieces | 1) * e;
 }
 
+// dots of two query heads (fp32 rows) with one key row; n a multiple of a 16-byte piece where `pieces`
 template <typename T>
-QD_DEVINL void dot_rows2(const float* q0, const float* q1, const T* k, int n, float& d0, float& d1) {
-    if ((n & 3) != 0) { d0 = dot_rows(q0, k, n); d1 = dot_rows(q1, k, n); return; }
-    float a0[4] = {0.f, 0.f, 0.f, 0.f}, a1[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 4
-    for (int d = 0; d < n; d += 4) {
-        const float4 kv = load4(k + d), x = load4(q0 + d), y = load4(q1 + d);
-        a0[0] = fmaf(x.x, kv.x, a0[0]); a0[1] = fmaf(x.y, kv.y, a0[1]); a0[2] = fmaf(x.z, kv.z, a0[2]); a0[3] = fmaf(x.w, kv.w, a0[3]);
-        a1[0] = fmaf(y.x, kv.x, a1[0]); a1[1] = fmaf(y.y, kv.y, a1[1]); a1[2] = fmaf(y.z, kv.z, a1[2]); a1[3] = fmaf(y.w, kv.w, a1[3]);
+QD_DEVINL void dot_rows2(const float* q0, const float* q1, const T* k, int n, bool pieces, float& d0, float& d1) {
+    float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
+    if (pieces) {
+        constexpr int E = 16 / (int)sizeof(T);
+#pragma unroll 2
+        for (int d = 0; d < n; d += E) {
+            float kv[8];
+            if (sizeof(T) == 2) unpack8(*reinterpret_cast<const uint4*>(k + d), kv);
+            else { const float4 x = *reinterpret_cast<const float4*>(k + d); kv[0] = x.x; kv[1] = x.y; kv[2] = x.z; kv[3] = x.w; }
+#pragma unroll
+            for (int i = 0; i < E; i += 4) {
+                const float4 x = load4(q0 + d + i), y = load4(q1 + d + i);
+                a[0] = fmaf(x.x, kv[i], a[0]); a[1] = fmaf(x.y, kv[i + 1], a[1]); a[2] = fmaf(x.z, kv[i + 2], a[2]); a[3] = fmaf(x.w, kv[i + 3], a[3]);
+                b[0] = fmaf(y.x, kv[i], b[0]); b[1] = fmaf(y.y, kv[i + 1], b[1]); b[2] = fmaf(y.z, kv[i + 2], b[2]); b[3] = fmaf(y.w, kv[i + 3], b[3]);
+            }
+        }
+    } else {
+        for (int d = 0; d < n; ++d) {
+            const float kv = load_f(k + d);
+            a[d & 3] = fmaf(q0[d], kv, a[d & 3]);
+            b[d & 3] = fmaf(q1[d], kv, b[d & 3]);
+        }
     }
-    d0 = (a0[0] + a0[1]) + (a0[2] + a0[3]);
-    d1 = (a1[0] + a1[1]) + (a1[2] + a1[3]);
+    d0 = (a[0] + a[1]) + (a[2] + a[3]);
+    d1 = (b[0] + b[1]) + (b[2] + b[3]);
 }
 
 template <typename T>
 static size_t step_smem(int share, int dim, int vdim, int rot) {
-    const int dp = (dim + kPad + 3) / 4 * 4, vp = (vdim + 3) / 4 * 4;
-    return sizeof(float) * ((size_t)share * dp + (size_t)share * vp + share * (kStepKeys + 4) + 8 + rot) +
-           sizeof(T) * ((size_t)(kStepKeys + 1) * dp + (size_t)(kStepKeys + 1) * vp) + 64;
+    const int dp = step_row<float>(dim), vp = step_row<float>(vdim);
+    return sizeof(float) * ((size_t)share * dp + (size_t)share * vp + share * (kStepKeys + 4)) +
+           sizeof(T) * (size_t)(2 * kStepKeys) * (step_row<T>(dim) + step_row<T>(vdim)) + sizeof(float) * (rot + 4);
 }
 
 template <typename T>
@@ -346,83 +354,104 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
     __shared__ float red[33];
     __shared__ bool last;
     const int share = p.heads / p.kv_heads, g = blockIdx.x, split = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int dim = p.dim, vdim = p.vdim, dp = (dim + kPad + 3) / 4 * 4, vp = (vdim + 3) / 4 * 4, half = p.rot / 2;
+    const int dim = p.dim, vdim = p.vdim, dp = step_row<float>(dim), vp = step_row<float>(vdim), half = p.rot / 2;
+    const int krow = step_row<T>(dim), vrow = step_row<T>(vdim);
     float* qs = shared;                                   // [share][dp]
     float* acc = qs + share * dp;                         // [share][vp]
     float* score = acc + share * vp;                      // [share][kStepKeys]
-    float* stat = score + share * kStepKeys;              // m, l, keep per head (four floats)
-    T* ks = reinterpret_cast<T*>(stat + share * 4);       // [kStepKeys + 1][dp]; the last row: the token's own key
-    T* vs = ks + (kStepKeys + 1) * dp;                    // [kStepKeys + 1][vp]
-    float* trig = reinterpret_cast<float*>(vs + (kStepKeys + 1) * vp);
+    float* stat = score + share * kStepKeys;              // maximum, denominator, rescaling factor per head (four floats)
+    T* ks = reinterpret_cast<T*>(stat + share * 4);       // two buffers [kStepKeys][krow]
+    T* vs = ks + 2 * kStepKeys * krow;                    // two buffers [kStepKeys][vrow]
+    float* trig = reinterpret_cast<float*>(vs + 2 * kStepKeys * vrow);
     const int position = p.position_ptr ? *p.position_ptr : p.position, lo = max(0, position - p.window + 1), n = position - lo + 1;
     const int per = max((n + sp.splits - 1) / sp.splits, 32), active = (n + per - 1) / per;
     if (split >= active) return;
     const int first = lo + split * per, end = min(first + per, position + 1);
+    const int qn = p.heads * dim, kn = p.kv_heads * dim, vn = p.kv_heads * vdim;
+    T* kc = reinterpret_cast<T*>(p.k_cache);
+    T* vc = reinterpret_cast<T*>(p.v_cache);
+
+    // a warp per cache row; the token's own row is not in the ring yet
+    constexpr int E = 16 / (int)sizeof(T);
+    const bool pieces = dim % E == 0 && vdim % E == 0;
+    auto stage = [&](int j0) {
+        const int buf = ((j0 - first) / kStepKeys) & 1, count = min(kStepKeys, end - j0);
+        T* kd = ks + buf * kStepKeys * krow;
+        T* vd = vs + buf * kStepKeys * vrow;
+        for (int r = warp; r < count; r += kStepThreads / 32) {
+            const int j = j0 + r;
+            if (j == position) continue;
+            const size_t row = (size_t)(j % p.capacity) * p.kv_heads + g;
+            if (pieces) {
+                const int kp = dim / E, all = kp + vdim / E;
+                for (int i = lane; i < all; i += 32) {
+                    if (i < kp) copy16_or_zero(kd + r * krow + i * E, kc + row * dim + i * E, true);
+                    else copy16_or_zero(vd + r * vrow + (i - kp) * E, vc + row * vdim + (i - kp) * E, true);
+                }
+            } else {
+                for (int d = lane; d < dim; d += 32) kd[r * krow + d] = kc[row * dim + d];
+                for (int d = lane; d < vdim; d += 32) vd[r * vrow + d] = vc[row * vdim + d];
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    stage(first);
 
     const T* q = reinterpret_cast<const T*>(p.q);
     const T* k = reinterpret_cast<const T*>(p.k);
     const T* v = reinterpret_cast<const T*>(p.v) + g * vdim;
-    const int qn = p.heads * dim, kn = p.kv_heads * dim, vn = p.kv_heads * vdim;
     for (int i = tid; i < half; i += kStepThreads) rotation(position, p.freq[i], p.freq[half + i], trig[i], trig[half + i]);
     float qq = 0.f, kk = 0.f;
     for (int i = tid; i < qn; i += kStepThreads) { const float x = load_f(q + i); qq = fmaf(x, x, qq); }
     for (int i = tid; i < kn; i += kStepThreads) { const float x = load_f(k + i); kk = fmaf(x, x, kk); }
     const float qr = 1.0f / sqrtf(block_sum(qq, red) / (float)qn + p.eps), kr = 1.0f / sqrtf(block_sum(kk, red) / (float)kn + p.eps);
-    for (int i = tid; i < share * dim; i += kStepThreads) {
-        const int e = g * share * dim + i;
-        qs[(i / dim) * dp + i % dim] = as_type<T>(rotated(q, p.q_norm, qr, e, i % dim, p.rot, trig, trig + half));
-    }
+    for (int h = warp; h < share; h += kStepThreads / 32)
+        for (int d = lane; d < dim; d += 32)
+            qs[h * dp + d] = as_type<T>(rotated(q, p.q_norm, qr, (g * share + h) * dim + d, d, p.rot, trig, trig + half));
     for (int i = tid; i < share * vp; i += kStepThreads) acc[i] = 0.f;
     for (int i = tid; i < share; i += kStepThreads) { stat[i * 4] = -INFINITY; stat[i * 4 + 1] = 0.f; }
-    T* kc = reinterpret_cast<T*>(p.k_cache);
-    T* vc = reinterpret_cast<T*>(p.v_cache);
-    if (end == position + 1) {                            // this split holds the token itself: its row goes into the ring
+    if (end == position + 1) {                            // this split holds the token itself: into its tile and into the ring
         const size_t slot = position % p.capacity;
+        const int r = (position - first) % kStepKeys, buf = ((position - first) / kStepKeys) & 1;
+        T* kd = ks + (size_t)(buf * kStepKeys + r) * krow;
+        T* vd = vs + (size_t)(buf * kStepKeys + r) * vrow;
         for (int d = tid; d < dim; d += kStepThreads) {
-            store_f(ks + kStepKeys * dp + d, rotated(k, p.k_norm, kr, g * dim + d, d, p.rot, trig, trig + half));
-            kc[slot * kn + g * dim + d] = ks[kStepKeys * dp + d];
+            store_f(kc + slot * kn + g * dim + d, rotated(k, p.k_norm, kr, g * dim + d, d, p.rot, trig, trig + half));
+            if (position - first < kStepKeys * 2) kd[d] = kc[slot * kn + g * dim + d];
         }
-        for (int d = tid; d < vdim; d += kStepThreads) { vs[kStepKeys * vp + d] = v[d]; vc[slot * vn + g * vdim + d] = v[d]; }
+        for (int d = tid; d < vdim; d += kStepThreads) {
+            vc[slot * vn + g * vdim + d] = v[d];
+            if (position - first < kStepKeys * 2) vd[d] = v[d];
+        }
     }
-    __syncthreads();
 
-    const bool quads = (dim & 3) == 0 && (vdim & 3) == 0;
+    const bool quads = (vdim & 3) == 0;
     for (int j0 = first; j0 < end; j0 += kStepKeys) {
-        const int count = min(kStepKeys, end - j0);
-        if (quads) {
-            const int kq = dim / 4, all = kq + vdim / 4;
-            for (int i = tid; i < count * all; i += kStepThreads) {
-                const int r = i / all, piece = i % all, j = j0 + r;
-                const size_t row = (size_t)(j % p.capacity) * p.kv_heads + g;
-                if (piece < kq) store4(ks + r * dp + piece * 4, load4(j == position ? ks + kStepKeys * dp + piece * 4 : kc + row * dim + piece * 4));
-                else {
-                    const int d = (piece - kq) * 4;
-                    store4(vs + r * vp + d, load4(j == position ? vs + kStepKeys * vp + d : vc + row * vdim + d));
-                }
-            }
-        } else {
-            for (int i = tid; i < count * (dim + vdim); i += kStepThreads) {
-                const int r = i / (dim + vdim), d = i % (dim + vdim), j = j0 + r;
-                const size_t row = (size_t)(j % p.capacity) * p.kv_heads + g;
-                if (d < dim) ks[r * dp + d] = j == position ? ks[kStepKeys * dp + d] : kc[row * dim + d];
-                else vs[r * vp + d - dim] = j == position ? vs[kStepKeys * vp + d - dim] : vc[row * vdim + d - dim];
-            }
+        const int buf = ((j0 - first) / kStepKeys) & 1, count = min(kStepKeys, end - j0);
+        T* kt = ks + buf * kStepKeys * krow;
+        T* vt = vs + buf * kStepKeys * vrow;
+        if (j0 + kStepKeys < end) { stage(j0 + kStepKeys); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
+        else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        if (position < j0 + kStepKeys && position >= j0 && position - first >= kStepKeys * 2) {      // its buffer was busy before
+            const size_t slot = position % p.capacity;
+            const int r = position - j0;
+            for (int d = tid; d < dim; d += kStepThreads) kt[r * krow + d] = kc[slot * kn + g * dim + d];
+            for (int d = tid; d < vdim; d += kStepThreads) vt[r * vrow + d] = v[d];
         }
         __syncthreads();
         {       // a thread's key against two heads at a time
             constexpr int kGroups = kStepThreads / kStepKeys;
             const int r = tid % kStepKeys;
             for (int h = tid / kStepKeys; h < share; h += 2 * kGroups) {
-                const int h2 = h + kGroups;
+                const int h2 = min(h + kGroups, share - 1);
                 float d0 = -INFINITY, d1 = -INFINITY;
                 if (r < count) {
-                    if (h2 < share) dot_rows2(qs + h * dp, qs + h2 * dp, ks + r * dp, dim, d0, d1);
-                    else d0 = dot_rows(qs + h * dp, ks + r * dp, dim);
+                    dot_rows2(qs + h * dp, qs + h2 * dp, kt + r * krow, dim, pieces, d0, d1);
                     d0 *= p.scale;
                     d1 *= p.scale;
                 }
                 score[h * kStepKeys + r] = d0;
-                if (h2 < share) score[h2 * kStepKeys + r] = d1;
+                if (h + kGroups < share) score[h2 * kStepKeys + r] = d1;
             }
         }
         __syncthreads();
@@ -450,9 +479,9 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
                 float4 a = load4(acc + h * vp + c);
                 a.x *= keep; a.y *= keep; a.z *= keep; a.w *= keep;
                 const float* w = score + h * kStepKeys;
-#pragma unroll 4
+#pragma unroll 8
                 for (int r = 0; r < count; ++r) {
-                    const float4 v4 = load4(vs + r * vp + c);
+                    const float4 v4 = load4(vt + r * vrow + c);
                     a.x = fmaf(w[r], v4.x, a.x); a.y = fmaf(w[r], v4.y, a.y); a.z = fmaf(w[r], v4.z, a.z); a.w = fmaf(w[r], v4.w, a.w);
                 }
                 store4(acc + h * vp + c, a);
@@ -462,7 +491,7 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
                 const int h = i / vdim, c = i % vdim;
                 float a = acc[h * vp + c] * stat[h * 4 + 2];
                 const float* w = score + h * kStepKeys;
-                for (int r = 0; r < count; ++r) a = fmaf(w[r], load_f(vs + r * vp + c), a);
+                for (int r = 0; r < count; ++r) a = fmaf(w[r], load_f(vt + r * vrow + c), a);
                 acc[h * vp + c] = a;
             }
         }

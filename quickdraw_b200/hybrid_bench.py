@@ -141,7 +141,7 @@ class Cases:
         like_prepare()
         walk_flops = 2.0 * 4 * tokens * heads * d * d
         fp32 = {n: self.rnd(tokens, w, dtype=F32, std=0.05) for n, w in
-                (("q", kv * d), ("k", kv * d), ("v", heads * d), ("beta", heads), ("kq", kv))}
+                (("q", kv * d), ("k", kv * d), ("v", heads * d), ("beta", heads), ("kq", 3 * kv))}
         fp32["g"] = -torch.rand(tokens, heads * d, device=self.device) * 0.1
         rec, raw = self.rnd(heads, d, d, dtype=F32, std=0.1), self.rnd(tokens, heads * d, dtype=F32)
         walk = lambda delta: lambda: call_hybrid("qd_linear_recurrence", ptr(fp32["q"]), ptr(fp32["k"]), ptr(fp32["g"]), ptr(fp32["v"]),

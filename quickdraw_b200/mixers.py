@@ -102,10 +102,10 @@ class LinearRecurrence:
         linear(proj, at["a1"], proj.shape[1], self.w.a2, decay, tokens=tokens, status=status)      # logits; decays in place later
         return (new(tokens, self.kv_heads * m.dim), new(tokens, self.kv_heads * m.dim), decay, new(tokens, m.heads * m.vdim))
 
-    def _walk(self, q, k, decay, v, beta, kq, history, gate, gate_column: int, act: int, dtype):
+    def _walk(self, q, k, decay, v, beta, scales, history, gate, gate_column: int, act: int, dtype):
         m, tokens = self.m, q.shape[0]
         raw = torch.empty((tokens, self.out_columns), dtype=F32, device=q.device)
-        call_hybrid("qd_linear_recurrence", ptr(q), ptr(k), ptr(decay), ptr(v), ptr(beta), ptr(kq), ptr(history.rec), ptr(raw), tokens,
+        call_hybrid("qd_linear_recurrence", ptr(q), ptr(k), ptr(decay), ptr(v), ptr(beta), ptr(scales), ptr(history.rec), ptr(raw), tokens,
                     m.heads, self.kv_heads, m.dim, m.vdim, int(beta is not None), stream_of(q))
         out = torch.empty((tokens, self.out_columns), dtype=dtype, device=q.device)
         call_hybrid("qd_head_norm_gate", ptr(raw), ptr(self.w.norm), column(gate, gate_column), gate.shape[1], ptr(out), tokens, m.heads,
@@ -149,13 +149,13 @@ class ChannelDelta(LinearRecurrence):
         m, tokens, dev = self.m, proj.shape[0], proj.device
         q, k, decay, v = self._operands(proj, at, status)
         beta = torch.empty((tokens, m.heads), dtype=F32, device=dev)
-        kq = torch.empty((tokens, m.kv_heads), dtype=F32, device=dev)
+        scales = torch.empty((tokens, m.kv_heads, 3), dtype=F32, device=dev)
         call_hybrid("qd_channel_delta_prepare", *[column(proj, at[n]) for n in "qkvb"], proj.shape[1], ptr(decay), ptr(self.w.dt_bias),
-                    *self._convolution(history), *place(position), ptr(q), ptr(k), ptr(decay), ptr(v), ptr(beta), ptr(kq), tokens,
+                    *self._convolution(history), *place(position), ptr(q), ptr(k), ptr(decay), ptr(v), ptr(beta), ptr(scales), tokens,
                     m.heads, m.kv_heads, m.dim, m.vdim, DTYPE_CODE[proj.dtype], stream_of(proj))
         gate = torch.empty((tokens, self.out_columns), dtype=proj.dtype, device=dev)
         linear(proj, at["g1"], proj.shape[1], self.w.g2, gate, tokens=tokens, status=status)
-        return self._walk(q, k, decay, v, beta, kq, history, gate, 0, SIGMOID, proj.dtype)
+        return self._walk(q, k, decay, v, beta, scales, history, gate, 0, SIGMOID, proj.dtype)
 
     def step(self, proj, at, history: LayerHistory, position, status):
         m = self.m
