@@ -212,7 +212,7 @@ QD_DEVINL void copy4(void* dst, const void* src) {
 QD_DEVINL void copies_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> QD_DEVINL void copies_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-constexpr int kRecThreads = 128, kRecCols = 32, kRecTile = 16;      // block: four warps x eight columns; tokens per staged tile
+constexpr int kRecCols = 32, kRecTile = 16;      // value columns of a block; tokens per staged tile
 
 struct RecurrenceParams {
     const float* q; const float* k; const float* g; const float* v; const float* beta;
@@ -227,36 +227,70 @@ constexpr int rec_token_floats(int row) { return 3 * row + kRecCols + 4; }
 // A token's vectors, this lane's rows.
 template <int J> struct RecVectors { ulonglong2 q[J], k[J], g[J]; };
 
-// Four tokens' read-outs of CC = KL / 4 columns, summed over the KL lanes of a key group: KL values over KL
-// lanes, so every round exchanges half of what is left and lane kl ends up with value kl (token kl / CC,
-// column kl % CC).
-template <int KL>
-QD_DEVINL float scatter_sum(float (&v)[KL], int kl) {
+// Sums of NV values over the KL lanes of a key group, NV <= KL: a round exchanges half of what is left, lane
+// kl ends up with the sum of value kl / (KL / NV).
+template <int KL, int NV>
+QD_DEVINL float scatter_sum(float (&v)[NV], int kl) {
+    int lanes = KL / 2;
 #pragma unroll
-    for (int x = KL / 2; x >= 1; x >>= 1) {
-        const bool upper = kl & x;
+    for (int n = NV / 2; n >= 1; n >>= 1, lanes >>= 1) {
+        const bool upper = kl & lanes;
 #pragma unroll
-        for (int i = 0; i < x; ++i)
-            v[i] = (upper ? v[i + x] : v[i]) + __shfl_xor_sync(0xffffffffu, upper ? v[i] : v[i + x], x);
+        for (int i = 0; i < n; ++i)
+            v[i] = (upper ? v[i + n] : v[i]) + __shfl_xor_sync(0xffffffffu, upper ? v[i] : v[i + n], lanes);
     }
+#pragma unroll
+    for (; lanes >= 1; lanes >>= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], lanes);
     return v[0];
 }
+// The inverse: v[0] of lane kl is value kl / (KL / NV); every lane gets all values.
+template <int KL, int NV>
+QD_DEVINL void gather_values(float (&v)[NV], int kl) {
+#pragma unroll
+    for (int n = 1; n < NV; n <<= 1) {
+        const int lanes = KL / NV * n;
+        const bool upper = kl & lanes;
+#pragma unroll
+        for (int i = 0; i < n; ++i) {
+            const float other = __shfl_xor_sync(0xffffffffu, v[i], lanes), own = v[i];
+            v[i] = upper ? other : own;
+            v[i + n] = upper ? own : other;
+        }
+    }
+}
+template <int N> QD_DEVINL void load_columns(const float* p, float (&v)[N]) {
+    if (N % 4 == 0) {
+#pragma unroll
+        for (int i = 0; i < N / 4; ++i) {
+            const float4 x = *reinterpret_cast<const float4*>(p + 4 * i);
+            v[4 * i] = x.x; v[(4 * i + 1) % N] = x.y; v[(4 * i + 2) % N] = x.z; v[(4 * i + 3) % N] = x.w;
+        }
+    } else if (N == 2) {
+        const float2 x = *reinterpret_cast<const float2*>(p);
+        v[0] = x.x; v[1 % N] = x.y;
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = p[i];
+    }
+}
 
-// KL lanes share a column's keys (rows 4 KL j + 4 kl + {0..3}), a lane holds CC = KL / 4 columns: more
-// columns per lane mean fewer shared-memory reads per state element, fewer lanes per column fewer rounds
-// of shuffles in the delta rule's dependent chain.
-template <int KL, int J, bool DELTA>
-__global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __grid_constant__ RecurrenceParams p) {
+// KL lanes share a column's keys (rows 4 KL j + 4 kl + {0..3}), a lane holds CC columns; a warp (32 / KL) CC,
+// a block kRecCols.  GATHER: the delta rule's predictions are summed by scatter and gather (fewer shuffles,
+// more rounds) instead of a butterfly per column.
+template <int KL, int CC> constexpr int rec_threads() { return kRecCols / (32 / KL * CC) * 32; }
+
+template <int KL, int CC, int J, bool DELTA, bool GATHER>
+__global__ void __launch_bounds__(rec_threads<KL, CC>()) linear_recurrence_kernel(const __grid_constant__ RecurrenceParams p) {
     chain_enter();
     extern __shared__ __align__(16) float tiles[];
-    constexpr int CC = KL / 4, kRow = 4 * KL * J, kToken = rec_token_floats(kRow);
+    constexpr int kRow = 4 * KL * J, kToken = rec_token_floats(kRow), kThreads = rec_threads<KL, CC>();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, kl = lane % KL, cl = lane / KL;
     const int head = blockIdx.x, kv = head / (p.heads / p.kv_heads), c0 = blockIdx.y * kRecCols;
-    const int local = warp * 8 + cl * CC, col = c0 + local;
+    const int local = (warp * (32 / KL) + cl) * CC, col = c0 + local;
     const int dim = p.dim, vdim = p.vdim;
     float* state = p.state + (size_t)head * dim * vdim;
 
-    for (int i = tid; i < 2 * kRecTile * kToken; i += kRecThreads) tiles[i] = 0.f;      // padding rows stay zero
+    for (int i = tid; i < 2 * kRecTile * kToken; i += kThreads) tiles[i] = 0.f;      // padding rows stay zero
     u64 s[J][2][CC];
 #pragma unroll
     for (int j = 0; j < J; ++j)
@@ -277,7 +311,7 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
     auto stage = [&](int tile) {
         const int t0 = tile * kRecTile, count = min(kRecTile, p.tokens - t0);
         float* base = tiles + (tile & 1) * kRecTile * kToken;
-        for (int piece = tid; piece < per; piece += kRecThreads) {
+        for (int piece = tid; piece < per; piece += kThreads) {
             const int which = piece / kp, e = (which < 3 ? piece - which * kp : piece - 3 * kp) * unit;
             const float* src;
             float* dst = base + (which < 3 ? which : 3) * kRow + e;
@@ -312,8 +346,7 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
     // one token; o: the read-outs of this lane's rows
     auto advance = [&](const RecVectors<J>& f, const float* token, float* o) {
         float v[CC];
-        if (CC == 2) { const float2 x = *reinterpret_cast<const float2*>(token + 3 * kRow + local); v[0] = x.x; v[1] = x.y; }
-        else { const float4 x = *reinterpret_cast<const float4*>(token + 3 * kRow + local); v[0] = x.x; v[1] = x.y; v[CC - 2] = x.z; v[CC - 1] = x.w; }
+        load_columns<CC>(token + 3 * kRow + local, v);
         u64 oa[CC], ob[CC];
 #pragma unroll
         for (int c = 0; c < CC; ++c) oa[c] = ob[c] = 0ull;
@@ -334,10 +367,15 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
                 }
 #pragma unroll
             for (int c = 0; c < CC; ++c) pred[c] = (lo2(pa[c]) + hi2(pa[c])) + (lo2(pb[c]) + hi2(pb[c]));
+            if (GATHER) {
+                scatter_sum<KL, CC>(pred, kl);
+                gather_values<KL, CC>(pred, kl);
+            } else {
 #pragma unroll
-            for (int x = 1; x < KL; x <<= 1)
+                for (int x = 1; x < KL; x <<= 1)
 #pragma unroll
-                for (int c = 0; c < CC; ++c) pred[c] += __shfl_xor_sync(0xffffffffu, pred[c], x);
+                    for (int c = 0; c < CC; ++c) pred[c] += __shfl_xor_sync(0xffffffffu, pred[c], x);
+            }
 #pragma unroll
             for (int j = 0; j < J; ++j)               // fills the shuffles' latency
 #pragma unroll
@@ -382,9 +420,9 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
         RecVectors<J> even, odd;                     // the next token's vectors are read while this one is reduced
         fetch(token, even);
         for (int tt = 0; tt < count; tt += 4, token += 4 * kToken) {
-            float o[KL];
+            float o[4 * CC];
 #pragma unroll
-            for (int i = 0; i < KL; ++i) o[i] = 0.f;
+            for (int i = 0; i < 4 * CC; ++i) o[i] = 0.f;
             if (tt + 1 < count) fetch(token + kToken, odd);
             advance(even, token, o);
             if (tt + 2 < count) fetch(token + 2 * kToken, even);
@@ -393,9 +431,9 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
             if (tt + 2 < count) advance(even, token + 2 * kToken, o + 2 * CC);
             if (tt + 4 < count) fetch(token + 4 * kToken, even);
             if (tt + 3 < count) advance(odd, token + 3 * kToken, o + 3 * CC);
-            const float mine = scatter_sum<KL>(o, kl);
-            const int t = kl / CC, c = kl % CC;
-            if (tt + t < count && col + c < vdim) out[t * out_stride + col + c] = mine;
+            const float mine = scatter_sum<KL, 4 * CC>(o, kl);
+            const int value = kl / (KL / (4 * CC)), t = value / CC, c = value % CC;
+            if (kl % (KL / (4 * CC)) == 0 && tt + t < count && col + c < vdim) out[t * out_stride + col + c] = mine;
             out += 4 * out_stride;
         }
         __syncthreads();                 // the buffer may be refilled
@@ -414,28 +452,19 @@ __global__ void __launch_bounds__(kRecThreads) linear_recurrence_kernel(const __
             }
 }
 
-template <int KL, int J, bool DELTA>
+template <int KL, int CC, int J, bool DELTA, bool GATHER>
 int launch_recurrence(const RecurrenceParams& p, cudaStream_t stream) {
     const size_t smem = 2ull * kRecTile * rec_token_floats(4 * KL * J) * 4;
-    if (!allow_smem(linear_recurrence_kernel<KL, J, DELTA>, smem)) return QD_ERR_LAUNCH;
-    return qd_launch(linear_recurrence_kernel<KL, J, DELTA>, dim3(p.heads, (p.vdim + kRecCols - 1) / kRecCols), dim3(kRecThreads), smem,
-                     stream, 1, p);
+    if (!allow_smem(linear_recurrence_kernel<KL, CC, J, DELTA, GATHER>, smem)) return QD_ERR_LAUNCH;
+    return qd_launch(linear_recurrence_kernel<KL, CC, J, DELTA, GATHER>, dim3(p.heads, (p.vdim + kRecCols - 1) / kRecCols),
+                     dim3(rec_threads<KL, CC>()), smem, stream, 1, p);
 }
 template <bool DELTA>
 int recurrence(const RecurrenceParams& p, cudaStream_t stream) {
-    if (DELTA) {
-        if (p.dim <= 32) return launch_recurrence<8, 1, true>(p, stream);
-        if (p.dim <= 64) return launch_recurrence<8, 2, true>(p, stream);
-        if (p.dim <= 96) return launch_recurrence<8, 3, true>(p, stream);
-        if (p.dim <= 128) return launch_recurrence<8, 4, true>(p, stream);
-        if (p.dim <= 192) return launch_recurrence<16, 3, true>(p, stream);
-        if (p.dim <= 256) return launch_recurrence<16, 4, true>(p, stream);
-        return QD_ERR_UNSUPPORTED;
-    }
-    if (p.dim <= 64) return launch_recurrence<16, 1, false>(p, stream);
-    if (p.dim <= 128) return launch_recurrence<16, 2, false>(p, stream);
-    if (p.dim <= 192) return launch_recurrence<16, 3, false>(p, stream);
-    if (p.dim <= 256) return launch_recurrence<16, 4, false>(p, stream);
+    if (p.dim <= 64) return launch_recurrence<16, 2, 1, DELTA, false>(p, stream);
+    if (p.dim <= 128) return launch_recurrence<16, 2, 2, DELTA, false>(p, stream);
+    if (p.dim <= 192) return launch_recurrence<16, 2, 3, DELTA, false>(p, stream);
+    if (p.dim <= 256) return launch_recurrence<16, 2, 4, DELTA, false>(p, stream);
     return QD_ERR_UNSUPPORTED;
 }
 
