@@ -97,7 +97,7 @@ int qd_window_attention(const void* q, const void* k, const void* v, const void*
     void* v_cache, int capacity, int window, const int* position_ptr, int position, void* q_scratch, void* out, int
     tokens, int heads, int kv_heads, int dim, int vdim, int dtype, void* stream);
 
-/* Floats of `partial` below (8-byte aligned). */
+/* Floats of `partial` below (16-byte aligned). */
 long long qd_window_attention_step_floats(int heads, int vdim, int splits);
 
 /* The same for one token in one launch; counters: kv_heads words, zero before the first call.

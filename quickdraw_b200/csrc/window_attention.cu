@@ -302,6 +302,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_flash_kernel(const __grid_con
 constexpr int kStepKeys = 64, kStepThreads = 256;
 
 struct AttnStep { AttnParams a; float* partial; unsigned int* counters; int splits; };
+__host__ __device__ constexpr size_t step_stats_floats(int heads, int splits) { return (2 * (size_t)heads * splits + 3) / 4 * 4; }
 
 // Elements of a shared row of n elements: 16-byte pieces, an odd number of them (rows read side by side
 // then start in different banks).
@@ -501,7 +502,7 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
     // partial results: (maximum, denominator) [head][split], then sums [head][split][vdim]; the last split of this
     // key/value head to arrive merges them
     float2* stats = reinterpret_cast<float2*>(sp.partial) + (size_t)g * share * sp.splits;
-    float* sums = sp.partial + 2 * (size_t)p.heads * sp.splits + (size_t)g * share * sp.splits * vdim;
+    float* sums = sp.partial + step_stats_floats(p.heads, sp.splits) + (size_t)g * share * sp.splits * vdim;
     for (int i = tid; i < share * vdim; i += kStepThreads) {
         const int h = i / vdim, c = i % vdim;
         sums[((size_t)h * sp.splits + split) * vdim + c] = acc[h * vp + c];
@@ -534,13 +535,27 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
         for (int i = 0; i < kStepKeys / 32; ++i) score[h * kStepKeys + i * 32 + lane] = mine[i].x * f;
     }
     __syncthreads();
-    for (int i = tid; i < share * vdim; i += kStepThreads) {
-        const int h = i / vdim, c = i % vdim;
-        const float* rows = sums + (size_t)h * sp.splits * vdim + c;
-        float o = 0.f;
-#pragma unroll 8
-        for (int s = 0; s < active; ++s) o = fmaf(__ldcg(rows + (size_t)s * vdim), score[h * kStepKeys + s], o);
-        store_f(reinterpret_cast<T*>(p.out) + (g * share + h) * vdim + c, o);
+    T* out = reinterpret_cast<T*>(p.out) + (size_t)g * share * vdim;
+    if (quads) {
+        for (int i = tid; i < share * (vdim / 4); i += kStepThreads) {
+            const int h = i / (vdim / 4), c = i % (vdim / 4) * 4;
+            const float* rows = sums + (size_t)h * sp.splits * vdim + c;
+            float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 16
+            for (int s = 0; s < active; ++s) {
+                const float4 x = __ldcg(reinterpret_cast<const float4*>(rows + (size_t)s * vdim));
+                const float f = score[h * kStepKeys + s];
+                o.x = fmaf(x.x, f, o.x); o.y = fmaf(x.y, f, o.y); o.z = fmaf(x.z, f, o.z); o.w = fmaf(x.w, f, o.w);
+            }
+            store4(out + h * vdim + c, o);
+        }
+    } else {
+        for (int i = tid; i < share * vdim; i += kStepThreads) {
+            const int h = i / vdim, c = i % vdim;
+            float o = 0.f;
+            for (int s = 0; s < active; ++s) o = fmaf(__ldcg(sums + ((size_t)h * sp.splits + s) * vdim + c), score[h * kStepKeys + s], o);
+            store_f(out + h * vdim + c, o);
+        }
     }
 }
 
@@ -608,14 +623,16 @@ extern "C" int qd_window_attention(const void* q, const void* k, const void* v, 
     return QD_ERR_UNSUPPORTED;
 }
 
-extern "C" long long qd_window_attention_step_floats(int heads, int vdim, int splits) { return (long long)heads * splits * (vdim + 2); }
+extern "C" long long qd_window_attention_step_floats(int heads, int vdim, int splits) {
+    return (long long)qd::step_stats_floats(heads, splits) + (long long)heads * splits * vdim;
+}
 
 extern "C" int qd_window_attention_step(const void* q, const void* k, const void* v, const void* gate, const void* q_norm,
                                         const void* k_norm, const float* freq, int rot, const void* sink, float scale, float eps,
                                         void* k_cache, void* v_cache, int capacity, int window, const int* position_ptr, int position,
                                         float* partial, unsigned int* counters, int splits, void* out, int heads, int kv_heads,
                                         int dim, int vdim, int dtype, void* stream) {
-    QD_ATTN_ARGS_OK(partial && counters && splits > 0 && splits <= qd::kStepKeys);
+    QD_ATTN_ARGS_OK(partial && counters && splits > 0 && splits <= qd::kStepKeys && qd::aligned16(partial));
     const qd::AttnStep sp = {{q, k, v, gate, 0, (const bf16*)q_norm, (const bf16*)k_norm, freq, rot, (const bf16*)sink, scale, eps, k_cache,
                               v_cache, capacity, window, position_ptr, position, nullptr, out, 1, heads, kv_heads, dim, vdim},
                              partial, counters, splits};
