@@ -4,9 +4,9 @@ Exports mirror the reference package (quickdraw/__init__.py:3-23); ``load_checkp
 not part of this package (weights are handed over as ``Checkpoint`` containers).
 """
 
-from .weights import (Checkpoint, FP8Linear, FullAttnWeights, GDNWeights, LayerWeights,
+from .weights import (Checkpoint, FezopelCheckpoint, FezopelConfig, FP8Linear, FullAttnWeights, GDNWeights, LayerWeights,
                       ModelConfig, MoEWeights, NVFP4Linear)
-from .state import DecodeState
+from .state import DecodeState, HybridState
 
 
 def __getattr__(name):
@@ -22,4 +22,5 @@ def __getattr__(name):
 
 
 __all__ = ["ModelConfig", "Checkpoint", "FP8Linear", "NVFP4Linear", "Engine", "DecodeState",
-           "bind_kernels", "GDNWeights", "FullAttnWeights", "MoEWeights", "LayerWeights"]
+           "bind_kernels", "GDNWeights", "FullAttnWeights", "MoEWeights", "LayerWeights",
+           "FezopelConfig", "FezopelCheckpoint", "HybridState"]

@@ -301,7 +301,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_flash_kernel(const __grid_con
 // ------------------------------------------------------------------------------------- decode
 constexpr int kStepKeys = 64, kStepThreads = 256;
 
-struct AttnStep { AttnParams a; float* partial; unsigned int* counters; int splits; };
+struct AttnStep { AttnParams a; float* partial; unsigned int* counters; int splits, buffers; };      // buffers: key tiles in shared memory, 1 or 2
 __host__ __device__ constexpr size_t step_stats_floats(int heads, int splits) { return (2 * (size_t)heads * splits + 3) / 4 * 4; }
 
 // Elements of a shared row of n elements: 16-byte pieces, an odd number of them (rows read side by side
@@ -341,10 +341,10 @@ QD_DEVINL void dot_rows2(const float* q0, const float* q1, const T* k, int n, bo
 }
 
 template <typename T>
-static size_t step_smem(int share, int dim, int vdim, int rot) {
+static size_t step_smem(int share, int dim, int vdim, int rot, int buffers) {
     const int dp = step_row<float>(dim), vp = step_row<float>(vdim);
     return sizeof(float) * ((size_t)share * dp + (size_t)share * vp + share * (kStepKeys + 4)) +
-           sizeof(T) * (size_t)(2 * kStepKeys) * (step_row<T>(dim) + step_row<T>(vdim)) + sizeof(float) * (rot + 4);
+           sizeof(T) * (size_t)(buffers * kStepKeys) * (step_row<T>(dim) + step_row<T>(vdim)) + sizeof(float) * (rot + 4);
 }
 
 template <typename T>
@@ -361,9 +361,9 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
     float* acc = qs + share * dp;                         // [share][vp]
     float* score = acc + share * vp;                      // [share][kStepKeys]
     float* stat = score + share * kStepKeys;              // maximum, denominator, rescaling factor per head (four floats)
-    T* ks = reinterpret_cast<T*>(stat + share * 4);       // two buffers [kStepKeys][krow]
-    T* vs = ks + 2 * kStepKeys * krow;                    // two buffers [kStepKeys][vrow]
-    float* trig = reinterpret_cast<float*>(vs + 2 * kStepKeys * vrow);
+    T* ks = reinterpret_cast<T*>(stat + share * 4);       // buffers of [kStepKeys][krow]
+    T* vs = ks + sp.buffers * kStepKeys * krow;           // buffers of [kStepKeys][vrow]
+    float* trig = reinterpret_cast<float*>(vs + sp.buffers * kStepKeys * vrow);
     const int position = p.position_ptr ? *p.position_ptr : p.position, lo = max(0, position - p.window + 1), n = position - lo + 1;
     const int per = max((n + sp.splits - 1) / sp.splits, 32), active = (n + per - 1) / per;
     if (split >= active) return;
@@ -376,7 +376,7 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
     constexpr int E = 16 / (int)sizeof(T);
     const bool pieces = dim % E == 0 && vdim % E == 0;
     auto stage = [&](int j0) {
-        const int buf = ((j0 - first) / kStepKeys) & 1, count = min(kStepKeys, end - j0);
+        const int buf = ((j0 - first) / kStepKeys) & (sp.buffers - 1), count = min(kStepKeys, end - j0);
         T* kd = ks + buf * kStepKeys * krow;
         T* vd = vs + buf * kStepKeys * vrow;
         for (int r = warp; r < count; r += kStepThreads / 32) {
@@ -413,27 +413,27 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
     for (int i = tid; i < share; i += kStepThreads) { stat[i * 4] = -INFINITY; stat[i * 4 + 1] = 0.f; }
     if (end == position + 1) {                            // this split holds the token itself: into its tile and into the ring
         const size_t slot = position % p.capacity;
-        const int r = (position - first) % kStepKeys, buf = ((position - first) / kStepKeys) & 1;
+        const int r = (position - first) % kStepKeys, buf = ((position - first) / kStepKeys) & (sp.buffers - 1);
         T* kd = ks + (size_t)(buf * kStepKeys + r) * krow;
         T* vd = vs + (size_t)(buf * kStepKeys + r) * vrow;
         for (int d = tid; d < dim; d += kStepThreads) {
             store_f(kc + slot * kn + g * dim + d, rotated(k, p.k_norm, kr, g * dim + d, d, p.rot, trig, trig + half));
-            if (position - first < kStepKeys * 2) kd[d] = kc[slot * kn + g * dim + d];
+            if (position - first < kStepKeys * sp.buffers) kd[d] = kc[slot * kn + g * dim + d];
         }
         for (int d = tid; d < vdim; d += kStepThreads) {
             vc[slot * vn + g * vdim + d] = v[d];
-            if (position - first < kStepKeys * 2) vd[d] = v[d];
+            if (position - first < kStepKeys * sp.buffers) vd[d] = v[d];
         }
     }
 
     const bool quads = (vdim & 3) == 0;
     for (int j0 = first; j0 < end; j0 += kStepKeys) {
-        const int buf = ((j0 - first) / kStepKeys) & 1, count = min(kStepKeys, end - j0);
+        const int buf = ((j0 - first) / kStepKeys) & (sp.buffers - 1), count = min(kStepKeys, end - j0);
         T* kt = ks + buf * kStepKeys * krow;
         T* vt = vs + buf * kStepKeys * vrow;
-        if (j0 + kStepKeys < end) { stage(j0 + kStepKeys); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
+        if (sp.buffers == 2 && j0 + kStepKeys < end) { stage(j0 + kStepKeys); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
         else asm volatile("cp.async.wait_group 0;" ::: "memory");
-        if (position < j0 + kStepKeys && position >= j0 && position - first >= kStepKeys * 2) {      // its buffer was busy before
+        if (position < j0 + kStepKeys && position >= j0 && position - first >= kStepKeys * sp.buffers) {      // its buffer was busy before
             const size_t slot = position % p.capacity;
             const int r = position - j0;
             for (int d = tid; d < dim; d += kStepThreads) kt[r * krow + d] = kc[slot * kn + g * dim + d];
@@ -497,6 +497,7 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
             }
         }
         __syncthreads();
+        if (sp.buffers == 1 && j0 + kStepKeys < end) stage(j0 + kStepKeys);
     }
 
     // partial results: (maximum, denominator) [head][split], then sums [head][split][vdim]; the last split of this
@@ -593,10 +594,12 @@ int chunk(const AttnParams& p, cudaStream_t s) {
     return qd_launch(attn_rows_kernel<T>, dim3((unsigned)(((long long)p.tokens * p.heads + 7) / 8)), dim3(256), 0, s, 1, p);
 }
 template <typename T>
-int step(const AttnStep& sp, cudaStream_t s) {
-    const size_t smem = step_smem<T>(sp.a.heads / sp.a.kv_heads, sp.a.dim, sp.a.vdim, sp.a.rot);
-    if (!allow_smem(attn_step_kernel<T>, smem)) return QD_ERR_UNSUPPORTED;
-    return qd_launch(attn_step_kernel<T>, dim3(sp.a.kv_heads, sp.splits), dim3(kStepThreads), smem, s, 1, sp);
+int step(AttnStep sp, cudaStream_t s) {
+    const auto smem = [&] { return step_smem<T>(sp.a.heads / sp.a.kv_heads, sp.a.dim, sp.a.vdim, sp.a.rot, sp.buffers); };
+    sp.buffers = 2;
+    if (smem() > 220 * 1024) sp.buffers = 1;
+    if (!allow_smem(attn_step_kernel<T>, smem())) return QD_ERR_UNSUPPORTED;
+    return qd_launch(attn_step_kernel<T>, dim3(sp.a.kv_heads, sp.splits), dim3(kStepThreads), smem(), s, 1, sp);
 }
 
 }  // namespace
@@ -635,7 +638,7 @@ extern "C" int qd_window_attention_step(const void* q, const void* k, const void
     QD_ATTN_ARGS_OK(partial && counters && splits > 0 && splits <= qd::kStepKeys && qd::aligned16(partial));
     const qd::AttnStep sp = {{q, k, v, gate, 0, (const bf16*)q_norm, (const bf16*)k_norm, freq, rot, (const bf16*)sink, scale, eps, k_cache,
                               v_cache, capacity, window, position_ptr, position, nullptr, out, 1, heads, kv_heads, dim, vdim},
-                             partial, counters, splits};
+                             partial, counters, splits, 2};
     if (dtype == QD_BF16) return qd::step<bf16>(sp, (cudaStream_t)stream);
     if (dtype == QD_F32) return qd::step<float>(sp, (cudaStream_t)stream);
     return QD_ERR_UNSUPPORTED;

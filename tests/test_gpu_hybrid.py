@@ -167,6 +167,7 @@ ATTENTIONS = {
     "shared heads": cases.attention(), "one kv head": cases.attention(heads=5, kv_heads=1, dim=32, vdim=16, window=33, rotary_dims=32),
     "own heads": cases.attention(heads=3, kv_heads=3, dim=16, vdim=64, window=7, rotary_dims=4), "window of one": cases.attention(window=1),
     "window beyond the prompt": cases.attention(window=1000, scale=-0.2), "wide": cases.attention(heads=2, kv_heads=1, dim=136, vdim=200, window=64),
+    "widest": cases.attention(heads=3, kv_heads=1, dim=256, vdim=256, window=200, rotary_dims=256),
     "no vectors": cases.attention(heads=3, kv_heads=3, dim=14, vdim=9, window=11, rotary_dims=6), "tile edges": cases.attention(window=64, heads=4, kv_heads=4),
 }
 
@@ -191,6 +192,23 @@ def test_window_attention(M, name, cut, dtype):
                            v=torch.full((capacity, m.kv_heads, m.vdim), float("nan"), dtype=dtype, device="cuda"))
     got = drive(mixer, proj.cuda(), at, history, cuts)
     assert error(got, exact) < (5e-5 if dtype == F32 else 2e-2)
+
+
+@pytest.mark.parametrize("splits", [1, 2, 5])
+@pytest.mark.parametrize("name", ["widest", "wide", "window beyond the prompt", "no vectors"])
+@pytest.mark.parametrize("dtype", [F32, BF16])
+def test_decoding_with_long_splits(M, name, splits, dtype):
+    """Splits of several key tiles (a large window has them), with one and with two tile buffers in shared memory."""
+    m, tokens = ATTENTIONS[name], 230
+    w, eps, proj, at, want = attention_case(m, tokens, dtype, sharp=3.0)
+    weights = WindowAttnWeights(**{k: None if v is None else v.cuda() for k, v in vars(w).items()})
+    mixer = M.WindowAttention(weights, m, eps, torch.device("cuda"))
+    mixer.splits = min(splits, mixer.splits)
+    capacity = min(tokens, m.window - 1 + 60)
+    history = LayerHistory(k=torch.empty(capacity, m.kv_heads, m.dim, dtype=dtype, device="cuda"),
+                           v=torch.empty(capacity, m.kv_heads, m.vdim, dtype=dtype, device="cuda"))
+    got = drive(mixer, proj.cuda(), at, history, [60, 60, 60] + [1] * 50)
+    assert error(got[180:], want()[180:]) < (5e-5 if dtype == F32 else 2e-2)
 
 
 @pytest.mark.parametrize("inside", [True, False])
