@@ -537,6 +537,39 @@ QD_DEVINL void prefetch_span(const void* p, size_t bytes) {
         asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(p) + at));
 }
 
+// One channel's convolution for a single token: up to four taps have all their inputs and weights requested at
+// once, before the position (which selects the ring rows) has arrived; more taps are walked.
+constexpr int kStepTaps = 4;
+template <typename T> struct StepConv {
+    float x, ring[kStepTaps], w[kStepTaps];
+    QD_DEVINL void request(const T* fresh, const bf16* taps, const ConvSource& src, int channel) {
+        x = load_f(fresh);
+#pragma unroll
+        for (int r = 0; r < kStepTaps; ++r) {
+            ring[r] = w[r] = 0.f;
+            if (src.taps <= kStepTaps && r < src.taps) {
+                ring[r] = load_f(reinterpret_cast<const T*>(src.history) + (size_t)r * src.channels + channel);
+                w[r] = ld_bf16(taps + src.taps - 1 - r);          // w[back]
+            }
+        }
+    }
+    QD_DEVINL float finish(const T* fresh, int position, const bf16* taps, const ConvSource& src, int channel) {
+        if (src.taps > kStepTaps) return conv_at(fresh, 0, 0, position, taps, src, channel);
+        float acc = 0.f;
+#pragma unroll
+        for (int back = kStepTaps - 1; back >= 1; --back) {
+            if (back < src.taps && position >= back) {
+                const int row = (position - back) % src.taps;
+                float v = ring[0];
+#pragma unroll
+                for (int r = 1; r < kStepTaps; ++r) v = row == r ? ring[r] : v;
+                acc = fmaf(v, w[back], acc);
+            }
+        }
+        return fmaf(x, w[0], acc);
+    }
+};
+
 template <typename T, bool DELTA, int KPT>
 __global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const __grid_constant__ StepParams p) {
     const int head = blockIdx.y, c0 = blockIdx.x * 32, tid = threadIdx.x, col = tid & 31, kg = tid >> 5;
@@ -563,22 +596,27 @@ __global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const __g
     const float scale = 1.0f / sqrtf((float)dim);
     float qv = 0.f, kvv = 0.f, beta = 0.f, rate = 0.f;
     if (DELTA) {
-        const int position = p.position_ptr ? *p.position_ptr : p.position;
         const ConvSource src = {p.history, p.taps, 2 * kv_keys + p.heads * vdim};
-        T* fresh = reinterpret_cast<T*>(p.history) + (size_t)(position % p.taps) * src.channels;
+        const int kc = kv * dim + tid, vch = head * vdim + c0 + col;
+        const bf16* qt = p.q_taps + (size_t)kc * p.taps;
+        const bf16* kt = p.k_taps + (size_t)kc * p.taps;
+        const bf16* vt = p.v_taps + (size_t)vch * p.taps;
+        const bool keyed = tid < dim, valued = kg == kStepGroups - 1 && col_ok;
+        StepConv<T> cq, ck, cv;
+        const int position = p.position_ptr ? *p.position_ptr : p.position;
+        if (keyed) { cq.request(q + tid, qt, src, kc); ck.request(k + tid, kt, src, kv_keys + kc); }
+        if (valued) cv.request(v + col, vt, src, 2 * kv_keys + vch);
         beta = sigmoid_precise(load_f(reinterpret_cast<const T*>(p.beta) + head));
         rate = expf(ld_bf16(p.a_log + head));
-        if (tid < dim) {
-            const int c = kv * dim + tid;
-            qv = silu_precise(conv_at(q + tid, 0, 0, position, p.q_taps + (size_t)c * p.taps, src, c));
-            kvv = silu_precise(conv_at(k + tid, 0, 0, position, p.k_taps + (size_t)c * p.taps, src, kv_keys + c));
-            if (blockIdx.x == 0 && head % (p.heads / p.kv_heads) == 0) { fresh[c] = q[tid]; fresh[kv_keys + c] = k[tid]; }
+        T* fresh = reinterpret_cast<T*>(p.history) + (size_t)(position % p.taps) * src.channels;
+        if (keyed) {
+            qv = silu_precise(cq.finish(q + tid, position, qt, src, kc));
+            kvv = silu_precise(ck.finish(k + tid, position, kt, src, kv_keys + kc));
         }
-        if (kg == kStepGroups - 1 && col_ok) {
-            const int c = head * vdim + c0 + col;
-            sv[col] = silu_precise(conv_at(v + col, 0, 0, position, p.v_taps + (size_t)c * p.taps, src, 2 * kv_keys + c));
-            fresh[2 * kv_keys + c] = v[col];
-        }
+        if (valued) sv[col] = silu_precise(cv.finish(v + col, position, vt, src, 2 * kv_keys + vch));
+        // the token's row of the ring: requested above by other blocks too, used by none of them
+        if (keyed && blockIdx.x == 0 && head % (p.heads / p.kv_heads) == 0) { fresh[kc] = q[tid]; fresh[kv_keys + kc] = k[tid]; }
+        if (valued) fresh[2 * kv_keys + vch] = v[col];
         const float qq = warp_sum(qv * qv), kk = warp_sum(kvv * kvv);
         if (col == 0) { norms[0][kg] = qq; norms[1][kg] = kk; }
     } else {
