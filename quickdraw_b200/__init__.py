@@ -4,8 +4,8 @@ Exports mirror the reference package (quickdraw/__init__.py:3-23); ``load_checkp
 not part of this package (weights are handed over as ``Checkpoint`` containers).
 """
 
-from .weights import (Checkpoint, FezopelCheckpoint, FezopelConfig, FP8Linear, FullAttnWeights, GDNWeights, LayerWeights,
-                      ModelConfig, MoEWeights, NVFP4Linear)
+from .weights import (Checkpoint, DokulixCheckpoint, DokulixConfig, FezopelCheckpoint, FezopelConfig, FP8Linear, FullAttnWeights,
+                      GDNWeights, LayerWeights, ModelConfig, MoEWeights, NVFP4Linear)
 from .state import DecodeState, HybridState
 
 
@@ -23,4 +23,4 @@ def __getattr__(name):
 
 __all__ = ["ModelConfig", "Checkpoint", "FP8Linear", "NVFP4Linear", "Engine", "DecodeState",
            "bind_kernels", "GDNWeights", "FullAttnWeights", "MoEWeights", "LayerWeights",
-           "FezopelConfig", "FezopelCheckpoint", "HybridState"]
+           "FezopelConfig", "FezopelCheckpoint", "DokulixConfig", "DokulixCheckpoint", "HybridState"]

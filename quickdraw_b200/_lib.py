@@ -1,5 +1,6 @@
 """ctypes binding of ``libquickdraw_b200.so`` (declarations: ``include/quickdraw_b200.h``) and of
-``libquickdraw_b200_hybrid.so`` (``include/quickdraw_b200_hybrid.h``), the kernels of the bf16-weight models.
+the libraries of the bf16-weight models (``include/quickdraw_b200_hybrid.h``): ``_hybrid`` with what all of them use,
+``_recurrent`` and ``_latent`` with the mixers that only some of them have.
 
 Each library is the only execution path of this package: if it cannot be loaded the
 import of any operator raises, there is no PyTorch or CPU fallback.
@@ -14,7 +15,6 @@ from pathlib import Path
 import torch
 
 LIB_PATH = Path(__file__).resolve().parent / "libquickdraw_b200.so"
-HYBRID_PATH = Path(__file__).resolve().parent / "libquickdraw_b200_hybrid.so"
 
 P, I, F, L = c_void_p, c_int, c_float, c_longlong
 
@@ -80,32 +80,59 @@ SIGNATURES = {
     "qd_seq_moe_combine_norm": [P, P, P, P, P, P, P, P, I, I, I, F, P],
 }
 
-# entry points of the second library (declarations: ``include/quickdraw_b200_hybrid.h``)
-HYBRID_SIGNATURES = {
-    "qd_set_chained_launches": [I],
-    "qd_linear": [P, L, I, P, P, L, I, I, I, I, I, P, P],
-    "qd_greedy": [P, I, P, P, P, P],
-    "qd_embed_norm": [P, P, I, P, P, P, P, I, I, F, I, P],
-    "qd_layer_norm_rows": [P, P, P, P, P, I, I, F, I, P],
-    "qd_sublayer_close": [P, P, L, P, P, P, P, P, P, L, P, I, P, P, P, I, I, F, I, P],
-    "qd_gla_prepare": [P, P, P, L, P, P, F, P, P, P, P, I, I, I, I, I, P],
-    "qd_channel_delta_prepare": [P, P, P, P, L, P, P, P, P, P, P, P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, I, P],
-    "qd_linear_recurrence": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
-    "qd_head_norm_gate": [P, P, P, L, P, I, I, I, F, I, I, P],
-    "qd_gla_step": [P, P, P, P, P, P, I, F, P, P, F, P, P, I, I, I, I, P],
-    "qd_channel_delta_step": [P, P, P, P, P, P, P, I, P, P, P, P, P, I, P, I, P, P, I, P, F, P, P, I, I, I, I, I, P],
-    "qd_window_attention": [P, P, P, P, L, P, P, P, I, P, F, F, P, P, I, I, P, I, P, P, I, I, I, I, I, I, P],
-    "qd_window_attention_step_floats": [I, I, I],
-    "qd_window_attention_step": [P, P, P, P, P, P, P, I, P, F, F, P, P, I, I, P, I, P, P, I, P, I, I, I, I, I, P],
+# entry points of the bf16-weight models by library (declarations: ``include/quickdraw_b200_hybrid.h``)
+HYBRID_LIBRARIES = {
+    "hybrid": {
+        "qd_set_chained_launches": [I],
+        "qd_linear": [P, L, I, P, P, L, I, I, I, I, I, I, P, I, P, F, F, P, P],
+        "qd_greedy": [P, I, P, P, P, P],
+        "qd_embed_norm": [P, P, I, P, P, P, P, I, I, F, I, P],
+        "qd_layer_norm_rows": [P, P, P, P, P, I, I, F, I, P],
+        "qd_sublayer_close": [P, P, L, P, P, P, P, P, P, L, P, I, P, P, P, I, I, F, I, P],
+        "qd_stream_norm": [P, P, I, P, P, P, P, P, P, F, P, I, I, F, I, P],
+        "qd_attention": [P, P],
+        "qd_attention_step_floats": [I, I, I],
+        "qd_attention_step": [P, P],
+    },
+    "recurrent": {
+        "qd_gla_prepare": [P, P, P, L, P, P, F, P, P, P, P, I, I, I, I, I, P],
+        "qd_channel_delta_prepare": [P, P, P, P, L, P, P, P, P, P, P, P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, I, P],
+        "qd_linear_recurrence": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, P],
+        "qd_head_norm_gate": [P, P, P, L, P, I, I, I, F, I, I, P],
+        "qd_gla_step": [P, P, P, P, P, P, I, F, P, P, F, P, P, I, I, I, I, P],
+        "qd_channel_delta_step": [P, P, P, P, P, P, P, I, P, P, P, P, P, I, P, I, P, P, I, P, F, P, P, I, I, I, I, I, P],
+    },
+    "latent": {
+        "qd_latent_prepare": [P, P],
+        "qd_rotate_half": [P, P, P, I, I, I, I, I, I, P],
+        "qd_latent_step_floats": [I, I, I],
+        "qd_latent_step": [P, P],
+    },
 }
-HYBRID_LONG_RESULTS = {"qd_window_attention_step_floats"}
+HYBRID_LONG_RESULTS = {"qd_attention_step_floats", "qd_latent_step_floats"}
+HYBRID_OWNER = {name: target for target, names in HYBRID_LIBRARIES.items() for name in names}
+
+
+def _structure(name: str, *kinds) -> type:
+    """A ctypes structure from (type, field names) pairs."""
+    return type(name, (ctypes.Structure,), {"_fields_": [(field, kind) for kind, names in kinds for field in names.split()]})
+
+
+AttentionArgs = _structure(
+    "AttentionArgs", (P, "q k v gate q_norm k_norm freq sink slopes k_cache v_cache k_shared position_ptr q_rows out partial counters"),
+    (L, "ld ld_gate ld_k ld_v ld_shared"), (F, "scale eps"),
+    (I, "norm rot sink_kind gate_kind mask span capacity position tokens heads kv_heads dim vdim shared_dim splits dtype"))
+LatentArgs = _structure(
+    "LatentArgs", (P, "q dq dkv gate dq_norm dkv_norm freq uk uv cache position_ptr q_latent absorbed partial out"), (L, "ld ld_cache"),
+    (F, "scale eps"), (I, "span capacity position tokens heads dim rot vdim q_rank kv_rank rot_column splits dtype"))
+STRUCTURES = {"qd_attention_args": AttentionArgs, "qd_latent_args": LatentArgs}
 
 LONG_RESULTS = {"qd_decode_workspace_bytes", "qd_program_bytes", "qd_exchange_bytes",
                 "qd_nvfp4_matmul_rows_scratch_bytes", "qd_seq_gdn_chunk_scratch_bytes",
                 "qd_nvfp4_expert_rows_scratch_bytes"}
 
 _lib = None
-_hybrid = None
+_hybrid: dict[str, ctypes.CDLL] = {}
 
 
 class LibraryMissing(RuntimeError):
@@ -137,12 +164,15 @@ def lib() -> ctypes.CDLL:
     return _lib
 
 
-def hybrid_lib() -> ctypes.CDLL:
-    """The library of the bf16-weight models, loaded on first use."""
-    global _hybrid
-    if _hybrid is None:
-        _hybrid = _open(HYBRID_PATH, " hybrid", HYBRID_SIGNATURES, HYBRID_LONG_RESULTS)
-    return _hybrid
+def hybrid_path(target: str) -> Path:
+    return LIB_PATH.with_name(f"libquickdraw_b200_{target}.so")
+
+
+def hybrid_lib(target: str = "hybrid") -> ctypes.CDLL:
+    """A library of the bf16-weight models, loaded on first use."""
+    if target not in _hybrid:
+        _hybrid[target] = _open(hybrid_path(target), f" {target}", HYBRID_LIBRARIES[target], HYBRID_LONG_RESULTS)
+    return _hybrid[target]
 
 
 def exported_symbols() -> list[str]:
@@ -176,6 +206,12 @@ def call(name: str, *args) -> None:
 
 
 def call_hybrid(name: str, *args) -> None:
-    code = getattr(hybrid_lib(), name)(*args)
+    library = hybrid_lib(HYBRID_OWNER[name])
+    code = getattr(library, name)(*args)
     if code != 0:
-        raise RuntimeError(f"{name} failed: {hybrid_lib().qd_error_string(code).decode()} (code {code})")
+        raise RuntimeError(f"{name} failed: {library.qd_error_string(code).decode()} (code {code})")
+
+
+def size_hybrid(name: str, *args) -> int:
+    """The result of an entry point that computes a size."""
+    return getattr(hybrid_lib(HYBRID_OWNER[name]), name)(*args)

@@ -1,9 +1,11 @@
-"""Build the C-ABI CUDA libraries in-tree: ``python -m quickdraw_b200.build [nvfp4|hybrid ...]``.
+"""Build the C-ABI CUDA libraries in-tree: ``python -m quickdraw_b200.build [nvfp4|hybrid|recurrent|latent ...]``.
 
 Plain nvcc, shared objects for sm_100a only, no link against libtorch: the host side passes raw
-device pointers through ctypes.  Two libraries, so that a model only needs its own kernels
-compiled: ``libquickdraw_b200.so`` (NVFP4 / FP8 models) and ``libquickdraw_b200_hybrid.so``
-(bf16-weight models).  Without a name both are built.
+device pointers through ctypes.  Several libraries, so that a model only needs its own kernels
+compiled: ``libquickdraw_b200.so`` (NVFP4 / FP8 models), ``libquickdraw_b200_hybrid.so`` (what all
+bf16-weight models use) and one for each family of mixers that only some of those have,
+``_recurrent`` (gated linear recurrences) and ``_latent`` (latent attention).  Without a name all
+are built.
 """
 
 from __future__ import annotations
@@ -16,36 +18,38 @@ from pathlib import Path
 PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 LIB = PKG / "libquickdraw_b200.so"
-HYBRID = PKG / "libquickdraw_b200_hybrid.so"
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-lineinfo", "-std=c++17",
          "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr"]
 
 COMMON = ("library",)
-HYBRID_SOURCES = ("linear", "residual", "linear_recurrence", "window_attention")
-HYBRID_HEADERS = ("common.cuh", "typed.cuh")
+HYBRID_SOURCES = {"hybrid": ("linear", "residual", "window_attention"), "recurrent": ("linear_recurrence",),
+                  "latent": ("latent_attention",)}
+HYBRID_HEADERS = ("common.cuh", "typed.cuh", "softmax_attention.cuh")
+TARGETS = ("nvfp4", *HYBRID_SOURCES)
 
 
 def sources(target: str) -> list[Path]:
-    if target == "hybrid":
-        return [CSRC / f"{name}.cu" for name in COMMON + HYBRID_SOURCES]
-    return [path for path in sorted(CSRC.glob("*.cu")) if path.stem not in HYBRID_SOURCES]
+    if target in HYBRID_SOURCES:
+        return [CSRC / f"{name}.cu" for name in COMMON + HYBRID_SOURCES[target]]
+    others = {name for names in HYBRID_SOURCES.values() for name in names}
+    return [path for path in sorted(CSRC.glob("*.cu")) if path.stem not in others]
 
 
 def library(target: str) -> Path:
-    return {"nvfp4": LIB, "hybrid": HYBRID}[target]
+    return LIB if target == "nvfp4" else PKG / f"libquickdraw_b200_{target}.so"
 
 
 def stale(target: str = "nvfp4") -> bool:
     lib = library(target)
     if not lib.exists():
         return True
-    headers = ([CSRC / name for name in HYBRID_HEADERS] if target == "hybrid" else sorted(CSRC.glob("*.cuh")))
+    headers = ([CSRC / name for name in HYBRID_HEADERS] if target in HYBRID_SOURCES else sorted(CSRC.glob("*.cuh")))
     headers += sorted((PKG.parent / "include").glob("*.h"))
     return max(p.stat().st_mtime for p in sources(target) + headers) > lib.stat().st_mtime
 
 
-def build(force: bool = False, verbose: bool = False, targets=("nvfp4", "hybrid")) -> list[Path]:
+def build(force: bool = False, verbose: bool = False, targets=TARGETS) -> list[Path]:
     """Compile what is out of date; every source of every requested library in parallel."""
     wanted = [t for t in targets if force or stale(t)]
     build_dir = PKG / "build"
@@ -70,5 +74,5 @@ def build(force: bool = False, verbose: bool = False, targets=("nvfp4", "hybrid"
 
 
 if __name__ == "__main__":
-    names = [a for a in sys.argv[1:] if not a.startswith("-")] or ["nvfp4", "hybrid"]
+    names = [a for a in sys.argv[1:] if not a.startswith("-")] or list(TARGETS)
     print(*build(force="--force" in sys.argv, verbose="-v" in sys.argv, targets=names), sep="\n")

@@ -1,5 +1,7 @@
-// Products with bf16 weights: y[t, n] = sum_k x[t, k] w[n, k], fp32 accumulation, optional exact GELU
-// on the leading columns (the up projection of a feed-forward whose launch also carries other rows).
+// Products with bf16 weights: y[t, n] = sum_k x[t, k] w[n, k], fp32 accumulation.  What may follow in the
+// same launch: a bias, the exact GELU on the leading columns (the up projection of a feed-forward whose
+// launch also carries other rows), a gated linear unit over neighbouring weight rows, the addition to
+// what y already holds (a residual stream).  What may precede it for few token rows: the RMS norm of x.
 // Three forms behind one entry point:
 //   linear_umma_kernel  many token rows, bf16 x: tcgen05.mma kind::f16, both operands by tiled TMA
 //                       (128-byte swizzle), accumulators in tensor memory.  Tensor-bound.
@@ -14,6 +16,17 @@
 namespace qd {
 namespace {
 
+// What follows the sums.  glu: weight rows 2i and 2i + 1 are a gate and its linear partner, y[i] = relu(gate) * partner.
+struct Finish { const float* bias; int gelu_cols; int glu; int add; };
+// RMS norm of x in front of the product: x / rms(x) * (offset + weight); weight == NULL: none.
+struct InputNorm { const bf16* weight; float offset, eps; };
+
+QD_DEVINL float finished(const Finish& f, float v, int n) {
+    if (f.bias) v += f.bias[n];
+    return n < f.gelu_cols ? gelu_erf(v) : v;
+}
+template <typename T> QD_DEVINL void put(T* y, float v, bool add) { store_f(y, add ? load_f(y) + v : v); }
+
 // ------------------------------------------------------------------------------ few token rows
 // Inputs staged at a time.  One weight row per warp (few rows: one or two blocks per SM): up to sixteen 16-byte
 // pieces per lane in flight; two rows per warp: eight, and more blocks.
@@ -22,9 +35,10 @@ constexpr int rows_chunk(int R, int NR) { return NR == 2 ? 1024 : (R <= 2 ? 4096
 template <typename TX, typename TY, int R, int NR>
 __global__ void __launch_bounds__(256)
 linear_rows_kernel(const TX* __restrict__ x, long long ldx, const bf16* __restrict__ w, TY* __restrict__ y,
-                   long long ldy, int tokens, int rows, int width, int gelu_cols) {
+                   long long ldy, int tokens, int rows, int width, const Finish f, const InputNorm norm) {
     constexpr int kRowsChunk = rows_chunk(R, NR);
     __shared__ __align__(16) float xs[R][kRowsChunk];
+    __shared__ float squares[R][8];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int n0 = (blockIdx.x * 8 + warp) * NR;
     constexpr int kPieces = kRowsChunk / 256;
@@ -47,13 +61,23 @@ linear_rows_kernel(const TX* __restrict__ x, long long ldx, const bf16* __restri
     for (int r = 0; r < NR; ++r)
 #pragma unroll
         for (int t = 0; t < R; ++t) acc[r][t] = 0.f;
+    float ss[R];                         // of this thread's inputs, for the norm
+#pragma unroll
+    for (int t = 0; t < R; ++t) ss[t] = 0.f;
     for (int k0 = 0; k0 < width; k0 += kRowsChunk) {
         if (k0) __syncthreads();
-        for (int i = threadIdx.x; i < R * (kRowsChunk / 4); i += 256) {
-            const int t = i / (kRowsChunk / 4), k = (i % (kRowsChunk / 4)) * 4;
-            const float4 v = (t < tokens && k0 + k < width) ? load4(x + t * ldx + k0 + k) : make_float4(0.f, 0.f, 0.f, 0.f);
-            *reinterpret_cast<float4*>(&xs[t][k]) = v;
-        }
+#pragma unroll
+        for (int t = 0; t < R; ++t)
+            for (int k = threadIdx.x * 4; k < kRowsChunk; k += 1024) {
+                const bool ok = t < tokens && k0 + k < width;
+                float4 v = ok ? load4(x + t * ldx + k0 + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+                if (norm.weight && ok) {
+                    const float4 g = load4(norm.weight + k0 + k);
+                    ss[t] = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss[t]))));
+                    v.x *= norm.offset + g.x; v.y *= norm.offset + g.y; v.z *= norm.offset + g.z; v.w *= norm.offset + g.w;
+                }
+                *reinterpret_cast<float4*>(&xs[t][k]) = v;
+            }
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < kPieces; ++i) {
@@ -75,14 +99,37 @@ linear_rows_kernel(const TX* __restrict__ x, long long ldx, const bf16* __restri
         }
         if (k0 + kRowsChunk < width) fetch(k0 + kRowsChunk);
     }
-#pragma unroll
-    for (int r = 0; r < NR; ++r)
+    if (norm.weight) {                   // the same factor for every row: applied to the sums
 #pragma unroll
         for (int t = 0; t < R; ++t) {
-            const float v = warp_sum(acc[r][t]);
-            if (lane == 0 && n0 + r < rows && t < tokens)
-                store_f(y + t * ldy + n0 + r, n0 + r < gelu_cols ? gelu_erf(v) : v);
+            const float part = warp_sum(ss[t]);
+            if (lane == 0) squares[t][warp] = part;
         }
+        __syncthreads();
+#pragma unroll
+        for (int t = 0; t < R; ++t) {
+            float total = 0.f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) total += squares[t][i];
+            const float factor = 1.0f / sqrtf(total / (float)width + norm.eps);
+#pragma unroll
+            for (int r = 0; r < NR; ++r) acc[r][t] *= factor;
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < R; ++t) {
+        float v[NR];
+#pragma unroll
+        for (int r = 0; r < NR; ++r) v[r] = warp_sum(acc[r][t]);
+        if (lane != 0 || t >= tokens) continue;
+        if (NR == 2 && f.glu) {
+            if (n0 < rows) put(y + t * ldy + n0 / 2, fmaxf(finished(f, v[0], n0), 0.f) * finished(f, v[NR - 1], n0 + 1), f.add);
+        } else {
+#pragma unroll
+            for (int r = 0; r < NR; ++r)
+                if (n0 + r < rows) put(y + t * ldy + n0 + r, finished(f, v[r], n0 + r), f.add);
+        }
+    }
 }
 
 // ---------------------------------------------------------------------------------- any shape
@@ -91,7 +138,7 @@ constexpr int kTileT = 64, kTileR = 64, kTileStep = 16;
 template <typename TX, typename TY>
 __global__ void __launch_bounds__(256)
 linear_tile_kernel(const TX* __restrict__ x, long long ldx, const bf16* __restrict__ w, TY* __restrict__ y,
-                   long long ldy, int tokens, int rows, int width, int gelu_cols) {
+                   long long ldy, int tokens, int rows, int width, const Finish f) {
     chain_enter();
     __shared__ __align__(16) float xs[kTileStep][kTileT + 4], ws[kTileStep][kTileR + 4];
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
@@ -126,7 +173,9 @@ linear_tile_kernel(const TX* __restrict__ x, long long ldx, const bf16* __restri
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
-            if (t < tokens && n < rows) store_f(y + t * ldy + n, n < gelu_cols ? gelu_erf(acc[i][j]) : acc[i][j]);
+            if (t >= tokens || n >= rows) continue;
+            if (!f.glu) put(y + t * ldy + n, finished(f, acc[i][j], n), f.add);
+            else if (!(j & 1)) put(y + t * ldy + n / 2, fmaxf(finished(f, acc[i][j], n), 0.f) * finished(f, acc[i][j | 1], n + 1), f.add);
         }
 }
 
@@ -171,7 +220,7 @@ QD_DEVINL void tmem_ld32(uint32_t addr, uint32_t (&v)[32]) {
     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 }
 
-struct LinearParams { void* y; long long ldy; int tokens, rows, width, gelu_cols; unsigned int* status; };
+struct LinearParams { void* y; long long ldy; int tokens, rows, width; Finish f; unsigned int* status; };
 
 template <typename TY, int HALVES, int TN>
 __global__ void __launch_bounds__(UmmaTile<HALVES, TN>::kThreads, UmmaTile<HALVES, TN>::kBlocksPerSm)
@@ -257,7 +306,7 @@ linear_umma_kernel(const __grid_constant__ LinearParams p, const __grid_constant
                 if (n0 + c >= p.rows) break;
                 uint32_t v[32];
                 tmem_ld32(tmem + ((uint32_t)(quadrant * 32) << 16) + half * TN + c, v);
-                const bool gelu = n0 + c < p.gelu_cols;
+                const bool gelu = n0 + c < p.f.gelu_cols;
                 if (t < p.tokens) {
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
@@ -265,9 +314,24 @@ linear_umma_kernel(const __grid_constant__ LinearParams p, const __grid_constant
                         if (n < p.rows) {                // rows is a multiple of eight
                             float f[8];
 #pragma unroll
-                            for (int q = 0; q < 8; ++q) {
-                                f[q] = __uint_as_float(v[j + q]);
-                                if (gelu && n + q < p.gelu_cols) f[q] = gelu_erf(f[q]);
+                            for (int q = 0; q < 8; ++q) f[q] = __uint_as_float(v[j + q]);
+                            if (p.f.bias) {
+                                const float4 a = load4(p.f.bias + n), b = load4(p.f.bias + n + 4);
+                                f[0] += a.x; f[1] += a.y; f[2] += a.z; f[3] += a.w; f[4] += b.x; f[5] += b.y; f[6] += b.z; f[7] += b.w;
+                            }
+                            if (gelu) {
+#pragma unroll
+                                for (int q = 0; q < 8; ++q)
+                                    if (n + q < p.f.gelu_cols) f[q] = gelu_erf(f[q]);
+                            }
+                            if (p.f.glu) {
+                                store4(row + n / 2, make_float4(fmaxf(f[0], 0.f) * f[1], fmaxf(f[2], 0.f) * f[3], fmaxf(f[4], 0.f) * f[5],
+                                                                fmaxf(f[6], 0.f) * f[7]));
+                                continue;
+                            }
+                            if (p.f.add) {
+                                const float4 a = load4(row + n), b = load4(row + n + 4);
+                                f[0] += a.x; f[1] += a.y; f[2] += a.z; f[3] += a.w; f[4] += b.x; f[5] += b.y; f[6] += b.z; f[7] += b.w;
                             }
                             store4(row + n, make_float4(f[0], f[1], f[2], f[3]));
                             store4(row + n + 4, make_float4(f[4], f[5], f[6], f[7]));
@@ -335,32 +399,33 @@ int umma_dispatch(const void* x, long long ldx, const void* w, const LinearParam
 
 template <typename TX, typename TY, int R>
 int launch_rows(const void* x, long long ldx, const void* w, void* y, long long ldy, int tokens, int rows, int width,
-                int gelu_cols, cudaStream_t stream) {
-    // two weight rows per warp once that still gives every SM a few blocks
-    if (rows >= device_sms() * 32)
+                const Finish& f, const InputNorm& norm, cudaStream_t stream) {
+    // two weight rows per warp once that still gives every SM a few blocks, and where pairs of rows belong together
+    if (f.glu || rows >= device_sms() * 32)
         return qd_launch(linear_rows_kernel<TX, TY, R, 2>, dim3((rows + 15) / 16), dim3(256), 0, stream, 2,
-                         (const TX*)x, ldx, (const bf16*)w, (TY*)y, ldy, tokens, rows, width, gelu_cols);
+                         (const TX*)x, ldx, (const bf16*)w, (TY*)y, ldy, tokens, rows, width, f, norm);
     return qd_launch(linear_rows_kernel<TX, TY, R, 1>, dim3((rows + 7) / 8), dim3(256), 0, stream, 2,
-                     (const TX*)x, ldx, (const bf16*)w, (TY*)y, ldy, tokens, rows, width, gelu_cols);
+                     (const TX*)x, ldx, (const bf16*)w, (TY*)y, ldy, tokens, rows, width, f, norm);
 }
 
 template <typename TX, typename TY>
 int dispatch(const void* x, long long ldx, const void* w, void* y, long long ldy, int tokens, int rows, int width,
-             int gelu_cols, unsigned int* status, cudaStream_t stream) {
+             const Finish& f, const InputNorm& norm, unsigned int* status, cudaStream_t stream) {
     const bool vectors = width % 8 == 0 && ldx % 8 == 0 && aligned16(x) && aligned16(w);
-    if (vectors && tokens <= 8) {
-        if (tokens == 1) return launch_rows<TX, TY, 1>(x, ldx, w, y, ldy, tokens, rows, width, gelu_cols, stream);
-        if (tokens == 2) return launch_rows<TX, TY, 2>(x, ldx, w, y, ldy, tokens, rows, width, gelu_cols, stream);
-        if (tokens <= 4) return launch_rows<TX, TY, 4>(x, ldx, w, y, ldy, tokens, rows, width, gelu_cols, stream);
-        return launch_rows<TX, TY, 8>(x, ldx, w, y, ldy, tokens, rows, width, gelu_cols, stream);
+    if (vectors && tokens <= 8 && (!norm.weight || ((uintptr_t)norm.weight & 7u) == 0)) {
+        if (tokens == 1) return launch_rows<TX, TY, 1>(x, ldx, w, y, ldy, tokens, rows, width, f, norm, stream);
+        if (tokens == 2) return launch_rows<TX, TY, 2>(x, ldx, w, y, ldy, tokens, rows, width, f, norm, stream);
+        if (tokens <= 4) return launch_rows<TX, TY, 4>(x, ldx, w, y, ldy, tokens, rows, width, f, norm, stream);
+        return launch_rows<TX, TY, 8>(x, ldx, w, y, ldy, tokens, rows, width, f, norm, stream);
     }
-    if (sizeof(TX) == 2 && vectors && rows % 8 == 0 && ldy % 8 == 0 && aligned16(y)) {
-        const LinearParams p = {y, ldy, tokens, rows, width, gelu_cols, status};
+    if (norm.weight) return QD_ERR_UNSUPPORTED;
+    if (sizeof(TX) == 2 && vectors && rows % 8 == 0 && ldy % 8 == 0 && aligned16(y) && aligned16(f.bias)) {
+        const LinearParams p = {y, ldy, tokens, rows, width, f, status};
         return umma_dispatch<TY>(x, ldx, w, p, stream);
     }
     const dim3 grid((rows + kTileR - 1) / kTileR, (tokens + kTileT - 1) / kTileT);
     return qd_launch(linear_tile_kernel<TX, TY>, grid, dim3(256), 0, stream, 1, (const TX*)x, ldx, (const bf16*)w, (TY*)y,
-                     ldy, tokens, rows, width, gelu_cols);
+                     ldy, tokens, rows, width, f);
 }
 
 // ---------------------------------------------------------------------------- greedy choice
@@ -426,12 +491,17 @@ int launch_greedy(int blocks, const float* logits, int count, unsigned long long
 }  // namespace qd
 
 extern "C" int qd_linear(const void* x, long long ldx, int x_dtype, const void* w, void* y, long long ldy, int y_dtype,
-                         int tokens, int rows, int width, int gelu_cols, unsigned int* status, void* stream) {
-    QD_CHECK_ARG(x && w && y && tokens > 0 && rows > 0 && width > 0 && ldx >= width && ldy >= rows && gelu_cols >= 0);
+                         int tokens, int rows, int width, int gelu_cols, int glu, const float* bias, int add, const void* norm,
+                         float norm_offset, float eps, unsigned int* status, void* stream) {
+    QD_CHECK_ARG(x && w && y && tokens > 0 && rows > 0 && width > 0 && ldx >= width && gelu_cols >= 0);
+    QD_CHECK_ARG(ldy >= (glu ? rows / 2 : rows) && (!glu || (rows % 2 == 0 && gelu_cols == 0 && !add)));
+    const qd::Finish f = {bias, gelu_cols, glu, add};
+    const qd::InputNorm n = {(const bf16*)norm, norm_offset, eps};
     cudaStream_t s = (cudaStream_t)stream;
-    if (x_dtype == QD_BF16 && y_dtype == QD_BF16) return qd::dispatch<bf16, bf16>(x, ldx, w, y, ldy, tokens, rows, width, gelu_cols, status, s);
-    if (x_dtype == QD_BF16 && y_dtype == QD_F32) return qd::dispatch<bf16, float>(x, ldx, w, y, ldy, tokens, rows, width, gelu_cols, status, s);
-    if (x_dtype == QD_F32 && y_dtype == QD_F32) return qd::dispatch<float, float>(x, ldx, w, y, ldy, tokens, rows, width, gelu_cols, status, s);
+    if (x_dtype == QD_BF16 && y_dtype == QD_BF16) return qd::dispatch<bf16, bf16>(x, ldx, w, y, ldy, tokens, rows, width, f, n, status, s);
+    if (x_dtype == QD_BF16 && y_dtype == QD_F32) return qd::dispatch<bf16, float>(x, ldx, w, y, ldy, tokens, rows, width, f, n, status, s);
+    if (x_dtype == QD_F32 && y_dtype == QD_F32) return qd::dispatch<float, float>(x, ldx, w, y, ldy, tokens, rows, width, f, n, status, s);
+    if (x_dtype == QD_F32 && y_dtype == QD_BF16) return qd::dispatch<float, bf16>(x, ldx, w, y, ldy, tokens, rows, width, f, n, status, s);
     return QD_ERR_UNSUPPORTED;
 }
 

@@ -1,7 +1,9 @@
-// The fp32 residual stream between the products: embedding rows, layer norm with weight and bias, the
-// end of a sublayer (sigmoid gate on the sublayer's result, its norm, the residual sum, the weighted
-// average over the embedding output and all layer results so far, the norm in front of the next
-// sublayer) in one launch.  One block per token; a row of the stream lives in shared memory.
+// The fp32 residual stream between the products.  Two styles.  Layer norms around a gated sublayer:
+// embedding rows, layer norm with weight and bias, the end of a sublayer (sigmoid gate on the sublayer's
+// result, its norm, the residual sum, the weighted average over the embedding output and all layer
+// results so far, the norm in front of the next sublayer) in one launch.  RMS norms in front of a
+// sublayer: embedding row or stream row, plus the sublayer's result, plus a vector (that of a pass over
+// looped layers), and the next RMS norm of the sum in one launch (stream_norm).  One block per token; a row of the stream lives in shared memory.
 // HBM-bound (a few bytes per element and operand); at one token bound by the launch and two reductions.
 #include "typed.cuh"
 
@@ -200,6 +202,88 @@ sublayer_close_vec_kernel(const __grid_constant__ CloseParams p) {
     }
 }
 
+struct StreamNorm {
+    const long long* tokens; const bf16* table; int vocab;      // the rows of a table ...
+    const float* x_in; const int* index;                        // ... or rows of the stream (index == NULL: row r)
+    const void* y; const bf16* step;                            // added where given: a row each, one vector for all
+    float* x_out;                                               // where given: the sum
+    const bf16* norm; float offset, eps; void* normed;          // where given: sum / rms(sum) * (offset + norm)
+    int width;
+};
+
+QD_DEVINL size_t source_row(const StreamNorm& p, size_t r) {
+    if (!p.table) return p.index ? (size_t)p.index[r] : r;
+    const long long id = p.tokens[r];
+    return (size_t)(id < 0 ? 0 : (id >= p.vocab ? p.vocab - 1 : id));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kMaxThreads) stream_norm_kernel(const __grid_constant__ StreamNorm p) {
+    chain_enter();
+    extern __shared__ float row[];
+    __shared__ float red[33];
+    const int width = p.width;
+    const size_t at = (size_t)blockIdx.x * width, src = source_row(p, blockIdx.x) * width;
+    const T* y = reinterpret_cast<const T*>(p.y) + at;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        float v = p.table ? ld_bf16(p.table + src + i) : p.x_in[src + i];
+        if (p.y) v += load_f(y + i);
+        if (p.step) v += ld_bf16(p.step + i);
+        if (p.x_out) p.x_out[at + i] = v;
+        row[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    if (!p.norm) return;
+    const float factor = 1.0f / sqrtf(block_sum(ss, red) / (float)width + p.eps);
+    T* normed = reinterpret_cast<T*>(p.normed) + at;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) store_f(normed + i, row[i] * factor * (p.offset + ld_bf16(p.norm + i)));
+}
+
+// The same for widths that split evenly: VPT groups of four consecutive elements per thread, in registers.
+template <typename T, int VPT>
+__global__ void __launch_bounds__(kMaxThreads) stream_norm_vec_kernel(const __grid_constant__ StreamNorm p) {
+    chain_enter();
+    __shared__ float red[33];
+    const int width = p.width, threads = blockDim.x;
+    const size_t at = (size_t)blockIdx.x * width, src = source_row(p, blockIdx.x) * width;
+    const T* y = reinterpret_cast<const T*>(p.y) + at;
+    float4 v[VPT];
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int i = (threadIdx.x + k * threads) * 4;
+        v[k] = p.table ? load4(p.table + src + i) : load4(p.x_in + src + i);
+    }
+    if (p.y)
+#pragma unroll
+        for (int k = 0; k < VPT; ++k) {
+            const float4 a = load4(y + (threadIdx.x + k * threads) * 4);
+            v[k].x += a.x; v[k].y += a.y; v[k].z += a.z; v[k].w += a.w;
+        }
+    if (p.step)
+#pragma unroll
+        for (int k = 0; k < VPT; ++k) {
+            const float4 a = load4(p.step + (threadIdx.x + k * threads) * 4);
+            v[k].x += a.x; v[k].y += a.y; v[k].z += a.z; v[k].w += a.w;
+        }
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        if (p.x_out) store4(p.x_out + at + (threadIdx.x + k * threads) * 4, v[k]);
+        ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, ss))));
+    }
+    if (!p.norm) return;
+    const float factor = 1.0f / sqrtf(block_sum(ss, red) / (float)width + p.eps);
+    T* normed = reinterpret_cast<T*>(p.normed) + at;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int i = (threadIdx.x + k * threads) * 4;
+        const float4 w = load4(p.norm + i);
+        store4(normed + i, make_float4(v[k].x * factor * (p.offset + w.x), v[k].y * factor * (p.offset + w.y),
+                                       v[k].z * factor * (p.offset + w.z), v[k].w * factor * (p.offset + w.w)));
+    }
+}
+
 int row_threads(int width) {
     int threads = (width / 4 + 31) / 32 * 32;
     return threads < 64 ? 64 : (threads > kMaxThreads ? kMaxThreads : threads);
@@ -240,6 +324,22 @@ int close(const CloseParams& p, int tokens, cudaStream_t s) {
     return qd_launch(sublayer_close_kernel<T>, dim3(tokens), dim3(row_threads(p.width)), smem, s, 1, p);
 }
 
+template <typename T>
+int stream_norm(const StreamNorm& p, int rows, cudaStream_t s) {
+    const int quads = p.width / 4;
+    const auto fits = [&](int vpt) { return quads % (32 * vpt) == 0 && quads / vpt <= kMaxThreads; };
+    if (p.width % 4 == 0 && aligned16(p.table) && aligned16(p.x_in) && aligned16(p.y) && aligned16(p.step) && aligned16(p.x_out) &&
+        aligned16(p.norm) && aligned16(p.normed)) {
+        if (fits(1) && (rows < 64 || quads <= 256)) return qd_launch(stream_norm_vec_kernel<T, 1>, dim3(rows), dim3(quads), 0, s, 1, p);
+        if (fits(2)) return qd_launch(stream_norm_vec_kernel<T, 2>, dim3(rows), dim3(quads / 2), 0, s, 1, p);
+        if (fits(4)) return qd_launch(stream_norm_vec_kernel<T, 4>, dim3(rows), dim3(quads / 4), 0, s, 1, p);
+        if (fits(1)) return qd_launch(stream_norm_vec_kernel<T, 1>, dim3(rows), dim3(quads), 0, s, 1, p);
+    }
+    const size_t smem = (size_t)p.width * 4;
+    if (!allow_smem(stream_norm_kernel<T>, smem)) return QD_ERR_UNSUPPORTED;
+    return qd_launch(stream_norm_kernel<T>, dim3(rows), dim3(row_threads(p.width)), smem, s, 1, p);
+}
+
 }  // namespace
 }  // namespace qd
 
@@ -271,5 +371,16 @@ extern "C" int qd_sublayer_close(const void* y, const void* gate, long long ld_g
                                width, eps};
     if (dtype == QD_BF16) return qd::close<bf16>(p, tokens, (cudaStream_t)stream);
     if (dtype == QD_F32) return qd::close<float>(p, tokens, (cudaStream_t)stream);
+    return QD_ERR_UNSUPPORTED;
+}
+
+extern "C" int qd_stream_norm(const void* tokens, const void* table, int vocab, const float* x_in, const int* index, const void* y,
+                              const void* step, float* x_out, const void* norm, float norm_offset, void* normed, int rows, int width,
+                              float eps, int dtype, void* stream) {
+    QD_CHECK_ARG((table ? tokens && vocab > 0 : x_in != nullptr) && rows > 0 && width > 0 && (x_out || norm) && (!norm || normed));
+    const qd::StreamNorm p = {(const long long*)tokens, (const bf16*)table, vocab, x_in, index, y, (const bf16*)step, x_out,
+                              (const bf16*)norm, norm_offset, eps, normed, width};
+    if (dtype == QD_BF16) return qd::stream_norm<bf16>(p, rows, (cudaStream_t)stream);
+    if (dtype == QD_F32) return qd::stream_norm<float>(p, rows, (cudaStream_t)stream);
     return QD_ERR_UNSUPPORTED;
 }

@@ -1,53 +1,46 @@
-// Sliding-window attention with a learned sink per head in the softmax's denominator, RMS norm over the
-// whole query / key projection, interleaved rotary positions, and one sigmoid output gate per head.
-// The window's keys and values live in a ring of `capacity` rows (position p in row p mod capacity), so a
-// sequence's cache does not grow with its length.
+// Grouped-query softmax attention over a bounded span of positions, with what a design may put around it:
+//   mask     the last `span` positions, or the positions of the same chunk of `span` positions from 0
+//   scores   scaled; minus a slope per head times the distance
+//   sink     none, a learned score per head, or a score of zero, in the softmax's denominator only
+//   q and k  RMS norm over the whole projection or per head, interleaved rotary positions
+//   result   times one sigmoid gate per head or per value column
+// The visible keys and values live in a ring of `capacity` rows (position p in row p mod capacity), so a
+// sequence's cache does not grow with its length.  Keys may end in columns that all heads share (k_shared).
 //
 // Prompt chunks: attn_prepare_kernel (norm, rotation, ring rows) and attn_flash_kernel (mma.sync m16n8k16;
 // 64 or 128 packed (token, head of the group) rows per block, key tiles of 64 through two cp.async buffers,
 // only the tiles a row of the block can see; probabilities as two bf16 pieces).  attn_rows_kernel covers fp32
 // and shapes without 16-byte rows.  Decode: attn_step_kernel, one launch: norm and rotation in every
-// block, blocks = (key/value head, split of the window), the last block of a head merges.
-#include "typed.cuh"
+// block, blocks = (key/value head, split of the span), the last block of a head merges.
+#include "softmax_attention.cuh"
 
 namespace qd {
 namespace {
 
-// Angle of a pair in fp32: position * (f_hi + f_lo) with the product's rounding error carried along, so
-// that the rotation is that of the exact angle to fp32 rounding at any position.
-QD_DEVINL void rotation(int position, float f_hi, float f_lo, float& c, float& s) {
-    const float a = (float)position * f_hi;
-    const float err = fmaf((float)position, f_hi, -a) + (float)position * f_lo;
-    float c0, s0;
-    sincosf(a, &s0, &c0);
-    c = fmaf(-err, s0, c0);
-    s = fmaf(err, c0, s0);
-}
-
-// normalised, rotated element e (within its head: d) of a projection row
+// normalised, rotated element d of the head whose elements start at `first` of a projection row
 template <typename T>
-QD_DEVINL float rotated(const T* row, const bf16* w, float rms, int e, int d, int rot, const float* cosine, const float* sine) {
-    const float x = load_f(row + e) * rms * ld_bf16(w + e);
+QD_DEVINL float rotated(const T* row, const bf16* w, int norm, float rms, int first, int d, int rot, const float* cosine, const float* sine) {
+    if (norm == QD_NORM_ROW) w += first;
+    const auto at = [&](int e) { return norm == QD_NORM_NONE ? load_f(row + first + e) : load_f(row + first + e) * rms * ld_bf16(w + e); };
+    const float x = at(d);
     if (d >= rot) return x;
     const int i = d >> 1;
-    const float other = load_f(row + (e ^ 1) + 0) * rms * ld_bf16(w + (e ^ 1));
+    const float other = at(d ^ 1);
     return (d & 1) ? fmaf(x, cosine[i], other * sine[i]) : fmaf(x, cosine[i], -other * sine[i]);
 }
 
-struct AttnParams {
-    const void* q; const void* k; const void* v; const void* gate; long long ld;      // projection rows
-    const bf16* q_norm; const bf16* k_norm; const float* freq; int rot;               // freq: [2][rot / 2], high and low parts
-    const bf16* sink; float scale, eps;
-    void* k_cache; void* v_cache; int capacity, window;
-    const int* position_ptr; int position;
-    void* q_out; void* out;
-    int tokens, heads, kv_heads, dim, vdim;
-};
+typedef qd_attention_args AttnParams;
+QD_DEVINL const bf16* as_bf16(const void* p) { return reinterpret_cast<const bf16*>(p); }
+// lowest position that `position` sees
+__host__ __device__ __forceinline__ int lowest_key(const AttnParams& p, int position) {
+    if (p.mask == QD_MASK_CHUNK) return position - position % p.span;
+    return position - p.span + 1 > 0 ? position - p.span + 1 : 0;
+}
 
 template <typename T>
 __global__ void __launch_bounds__(256) attn_prepare_kernel(const __grid_constant__ AttnParams p) {
     chain_enter();
-    extern __shared__ float trig[];                    // cosines, sines
+    extern __shared__ float trig[];                    // cosines, sines, head factors
     __shared__ float red[33];
     const int t = blockIdx.x, tid = threadIdx.x, half = p.rot / 2;
     const int position = (p.position_ptr ? *p.position_ptr : p.position) + t;
@@ -56,49 +49,80 @@ __global__ void __launch_bounds__(256) attn_prepare_kernel(const __grid_constant
     const T* k = reinterpret_cast<const T*>(p.k) + (long long)t * p.ld;
     const T* v = reinterpret_cast<const T*>(p.v) + (long long)t * p.ld;
     for (int i = tid; i < half; i += 256) rotation(position, p.freq[i], p.freq[half + i], trig[i], trig[half + i]);
-    float qq = 0.f, kk = 0.f;
-    for (int i = tid; i < qn; i += 256) { const float x = load_f(q + i); qq = fmaf(x, x, qq); }
-    for (int i = tid; i < kn; i += 256) { const float x = load_f(k + i); kk = fmaf(x, x, kk); }
-    const float qr = 1.0f / sqrtf(block_sum(qq, red) / (float)qn + p.eps), kr = 1.0f / sqrtf(block_sum(kk, red) / (float)kn + p.eps);
+    float* head_rms = trig + p.rot;                    // of the query heads, then of the key heads
+    float qr = 1.f, kr = 1.f;
+    if (p.norm == QD_NORM_ROW) {
+        float qq = 0.f, kk = 0.f;
+        for (int i = tid; i < qn; i += 256) { const float x = load_f(q + i); qq = fmaf(x, x, qq); }
+        for (int i = tid; i < kn; i += 256) { const float x = load_f(k + i); kk = fmaf(x, x, kk); }
+        qr = 1.0f / sqrtf(block_sum(qq, red) / (float)qn + p.eps);
+        kr = 1.0f / sqrtf(block_sum(kk, red) / (float)kn + p.eps);
+    } else if (p.norm == QD_NORM_HEAD) {
+        for (int h = tid >> 5; h < p.heads + p.kv_heads; h += 8) {
+            const T* row = h < p.heads ? q + h * p.dim : k + (h - p.heads) * p.dim;
+            float ss = 0.f;
+            for (int d = tid & 31; d < p.dim; d += 32) { const float x = load_f(row + d); ss = fmaf(x, x, ss); }
+            ss = warp_sum(ss);
+            if ((tid & 31) == 0) head_rms[h] = 1.0f / sqrtf(ss / (float)p.dim + p.eps);
+        }
+    }
+    __syncthreads();
     const size_t slot = position % p.capacity;
-    T* ring_k = reinterpret_cast<T*>(p.k_cache) + slot * kn;
-    T* ring_v = reinterpret_cast<T*>(p.v_cache) + slot * vn;
-    T* q_out = reinterpret_cast<T*>(p.q_out) + (size_t)t * qn;
-    for (int i = tid; i < qn; i += 256) store_f(q_out + i, rotated(q, p.q_norm, qr, i, i % p.dim, p.rot, trig, trig + half));
-    for (int i = tid; i < kn; i += 256) store_f(ring_k + i, rotated(k, p.k_norm, kr, i, i % p.dim, p.rot, trig, trig + half));
+    T* ring_k = reinterpret_cast<T*>(p.k_cache) + slot * p.ld_k;
+    T* ring_v = reinterpret_cast<T*>(p.v_cache) + slot * p.ld_v;
+    T* q_out = reinterpret_cast<T*>(p.q_rows) + (size_t)t * qn;
+    const bool heads = p.norm == QD_NORM_HEAD;
+    for (int i = tid; i < qn; i += 256) {
+        const int h = i / p.dim;
+        store_f(q_out + i, rotated(q, as_bf16(p.q_norm), p.norm, heads ? head_rms[h] : qr, h * p.dim, i - h * p.dim, p.rot, trig, trig + half));
+    }
+    for (int i = tid; i < kn; i += 256) {
+        const int h = i / p.dim;
+        store_f(ring_k + i, rotated(k, as_bf16(p.k_norm), p.norm, heads ? head_rms[p.heads + h] : kr, h * p.dim, i - h * p.dim, p.rot, trig,
+                                    trig + half));
+    }
     for (int i = tid; i < vn; i += 256) ring_v[i] = v[i];
 }
 
 // ----------------------------------------------------------------------------- any type, any shape
-constexpr int kRowsPerLane = 8;                        // value columns per lane: vdim <= 256
+constexpr int kRowsPerLane = 8;                        // value columns per lane: 256 per block column
+
+template <typename T>
+QD_DEVINL void add_dot(const T* q, const T* k, int n, float (&dot)[4]) {
+    int d = 0;
+    for (; d + 4 <= n; d += 4)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) dot[i] = fmaf(load_f(q + d + i), load_f(k + d + i), dot[i]);
+    for (; d < n; ++d) dot[0] = fmaf(load_f(q + d), load_f(k + d), dot[0]);
+}
 
 template <typename T>
 __global__ void __launch_bounds__(256) attn_rows_kernel(const __grid_constant__ AttnParams p) {
     chain_enter();
     const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-    const int lane = threadIdx.x & 31;
+    const int lane = threadIdx.x & 31, c0 = blockIdx.y * 32 * kRowsPerLane + lane;
     if (item >= (long long)p.tokens * p.heads) return;
     const int t = (int)(item / p.heads), h = (int)(item % p.heads), g = h / (p.heads / p.kv_heads);
-    const int position = (p.position_ptr ? *p.position_ptr : p.position) + t, lo = max(0, position - p.window + 1);
-    const T* q = reinterpret_cast<const T*>(p.q_out) + item * p.dim;
-    const T* kc = reinterpret_cast<const T*>(p.k_cache);
-    const T* vc = reinterpret_cast<const T*>(p.v_cache);
-    const float sink = ld_bf16(p.sink + h);
-    float m = sink, l = 1.f, acc[kRowsPerLane];        // the sink is the first term of the running softmax
+    const int position = (p.position_ptr ? *p.position_ptr : p.position) + t, lo = lowest_key(p, position);
+    const T* q = reinterpret_cast<const T*>(p.q_rows) + item * (p.dim + p.shared_dim);
+    const T* kc = reinterpret_cast<const T*>(p.k_cache) + g * p.dim;
+    const T* vc = reinterpret_cast<const T*>(p.v_cache) + g * p.vdim;
+    const T* common = reinterpret_cast<const T*>(p.k_shared);
+    const float slope = p.slopes ? p.slopes[h] : 0.f;
+    // the sink is the first term of the running softmax
+    float m = -INFINITY, l = 0.f, acc[kRowsPerLane];
+    if (p.sink_kind != QD_SINK_NONE) { m = p.sink_kind == QD_SINK_LEARNED ? ld_bf16(as_bf16(p.sink) + h) : 0.f; l = 1.f; }
 #pragma unroll
     for (int c = 0; c < kRowsPerLane; ++c) acc[c] = 0.f;
     for (int j0 = lo; j0 <= position; j0 += 32) {
         const int j = j0 + lane;
         float score = -INFINITY;
         if (j <= position) {
-            const T* k = kc + ((size_t)(j % p.capacity) * p.kv_heads + g) * p.dim;
+            const size_t slot = j % p.capacity;
             float dot[4] = {0.f, 0.f, 0.f, 0.f};
-            int d = 0;
-            for (; d + 4 <= p.dim; d += 4)
-#pragma unroll
-                for (int i = 0; i < 4; ++i) dot[i] = fmaf(load_f(q + d + i), load_f(k + d + i), dot[i]);
-            for (; d < p.dim; ++d) dot[0] = fmaf(load_f(q + d), load_f(k + d), dot[0]);
-            score = ((dot[0] + dot[1]) + (dot[2] + dot[3])) * p.scale;
+            add_dot(q, kc + slot * p.ld_k, p.dim, dot);
+            if (p.shared_dim) add_dot(q + p.dim, common + slot * p.ld_shared, p.shared_dim, dot);
+            score = ((dot[0] + dot[1]) + (dot[2] + dot[3])) * p.scale - slope * (float)(position - j);
         }
         const float top = fmaxf(m, warp_max(score)), keep = expf(m - top), w = j <= position ? expf(score - top) : 0.f;
         l = l * keep + warp_sum(w);
@@ -108,52 +132,39 @@ __global__ void __launch_bounds__(256) attn_rows_kernel(const __grid_constant__ 
         const int count = min(32, position - j0 + 1);
         for (int i = 0; i < count; ++i) {
             const float wi = __shfl_sync(0xffffffffu, w, i);
-            const T* v = vc + ((size_t)((j0 + i) % p.capacity) * p.kv_heads + g) * p.vdim;
+            const T* v = vc + (size_t)((j0 + i) % p.capacity) * p.ld_v;
 #pragma unroll
             for (int c = 0; c < kRowsPerLane; ++c)
-                if (c * 32 + lane < p.vdim) acc[c] = fmaf(wi, load_f(v + c * 32 + lane), acc[c]);
+                if (c0 + c * 32 < p.vdim) acc[c] = fmaf(wi, load_f(v + c0 + c * 32), acc[c]);
         }
     }
-    const float gate = sigmoid_precise(load_f(reinterpret_cast<const T*>(p.gate) + (long long)t * p.ld + h)) / l;
+    const T* gate = reinterpret_cast<const T*>(p.gate) + (long long)t * p.ld_gate;
+    const float f = (p.gate_kind == QD_GATE_HEAD ? sigmoid_precise(load_f(gate + h)) : 1.f) / l;
     T* out = reinterpret_cast<T*>(p.out) + item * p.vdim;
 #pragma unroll
-    for (int c = 0; c < kRowsPerLane; ++c)
-        if (c * 32 + lane < p.vdim) store_f(out + c * 32 + lane, acc[c] * gate);
+    for (int c = 0; c < kRowsPerLane; ++c) {
+        const int column = c0 + c * 32;
+        if (column >= p.vdim) continue;
+        const float g2 = p.gate_kind == QD_GATE_VALUE ? sigmoid_precise(load_f(gate + h * p.vdim + column)) : 1.f;
+        store_f(out + column, acc[c] * f * g2);
+    }
 }
 
 // ------------------------------------------------------------------------------- tensor cores
 constexpr int kFlashKeys = 64;
-constexpr float kLog2e = 1.4426950408889634f;
-
-QD_DEVINL void mma_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-QD_DEVINL void ldmatrix4(uint32_t (&r)[4], const void* p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
-}
-QD_DEVINL void ldmatrix4_t(uint32_t (&r)[4], const void* p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
-}
-QD_DEVINL void copy16_or_zero(void* dst, const void* src, bool ok) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(ok ? 16 : 0) : "memory");
-}
-QD_DEVINL uint32_t pack_pair(float lo, float hi) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t*>(&v);
+template <int DV> size_t flash_smem(const qd_attention_args& p, int warps) {
+    const int krow = ((p.dim + p.shared_dim + 15) & ~15) + 8;
+    return sizeof(bf16) * ((size_t)(warps * 16 + 2 * kFlashKeys) * krow + 2ull * kFlashKeys * (DV + 8));
 }
 
-// dim, vdim multiples of eight, vdim <= DV (a multiple of sixteen).  Shared rows are padded to an odd
+// dim, shared_dim, vdim and the row strides multiples of eight, vdim <= DV (a multiple of sixteen).  Shared rows are padded to an odd
 // number of 16-byte pieces: the eight rows an ldmatrix phase touches fall into different banks.
 template <int DV, int WARPS>
 __global__ void __launch_bounds__(WARPS * 32) attn_flash_kernel(const __grid_constant__ AttnParams p) {
     chain_enter();
     extern __shared__ __align__(16) bf16 tiles[];
     constexpr int kVRow = DV + 8, kFlashRows = WARPS * 16, kFlashThreads = WARPS * 32;
-    const int dk = (p.dim + 15) & ~15, krow = dk + 8;
+    const int qdim = p.dim + p.shared_dim, dk = (qdim + 15) & ~15, krow = dk + 8;
     bf16* qs = tiles;
     bf16* ks = qs + kFlashRows * krow;
     bf16* vs = ks + 2 * kFlashKeys * krow;
@@ -162,33 +173,35 @@ __global__ void __launch_bounds__(WARPS * 32) attn_flash_kernel(const __grid_con
     const int r0 = blockIdx.x * kFlashRows;
     const int base = p.position_ptr ? *p.position_ptr : p.position;
     const int pos_first = base + r0 / share, pos_last = base + (min(r0 + kFlashRows, total) - 1) / share;
-    const int key_first = max(0, pos_first - p.window + 1);
+    const int key_first = lowest_key(p, pos_first);
     const int ntiles = (pos_last - key_first) / kFlashKeys + 1;
-    const bf16* kc = reinterpret_cast<const bf16*>(p.k_cache);
-    const bf16* vc = reinterpret_cast<const bf16*>(p.v_cache);
-    const bf16* q = reinterpret_cast<const bf16*>(p.q_out);
+    const bf16* kc = as_bf16(p.k_cache) + g * p.dim;
+    const bf16* vc = as_bf16(p.v_cache) + g * p.vdim;
+    const bf16* common = as_bf16(p.k_shared);
+    const bf16* q = as_bf16(p.q_rows);
 
     // padding columns stay zero
     const int all = (kFlashRows + 2 * kFlashKeys) * krow + 2 * kFlashKeys * kVRow;
     for (int i = tid; i < all / 8; i += kFlashThreads) reinterpret_cast<uint4*>(tiles)[i] = make_uint4(0u, 0u, 0u, 0u);
     __syncthreads();
-    const int kp = p.dim / 8, vp = p.vdim / 8;
-    for (int i = tid; i < kFlashRows * kp; i += kFlashThreads) {
-        const int r = i / kp, piece = i % kp, row = r0 + r;
+    const int kp = p.dim / 8, qp = qdim / 8, vp = p.vdim / 8;          // 16-byte pieces
+    for (int i = tid; i < kFlashRows * qp; i += kFlashThreads) {
+        const int r = i / qp, piece = i % qp, row = r0 + r;
         const bool ok = row < total;
-        const size_t src = ok ? ((size_t)(row / share) * p.heads + g * share + row % share) * p.dim + piece * 8 : 0;
+        const size_t src = ok ? ((size_t)(row / share) * p.heads + g * share + row % share) * qdim + piece * 8 : 0;
         copy16_or_zero(qs + r * krow + piece * 8, q + src, ok);
     }
     auto stage = [&](int tile) {
         const int j0 = key_first + tile * kFlashKeys;
         bf16* kd = ks + (tile & 1) * kFlashKeys * krow;
         bf16* vd = vs + (tile & 1) * kFlashKeys * kVRow;
-        for (int i = tid; i < kFlashKeys * (kp + vp); i += kFlashThreads) {
-            const int r = i / (kp + vp), piece = i % (kp + vp), j = j0 + r;
+        for (int i = tid; i < kFlashKeys * (qp + vp); i += kFlashThreads) {
+            const int r = i / (qp + vp), piece = i % (qp + vp), j = j0 + r;
             const bool ok = j <= pos_last;
-            const size_t row = ok ? (size_t)(j % p.capacity) * p.kv_heads + g : 0;
-            if (piece < kp) copy16_or_zero(kd + r * krow + piece * 8, kc + row * p.dim + piece * 8, ok);
-            else copy16_or_zero(vd + r * kVRow + (piece - kp) * 8, vc + row * p.vdim + (piece - kp) * 8, ok);
+            const size_t slot = ok ? j % p.capacity : 0;
+            if (piece < kp) copy16_or_zero(kd + r * krow + piece * 8, kc + slot * p.ld_k + piece * 8, ok);
+            else if (piece < qp) copy16_or_zero(kd + r * krow + piece * 8, common + slot * p.ld_shared + (piece - kp) * 8, ok);
+            else copy16_or_zero(vd + r * kVRow + (piece - qp) * 8, vc + slot * p.ld_v + (piece - qp) * 8, ok);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -202,7 +215,12 @@ __global__ void __launch_bounds__(WARPS * 32) attn_flash_kernel(const __grid_con
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     const int row_of[2] = {r0 + warp * 16 + (lane >> 2), r0 + warp * 16 + (lane >> 2) + 8};
     const int pos_of[2] = {base + row_of[0] / share, base + row_of[1] / share};
+    const int lo_of[2] = {lowest_key(p, pos_of[0]), lowest_key(p, pos_of[1])}, lo_last = lowest_key(p, pos_last);
     const float scale = p.scale * kLog2e;
+    float slope[2] = {0.f, 0.f};
+    if (p.slopes)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) slope[i] = p.slopes[g * share + row_of[i] % share] * kLog2e;
     // ldmatrix addresses: lane -> (row within 16, 8-column half)
     const bf16* qa = qs + (warp * 16 + (lane & 15)) * krow + (lane >> 4) * 8;
     const int kb = ((lane & 7) + ((lane >> 4) << 3)) * krow + ((lane >> 3) & 1) * 8;
@@ -232,14 +250,14 @@ __global__ void __launch_bounds__(WARPS * 32) attn_flash_kernel(const __grid_con
             }
         }
         // every key of the tile visible to every row: no masking
-        const bool inside = j0 + kFlashKeys - 1 <= pos_first && j0 > pos_last - p.window;
+        const bool inside = j0 + kFlashKeys - 1 <= pos_first && j0 >= lo_last;
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int n = 0; n < 8; ++n)
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
                 const int j = j0 + n * 8 + (lane & 3) * 2 + (c & 1), pos = pos_of[c >> 1];
-                s[n][c] = (inside || (j <= pos && j > pos - p.window)) ? s[n][c] * scale : -INFINITY;
+                s[n][c] = (inside || (j <= pos && j >= lo_of[c >> 1])) ? fmaf(s[n][c], scale, slope[c >> 1] * (float)(j - pos)) : -INFINITY;
                 mx[c >> 1] = fmaxf(mx[c >> 1], s[n][c]);
             }
 #pragma unroll
@@ -288,20 +306,33 @@ __global__ void __launch_bounds__(WARPS * 32) attn_flash_kernel(const __grid_con
         l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
         if (row_of[i] >= total) continue;
         const int t = row_of[i] / share, h = g * share + row_of[i] % share;
-        const float sink = ld_bf16(p.sink + h) * kLog2e, top = fmaxf(m[i], sink), keep = exp2f(m[i] - top);
-        const float gate = sigmoid_precise(ld_bf16(reinterpret_cast<const bf16*>(p.gate) + (long long)t * p.ld + h));
-        const float f = keep / (l[i] * keep + exp2f(sink - top)) * gate;
+        const bf16* gate = as_bf16(p.gate) + (long long)t * p.ld_gate;
+        float f = 1.f / l[i];
+        if (p.sink_kind != QD_SINK_NONE) {
+            const float sink = p.sink_kind == QD_SINK_LEARNED ? ld_bf16(as_bf16(p.sink) + h) * kLog2e : 0.f;
+            const float top = fmaxf(m[i], sink), keep = exp2f(m[i] - top);
+            f = keep / (l[i] * keep + exp2f(sink - top));
+        }
+        if (p.gate_kind == QD_GATE_HEAD) f *= sigmoid_precise(ld_bf16(gate + h));
         bf16* out = reinterpret_cast<bf16*>(p.out) + ((size_t)t * p.heads + h) * p.vdim + (lane & 3) * 2;
 #pragma unroll
         for (int n = 0; n < DV / 8; ++n)
-            if (n * 8 < p.vdim) *reinterpret_cast<uint32_t*>(out + n * 8) = pack_pair(o[n][2 * i] * f, o[n][2 * i + 1] * f);
+            if (n * 8 < p.vdim) {
+                float a = o[n][2 * i] * f, b = o[n][2 * i + 1] * f;
+                if (p.gate_kind == QD_GATE_VALUE) {
+                    const bf16* z = gate + h * p.vdim + (lane & 3) * 2 + n * 8;
+                    a *= sigmoid_precise(ld_bf16(z));
+                    b *= sigmoid_precise(ld_bf16(z + 1));
+                }
+                *reinterpret_cast<uint32_t*>(out + n * 8) = pack_pair(a, b);
+            }
     }
 }
 
 // ------------------------------------------------------------------------------------- decode
 constexpr int kStepKeys = 64, kStepThreads = 256;
 
-struct AttnStep { AttnParams a; float* partial; unsigned int* counters; int splits, buffers; };      // buffers: key tiles in shared memory, 1 or 2
+struct AttnStep { AttnParams a; int buffers; };      // buffers: key tiles in shared memory, 1 or 2
 __host__ __device__ constexpr size_t step_stats_floats(int heads, int splits) { return (2 * (size_t)heads * splits + 3) / 4 * 4; }
 
 // Elements of a shared row of n elements: 16-byte pieces, an odd number of them (rows read side by side
@@ -340,6 +371,7 @@ QD_DEVINL void dot_rows2(const float* q0, const float* q1, const T* k, int n, bo
     d1 = (b[0] + b[1]) + (b[2] + b[3]);
 }
 
+// shared memory of attn_step_kernel
 template <typename T>
 static size_t step_smem(int share, int dim, int vdim, int rot, int buffers) {
     const int dp = step_row<float>(dim), vp = step_row<float>(vdim);
@@ -364,17 +396,17 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
     T* ks = reinterpret_cast<T*>(stat + share * 4);       // buffers of [kStepKeys][krow]
     T* vs = ks + sp.buffers * kStepKeys * krow;           // buffers of [kStepKeys][vrow]
     float* trig = reinterpret_cast<float*>(vs + sp.buffers * kStepKeys * vrow);
-    const int position = p.position_ptr ? *p.position_ptr : p.position, lo = max(0, position - p.window + 1), n = position - lo + 1;
-    const int per = max((n + sp.splits - 1) / sp.splits, 32), active = (n + per - 1) / per;
+    const int position = p.position_ptr ? *p.position_ptr : p.position, lo = lowest_key(p, position), n = position - lo + 1;
+    const int per = max((n + p.splits - 1) / p.splits, 32), active = (n + per - 1) / per;
     if (split >= active) return;
     const int first = lo + split * per, end = min(first + per, position + 1);
-    const int qn = p.heads * dim, kn = p.kv_heads * dim, vn = p.kv_heads * vdim;
-    T* kc = reinterpret_cast<T*>(p.k_cache);
-    T* vc = reinterpret_cast<T*>(p.v_cache);
+    const int qn = p.heads * dim, kn = p.kv_heads * dim;
+    T* kc = reinterpret_cast<T*>(p.k_cache) + g * dim;
+    T* vc = reinterpret_cast<T*>(p.v_cache) + g * vdim;
 
     // a warp per cache row; the token's own row is not in the ring yet
     constexpr int E = 16 / (int)sizeof(T);
-    const bool pieces = dim % E == 0 && vdim % E == 0;
+    const bool pieces = dim % E == 0 && vdim % E == 0 && p.ld_k % E == 0 && p.ld_v % E == 0;
     auto stage = [&](int j0) {
         const int buf = ((j0 - first) / kStepKeys) & (sp.buffers - 1), count = min(kStepKeys, end - j0);
         T* kd = ks + buf * kStepKeys * krow;
@@ -382,16 +414,17 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
         for (int r = warp; r < count; r += kStepThreads / 32) {
             const int j = j0 + r;
             if (j == position) continue;
-            const size_t row = (size_t)(j % p.capacity) * p.kv_heads + g;
+            const T* krow_of = kc + (size_t)(j % p.capacity) * p.ld_k;
+            const T* vrow_of = vc + (size_t)(j % p.capacity) * p.ld_v;
             if (pieces) {
                 const int kp = dim / E, all = kp + vdim / E;
                 for (int i = lane; i < all; i += 32) {
-                    if (i < kp) copy16_or_zero(kd + r * krow + i * E, kc + row * dim + i * E, true);
-                    else copy16_or_zero(vd + r * vrow + (i - kp) * E, vc + row * vdim + (i - kp) * E, true);
+                    if (i < kp) copy16_or_zero(kd + r * krow + i * E, krow_of + i * E, true);
+                    else copy16_or_zero(vd + r * vrow + (i - kp) * E, vrow_of + (i - kp) * E, true);
                 }
             } else {
-                for (int d = lane; d < dim; d += 32) kd[r * krow + d] = kc[row * dim + d];
-                for (int d = lane; d < vdim; d += 32) vd[r * vrow + d] = vc[row * vdim + d];
+                for (int d = lane; d < dim; d += 32) kd[r * krow + d] = krow_of[d];
+                for (int d = lane; d < vdim; d += 32) vd[r * vrow + d] = vrow_of[d];
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -402,13 +435,31 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
     const T* k = reinterpret_cast<const T*>(p.k);
     const T* v = reinterpret_cast<const T*>(p.v) + g * vdim;
     for (int i = tid; i < half; i += kStepThreads) rotation(position, p.freq[i], p.freq[half + i], trig[i], trig[half + i]);
-    float qq = 0.f, kk = 0.f;
-    for (int i = tid; i < qn; i += kStepThreads) { const float x = load_f(q + i); qq = fmaf(x, x, qq); }
-    for (int i = tid; i < kn; i += kStepThreads) { const float x = load_f(k + i); kk = fmaf(x, x, kk); }
-    const float qr = 1.0f / sqrtf(block_sum(qq, red) / (float)qn + p.eps), kr = 1.0f / sqrtf(block_sum(kk, red) / (float)kn + p.eps);
-    for (int h = warp; h < share; h += kStepThreads / 32)
-        for (int d = lane; d < dim; d += 32)
-            qs[h * dp + d] = as_type<T>(rotated(q, p.q_norm, qr, (g * share + h) * dim + d, d, p.rot, trig, trig + half));
+    float qr = 1.f, kr = 1.f;
+    if (p.norm == QD_NORM_ROW) {
+        float qq = 0.f, kk = 0.f;
+        for (int i = tid; i < qn; i += kStepThreads) { const float x = load_f(q + i); qq = fmaf(x, x, qq); }
+        for (int i = tid; i < kn; i += kStepThreads) { const float x = load_f(k + i); kk = fmaf(x, x, kk); }
+        qr = 1.0f / sqrtf(block_sum(qq, red) / (float)qn + p.eps);
+        kr = 1.0f / sqrtf(block_sum(kk, red) / (float)kn + p.eps);
+    } else {
+        if (p.norm == QD_NORM_HEAD && end == position + 1) {
+            float kk = 0.f;
+            for (int d = tid; d < dim; d += kStepThreads) { const float x = load_f(k + g * dim + d); kk = fmaf(x, x, kk); }
+            kr = 1.0f / sqrtf(block_sum(kk, red) / (float)dim + p.eps);
+        }
+        __syncthreads();                                  // the rotation table
+    }
+    for (int h = warp; h < share; h += kStepThreads / 32) {
+        const int at = (g * share + h) * dim;
+        float r = qr;
+        if (p.norm == QD_NORM_HEAD) {
+            float qq = 0.f;
+            for (int d = lane; d < dim; d += 32) { const float x = load_f(q + at + d); qq = fmaf(x, x, qq); }
+            r = 1.0f / sqrtf(warp_sum(qq) / (float)dim + p.eps);
+        }
+        for (int d = lane; d < dim; d += 32) qs[h * dp + d] = as_type<T>(rotated(q, as_bf16(p.q_norm), p.norm, r, at, d, p.rot, trig, trig + half));
+    }
     for (int i = tid; i < share * vp; i += kStepThreads) acc[i] = 0.f;
     for (int i = tid; i < share; i += kStepThreads) { stat[i * 4] = -INFINITY; stat[i * 4 + 1] = 0.f; }
     if (end == position + 1) {                            // this split holds the token itself: into its tile and into the ring
@@ -417,11 +468,11 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
         T* kd = ks + (size_t)(buf * kStepKeys + r) * krow;
         T* vd = vs + (size_t)(buf * kStepKeys + r) * vrow;
         for (int d = tid; d < dim; d += kStepThreads) {
-            store_f(kc + slot * kn + g * dim + d, rotated(k, p.k_norm, kr, g * dim + d, d, p.rot, trig, trig + half));
-            if (position - first < kStepKeys * sp.buffers) kd[d] = kc[slot * kn + g * dim + d];
+            store_f(kc + slot * p.ld_k + d, rotated(k, as_bf16(p.k_norm), p.norm, kr, g * dim, d, p.rot, trig, trig + half));
+            if (position - first < kStepKeys * sp.buffers) kd[d] = kc[slot * p.ld_k + d];
         }
         for (int d = tid; d < vdim; d += kStepThreads) {
-            vc[slot * vn + g * vdim + d] = v[d];
+            vc[slot * p.ld_v + d] = v[d];
             if (position - first < kStepKeys * sp.buffers) vd[d] = v[d];
         }
     }
@@ -436,7 +487,7 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
         if (position < j0 + kStepKeys && position >= j0 && position - first >= kStepKeys * sp.buffers) {      // its buffer was busy before
             const size_t slot = position % p.capacity;
             const int r = position - j0;
-            for (int d = tid; d < dim; d += kStepThreads) kt[r * krow + d] = kc[slot * kn + g * dim + d];
+            for (int d = tid; d < dim; d += kStepThreads) kt[r * krow + d] = kc[slot * p.ld_k + d];
             for (int d = tid; d < vdim; d += kStepThreads) vt[r * vrow + d] = v[d];
         }
         __syncthreads();
@@ -450,6 +501,11 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
                     dot_rows2(qs + h * dp, qs + h2 * dp, kt + r * krow, dim, pieces, d0, d1);
                     d0 *= p.scale;
                     d1 *= p.scale;
+                    if (p.slopes) {
+                        const float distance = (float)(position - j0 - r);
+                        d0 = fmaf(-p.slopes[g * share + h], distance, d0);
+                        d1 = fmaf(-p.slopes[g * share + h2], distance, d1);
+                    }
                 }
                 score[h * kStepKeys + r] = d0;
                 if (h + kGroups < share) score[h2 * kStepKeys + r] = d1;
@@ -502,45 +558,48 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
 
     // partial results: (maximum, denominator) [head][split], then sums [head][split][vdim]; the last split of this
     // key/value head to arrive merges them
-    float2* stats = reinterpret_cast<float2*>(sp.partial) + (size_t)g * share * sp.splits;
-    float* sums = sp.partial + step_stats_floats(p.heads, sp.splits) + (size_t)g * share * sp.splits * vdim;
+    float2* stats = reinterpret_cast<float2*>(p.partial) + (size_t)g * share * p.splits;
+    float* sums = p.partial + step_stats_floats(p.heads, p.splits) + (size_t)g * share * p.splits * vdim;
     for (int i = tid; i < share * vdim; i += kStepThreads) {
         const int h = i / vdim, c = i % vdim;
-        sums[((size_t)h * sp.splits + split) * vdim + c] = acc[h * vp + c];
+        sums[((size_t)h * p.splits + split) * vdim + c] = acc[h * vp + c];
     }
-    for (int h = tid; h < share; h += kStepThreads) stats[h * sp.splits + split] = make_float2(stat[h * 4], stat[h * 4 + 1]);
+    for (int h = tid; h < share; h += kStepThreads) stats[h * p.splits + split] = make_float2(stat[h * 4], stat[h * 4 + 1]);
     __threadfence();
     __syncthreads();
-    if (tid == 0) last = atomicAdd(sp.counters + g, 1u) == (unsigned)active - 1u;
+    if (tid == 0) last = atomicAdd(p.counters + g, 1u) == (unsigned)active - 1u;
     __syncthreads();
     if (!last) return;
     __threadfence();
-    if (tid == 0) sp.counters[g] = 0u;
+    if (tid == 0) p.counters[g] = 0u;
     // factor of every split (sink, denominator and gate included) into the score rows, then the weighted sums
     for (int h = warp; h < share; h += kStepThreads / 32) {
         const int head = g * share + h;
-        const float sink = ld_bf16(p.sink + head);
+        const float sink = p.sink_kind == QD_SINK_NONE ? -INFINITY : (p.sink_kind == QD_SINK_LEARNED ? ld_bf16(as_bf16(p.sink) + head) : 0.f);
         float2 mine[kStepKeys / 32];
         float top = sink, sum = 0.f;
 #pragma unroll
         for (int i = 0; i < kStepKeys / 32; ++i) {
             const int s = i * 32 + lane;
-            mine[i] = s < active ? __ldcg(stats + h * sp.splits + s) : make_float2(-INFINITY, 0.f);
+            mine[i] = s < active ? __ldcg(stats + h * p.splits + s) : make_float2(-INFINITY, 0.f);
             top = fmaxf(top, mine[i].x);
         }
         top = warp_max(top);
 #pragma unroll
         for (int i = 0; i < kStepKeys / 32; ++i) { mine[i].x = expf(mine[i].x - top); sum = fmaf(mine[i].y, mine[i].x, sum); }
-        const float f = sigmoid_precise(load_f(reinterpret_cast<const T*>(p.gate) + head)) / (warp_sum(sum) + expf(sink - top));
+        const float gate_of = p.gate_kind == QD_GATE_HEAD ? sigmoid_precise(load_f(reinterpret_cast<const T*>(p.gate) + head)) : 1.f;
+        const float f = gate_of / (warp_sum(sum) + expf(sink - top));
 #pragma unroll
         for (int i = 0; i < kStepKeys / 32; ++i) score[h * kStepKeys + i * 32 + lane] = mine[i].x * f;
     }
     __syncthreads();
     T* out = reinterpret_cast<T*>(p.out) + (size_t)g * share * vdim;
+    const T* gate = reinterpret_cast<const T*>(p.gate) + (size_t)g * share * vdim;
+    const auto value_gate = [&](int i) { return p.gate_kind == QD_GATE_VALUE ? sigmoid_precise(load_f(gate + i)) : 1.f; };
     if (quads) {
         for (int i = tid; i < share * (vdim / 4); i += kStepThreads) {
             const int h = i / (vdim / 4), c = i % (vdim / 4) * 4;
-            const float* rows = sums + (size_t)h * sp.splits * vdim + c;
+            const float* rows = sums + (size_t)h * p.splits * vdim + c;
             float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 16
             for (int s = 0; s < active; ++s) {
@@ -548,41 +607,46 @@ __global__ void __launch_bounds__(kStepThreads) attn_step_kernel(const __grid_co
                 const float f = score[h * kStepKeys + s];
                 o.x = fmaf(x.x, f, o.x); o.y = fmaf(x.y, f, o.y); o.z = fmaf(x.z, f, o.z); o.w = fmaf(x.w, f, o.w);
             }
-            store4(out + h * vdim + c, o);
+            const int i0 = h * vdim + c;
+            o.x *= value_gate(i0); o.y *= value_gate(i0 + 1); o.z *= value_gate(i0 + 2); o.w *= value_gate(i0 + 3);
+            store4(out + i0, o);
         }
     } else {
         for (int i = tid; i < share * vdim; i += kStepThreads) {
             const int h = i / vdim, c = i % vdim;
             float o = 0.f;
-            for (int s = 0; s < active; ++s) o = fmaf(__ldcg(sums + ((size_t)h * sp.splits + s) * vdim + c), score[h * kStepKeys + s], o);
-            store_f(out + h * vdim + c, o);
+            for (int s = 0; s < active; ++s) o = fmaf(__ldcg(sums + ((size_t)h * p.splits + s) * vdim + c), score[h * kStepKeys + s], o);
+            store_f(out + h * vdim + c, o * value_gate(h * vdim + c));
         }
     }
 }
 
 template <int DV, int WARPS>
 int launch_flash_rows(const AttnParams& p, long long rows, cudaStream_t s) {
-    const int krow = ((p.dim + 15) & ~15) + 8;
-    const size_t smem = sizeof(bf16) * ((size_t)(WARPS * 16 + 2 * kFlashKeys) * krow + 2ull * kFlashKeys * (DV + 8));
-    if (!allow_smem(attn_flash_kernel<DV, WARPS>, smem)) return QD_ERR_UNSUPPORTED;
     const dim3 grid((unsigned)((rows + WARPS * 16 - 1) / (WARPS * 16)), p.kv_heads);
+    const size_t smem = flash_smem<DV>(p, WARPS);
+    if (!allow_smem(attn_flash_kernel<DV, WARPS>, smem)) return QD_ERR_UNSUPPORTED;
     return qd_launch(attn_flash_kernel<DV, WARPS>, grid, dim3(WARPS * 32), smem, s, 1, p);
 }
 template <int DV>
 int launch_flash(const AttnParams& p, cudaStream_t s) {
     const long long rows = (long long)p.tokens * (p.heads / p.kv_heads);
     // 128 rows share a key tile once such blocks fill the GPU
-    if (rows * p.kv_heads >= 128ll * device_sms()) return launch_flash_rows<DV, 8>(p, rows, s);
+    if (rows * p.kv_heads >= 128ll * device_sms() && flash_smem<DV>(p, 8) <= kMaxSmem) return launch_flash_rows<DV, 8>(p, rows, s);
     return launch_flash_rows<DV, 4>(p, rows, s);
 }
 template <typename T>
 int chunk(const AttnParams& p, cudaStream_t s) {
-    const size_t trig = (size_t)(p.rot + 1) * 4;
-    if (!allow_smem(attn_prepare_kernel<T>, trig)) return QD_ERR_UNSUPPORTED;
-    const int rc = qd_launch(attn_prepare_kernel<T>, dim3(p.tokens), dim3(256), trig, s, 1, p);
-    if (rc != QD_OK) return rc;
-    const bool rows16 = sizeof(T) == 2 && p.dim % 8 == 0 && p.vdim % 8 == 0 && aligned16(p.q_out) && aligned16(p.k_cache) && aligned16(p.v_cache);
-    if (rows16 && p.dim <= 256 && p.vdim <= 256 && ((uintptr_t)p.out & 3u) == 0) {
+    if (p.q) {
+        const size_t shared = (size_t)(p.rot + p.heads + p.kv_heads + 1) * 4;
+        if (!allow_smem(attn_prepare_kernel<T>, shared)) return QD_ERR_UNSUPPORTED;
+        const int rc = qd_launch(attn_prepare_kernel<T>, dim3(p.tokens), dim3(256), shared, s, 1, p);
+        if (rc != QD_OK) return rc;
+    }
+    const bool rows16 = sizeof(T) == 2 && p.dim % 8 == 0 && p.vdim % 8 == 0 && p.shared_dim % 8 == 0 && p.ld_k % 8 == 0 && p.ld_v % 8 == 0 &&
+                        p.ld_shared % 8 == 0 && aligned16(p.q_rows) && aligned16(p.k_cache) && aligned16(p.v_cache) && aligned16(p.k_shared) &&
+                        ((uintptr_t)p.out & 3u) == 0;
+    if (rows16 && p.vdim <= 256 && flash_smem<256>(p, 4) <= kMaxSmem) {
         if (p.vdim <= 32) return launch_flash<32>(p, s);
         if (p.vdim <= 64) return launch_flash<64>(p, s);
         if (p.vdim <= 96) return launch_flash<96>(p, s);
@@ -590,56 +654,50 @@ int chunk(const AttnParams& p, cudaStream_t s) {
         if (p.vdim <= 192) return launch_flash<192>(p, s);
         return launch_flash<256>(p, s);
     }
-    if (p.vdim > 32 * kRowsPerLane) return QD_ERR_UNSUPPORTED;
-    return qd_launch(attn_rows_kernel<T>, dim3((unsigned)(((long long)p.tokens * p.heads + 7) / 8)), dim3(256), 0, s, 1, p);
+    const dim3 grid((unsigned)(((long long)p.tokens * p.heads + 7) / 8), (p.vdim + 32 * kRowsPerLane - 1) / (32 * kRowsPerLane));
+    return qd_launch(attn_rows_kernel<T>, grid, dim3(256), 0, s, 1, p);
 }
 template <typename T>
-int step(AttnStep sp, cudaStream_t s) {
-    const auto smem = [&] { return step_smem<T>(sp.a.heads / sp.a.kv_heads, sp.a.dim, sp.a.vdim, sp.a.rot, sp.buffers); };
-    sp.buffers = 2;
+int step(const AttnParams& a, cudaStream_t s) {
+    AttnStep sp = {a, 2};
+    const auto smem = [&] { return step_smem<T>(a.heads / a.kv_heads, a.dim, a.vdim, a.rot, sp.buffers); };
     if (smem() > 220 * 1024) sp.buffers = 1;
     if (!allow_smem(attn_step_kernel<T>, smem())) return QD_ERR_UNSUPPORTED;
-    return qd_launch(attn_step_kernel<T>, dim3(sp.a.kv_heads, sp.splits), dim3(kStepThreads), smem(), s, 1, sp);
+    return qd_launch(attn_step_kernel<T>, dim3(a.kv_heads, a.splits), dim3(kStepThreads), smem(), s, 1, sp);
+}
+
+bool valid(const AttnParams& a) {
+    const bool caches = a.k_cache && a.v_cache && a.out && a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.vdim > 0 &&
+                        a.span > 0 && a.position >= 0 && a.capacity > 0 && a.shared_dim >= 0 && (a.shared_dim == 0 || a.k_shared) &&
+                        a.ld_k >= (long long)a.kv_heads * a.dim && a.ld_v >= (long long)a.kv_heads * a.vdim && a.ld_shared >= a.shared_dim;
+    const bool extras = (a.sink_kind != QD_SINK_LEARNED || a.sink) && (a.gate_kind == QD_GATE_NONE || a.gate) &&
+                        (a.mask == QD_MASK_WINDOW || a.mask == QD_MASK_CHUNK);
+    if (!a.q) return caches && extras;
+    return caches && extras && a.k && a.v && a.shared_dim == 0 && (a.norm == QD_NORM_NONE || (a.q_norm && a.k_norm)) && a.rot >= 0 && a.rot % 2 == 0 &&
+           a.rot <= a.dim && (a.rot == 0 || (a.freq && a.dim % 2 == 0));
 }
 
 }  // namespace
 }  // namespace qd
 
-#define QD_ATTN_ARGS_OK(tokens_ok)                                                                                         \
-    QD_CHECK_ARG(q && k && v && gate && q_norm && k_norm && sink && k_cache && v_cache && out && (tokens_ok));             \
-    QD_CHECK_ARG(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && vdim > 0 && window > 0 && position >= 0); \
-    QD_CHECK_ARG(rot >= 0 && rot % 2 == 0 && rot <= dim && (rot == 0 || (freq && dim % 2 == 0)) && capacity >= window)
-
-extern "C" int qd_window_attention(const void* q, const void* k, const void* v, const void* gate, long long ld, const void* q_norm,
-                                   const void* k_norm, const float* freq, int rot, const void* sink, float scale, float eps,
-                                   void* k_cache, void* v_cache, int capacity, int window, const int* position_ptr, int position,
-                                   void* q_scratch, void* out, int tokens, int heads, int kv_heads, int dim, int vdim, int dtype,
-                                   void* stream) {
-    QD_ATTN_ARGS_OK(tokens > 0 && q_scratch);
+extern "C" int qd_attention(const qd_attention_args* args, void* stream) {
+    QD_CHECK_ARG(args && qd::valid(*args) && args->tokens > 0 && args->q_rows);
+    const qd_attention_args& a = *args;
     // a chunk's own rows must not push out rows that its first token still sees
-    if (tokens + window - 1 > capacity && (position_ptr || position + tokens > capacity)) return QD_ERR_ARG;
-    const qd::AttnParams p = {q, k, v, gate, ld, (const bf16*)q_norm, (const bf16*)k_norm, freq, rot, (const bf16*)sink, scale, eps,
-                              k_cache, v_cache, capacity, window, position_ptr, position, q_scratch, out, tokens, heads, kv_heads,
-                              dim, vdim};
-    if (dtype == QD_BF16) return qd::chunk<bf16>(p, (cudaStream_t)stream);
-    if (dtype == QD_F32) return qd::chunk<float>(p, (cudaStream_t)stream);
+    if ((long long)a.tokens + a.span - 1 > a.capacity && (a.position_ptr || (long long)a.position + a.tokens > a.capacity)) return QD_ERR_ARG;
+    if (a.dtype == QD_BF16) return qd::chunk<bf16>(a, (cudaStream_t)stream);
+    if (a.dtype == QD_F32) return qd::chunk<float>(a, (cudaStream_t)stream);
     return QD_ERR_UNSUPPORTED;
 }
 
-extern "C" long long qd_window_attention_step_floats(int heads, int vdim, int splits) {
+extern "C" long long qd_attention_step_floats(int heads, int vdim, int splits) {
     return (long long)qd::step_stats_floats(heads, splits) + (long long)heads * splits * vdim;
 }
 
-extern "C" int qd_window_attention_step(const void* q, const void* k, const void* v, const void* gate, const void* q_norm,
-                                        const void* k_norm, const float* freq, int rot, const void* sink, float scale, float eps,
-                                        void* k_cache, void* v_cache, int capacity, int window, const int* position_ptr, int position,
-                                        float* partial, unsigned int* counters, int splits, void* out, int heads, int kv_heads,
-                                        int dim, int vdim, int dtype, void* stream) {
-    QD_ATTN_ARGS_OK(partial && counters && splits > 0 && splits <= qd::kStepKeys && qd::aligned16(partial));
-    const qd::AttnStep sp = {{q, k, v, gate, 0, (const bf16*)q_norm, (const bf16*)k_norm, freq, rot, (const bf16*)sink, scale, eps, k_cache,
-                              v_cache, capacity, window, position_ptr, position, nullptr, out, 1, heads, kv_heads, dim, vdim},
-                             partial, counters, splits, 2};
-    if (dtype == QD_BF16) return qd::step<bf16>(sp, (cudaStream_t)stream);
-    if (dtype == QD_F32) return qd::step<float>(sp, (cudaStream_t)stream);
+extern "C" int qd_attention_step(const qd_attention_args* args, void* stream) {
+    QD_CHECK_ARG(args && qd::valid(*args) && args->q && args->partial && args->counters && args->capacity >= args->span);
+    QD_CHECK_ARG(args->splits > 0 && args->splits <= qd::kStepKeys && qd::aligned16(args->partial));
+    if (args->dtype == QD_BF16) return qd::step<bf16>(*args, (cudaStream_t)stream);
+    if (args->dtype == QD_F32) return qd::step<float>(*args, (cudaStream_t)stream);
     return QD_ERR_UNSUPPORTED;
 }

@@ -17,7 +17,7 @@ the history and what advances it.  ``extend`` continues the current request by g
 returns the logits at chosen places (a replayed trace, a scored continuation).
 
 Backends: ``"b200"`` (default) runs the fused CUDA step where the checkpoint has the
-36B-A3B widths (or is a bf16-weight hybrid) and the composed operator table otherwise; passing ``kernels=`` or
+36B-A3B widths (or belongs to a bf16-weight design) and the composed operator table otherwise; passing ``kernels=`` or
 ``step=`` gives the ``"custom"`` backend used by tests (no graph).  There is no CPU
 backend: on a CPU device only a caller-supplied ``step`` can run.
 """
@@ -29,7 +29,7 @@ from dataclasses import dataclass
 import torch
 
 from .registry import design_of, design_of_directory
-from .weights import Checkpoint, FezopelCheckpoint
+from .weights import Checkpoint, DokulixCheckpoint, FezopelCheckpoint
 
 
 @dataclass
@@ -51,7 +51,7 @@ class Snapshot:
 
 
 class Engine:
-    def __init__(self, ckpt: Checkpoint | FezopelCheckpoint, max_context: int = 32768, device: str = "cuda",
+    def __init__(self, ckpt: Checkpoint | FezopelCheckpoint | DokulixCheckpoint, max_context: int = 32768, device: str = "cuda",
                  backend: str | None = None, *, kernels: dict | None = None, step=None,
                  cuda_graph: bool = True, prefill_chunk_size: int = 2048,
                  sequence_prefill: bool = True, dtype: torch.dtype = torch.bfloat16, _step_object=None):
@@ -82,10 +82,9 @@ class Engine:
             assert on_cuda, "the b200 backend needs a CUDA device; there is no CPU path"
             from . import fused
             from .kernels import bind_kernels
-            if design.library == "hybrid":
+            if design.model is not None:
                 assert kernels is None, "the operator table is for NVFP4 checkpoints"
-                from .hybrid import HybridModel
-                self.fused = self.step = self.chunk_prefill = HybridModel(ckpt, dtype)
+                self.fused = self.step = self.chunk_prefill = design.model(ckpt, dtype)
                 self.sequence_prefill = sequence_prefill
             elif kernels is None and fused.supports(ckpt):
                 self.fused = fused.FusedStep(ckpt)

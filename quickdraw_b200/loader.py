@@ -26,9 +26,10 @@ from pathlib import Path
 
 import torch
 
-from .weights import (ChannelDeltaConfig, ChannelDeltaWeights, Checkpoint, FezopelCheckpoint, FezopelConfig, FP8Linear,
-                      FullAttnWeights, GDNWeights, GeluMLPWeights, GLAConfig, GLAWeights, HybridLayerWeights, LayerWeights,
-                      ModelConfig, MoEWeights, NormWeights, NVFP4Linear, SublayerWeights, WindowAttnConfig, WindowAttnWeights)
+from .weights import (ChannelDeltaConfig, ChannelDeltaWeights, Checkpoint, ChunkAttnConfig, ChunkAttnWeights, DokulixCheckpoint,
+                      DokulixConfig, FezopelCheckpoint, FezopelConfig, FP8Linear, FullAttnWeights, GDNWeights, GeluMLPWeights, GLAConfig,
+                      GLAWeights, HybridLayerWeights, LatentAttnConfig, LatentAttnWeights, LayerWeights, ModelConfig, MoEWeights, NormWeights,
+                      NVFP4Linear, PreNormLayerWeights, ReGLUWeights, SublayerWeights, WindowAttnConfig, WindowAttnWeights)
 
 ROOT = "model.language_model."
 LAYER_NAME = re.compile(r"model\.language_model\.layers\.(\d+)\.")
@@ -285,12 +286,18 @@ HYBRID_FIELDS = {
     WindowAttnConfig: (WindowAttnWeights, {"q_norm": "q.norm", "k_norm": "k.norm"}),
     GLAConfig: (GLAWeights, {"a2_b": "a2.b"}),
     ChannelDeltaConfig: (ChannelDeltaWeights, {"q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv"}),
+    ChunkAttnConfig: (ChunkAttnWeights, {"q_norm": "q.norm", "k_norm": "k.norm", "q_b": "q.b", "k_b": "k.b", "v_b": "v.b", "o_b": "o.b"}),
+    LatentAttnConfig: (LatentAttnWeights, {"dq_norm": "dq.norm", "dkv_norm": "dkv.norm"}),
 }
 
 
-def hybrid_shapes(config: FezopelConfig, low_rank=lambda name: None) -> dict[str, tuple]:
-    """Every tensor name of the checkpoint and its shape; None where only the tensor knows it (the
-    inner size of the low-rank products, unless ``low_rank(name of the inner matrix)`` tells)."""
+def _mixer_of(cfg, at: str, get):
+    """A mixer's container from the tensors below ``<at>mix.``."""
+    container, renamed = HYBRID_FIELDS[type(cfg)]
+    return container(**{f.name: get(at + "mix." + renamed.get(f.name, f.name)) for f in fields(container)})
+
+
+def fezopel_shapes(config: FezopelConfig, low_rank=lambda name: None) -> dict[str, tuple]:
     w = config.hidden_size
     shapes: dict[str, tuple] = {"embed": (config.vocab_size, w), "head": (config.vocab_size, w)}
 
@@ -327,29 +334,78 @@ def hybrid_shapes(config: FezopelConfig, low_rank=lambda name: None) -> dict[str
     return shapes
 
 
-def assemble_hybrid(config: FezopelConfig, get) -> FezopelCheckpoint:
-    """The containers from ``get(tensor name)``."""
+def assemble_fezopel(config: FezopelConfig, get) -> FezopelCheckpoint:
     norm = lambda name: NormWeights(get(name), get(name + ".b"))
     around = lambda at, which: SublayerWeights(norm(f"{at}norm{which}"), get(f"{at}rg{which}"), get(f"{at}rg{which}.b"),
                                                norm(f"{at}norm{which}b"))
     layers = []
     for i, layer in enumerate(config.layers):
-        at = f"l{i}."
-        container, renamed = HYBRID_FIELDS[type(layer.mixer)]
-        mixer = container(**{f.name: get(at + "mix." + renamed.get(f.name, f.name)) for f in fields(container)})
-        has_mlp = layer.ff is not None
+        at, has_mlp = f"l{i}.", layer.ff is not None
         layers.append(HybridLayerWeights(
-            idx=i, mixer=mixer, around_mixer=around(at, "1"), depth=get(at + "dwa"),
+            idx=i, mixer=_mixer_of(layer.mixer, at, get), around_mixer=around(at, "1"), depth=get(at + "dwa"),
             mlp=GeluMLPWeights(get(at + "mlp.up"), get(at + "mlp.down")) if has_mlp else None,
             around_mlp=around(at, "2") if has_mlp else None))
     return FezopelCheckpoint(config=config, embed_tokens=get("embed"), final_norm=norm("final.norm"), lm_head=get("head"),
                              layers=layers)
 
 
-def load_hybrid_checkpoint(path: str | Path, device: str | torch.device = "cuda") -> FezopelCheckpoint:
+def dokulix_shapes(config: DokulixConfig, low_rank=None) -> dict[str, tuple]:
+    w = config.hidden_size
+    shapes: dict[str, tuple] = {"embed": (config.vocab_size, w), "head": (config.vocab_size, w), "final.norm": (w,)}
+    if config.loop is not None:
+        shapes["loop.step"] = (config.loop.times, w)
+    for i, layer in enumerate(config.layers):
+        at, m = f"l{i}.", layer.mixer
+        shapes[at + "norm1"] = (w,)
+        if layer.ff is not None:
+            shapes |= {at + "norm2": (w,), at + "mlp.gate": (layer.ff, w), at + "mlp.up": (layer.ff, w), at + "mlp.down": (w, layer.ff)}
+        keys, values = m.heads * m.dim, m.heads * m.vdim
+        if isinstance(m, LatentAttnConfig):
+            own = {"dq": (m.q_rank, w), "dq.norm": (m.q_rank,), "uq": (m.heads * (m.dim + m.rot_dim), m.q_rank),
+                   "dkv": (m.kv_rank + m.rot_dim, w), "dkv.norm": (m.kv_rank,), "uk": (keys, m.kv_rank), "uv": (values, m.kv_rank),
+                   "g": (values, w), "o": (w, values)}
+        else:
+            kv_keys, kv_values = m.kv_heads * m.dim, m.kv_heads * m.vdim
+            own = {"q": (keys, w), "q.b": (keys,), "k": (kv_keys, w), "k.b": (kv_keys,), "v": (kv_values, w), "v.b": (kv_values,),
+                   "q.norm": (m.dim,), "k.norm": (m.dim,), "o": (w, values), "o.b": (w,)}
+        shapes.update({at + "mix." + name: shape for name, shape in own.items()})
+    return shapes
+
+
+def assemble_dokulix(config: DokulixConfig, get) -> DokulixCheckpoint:
+    layers = []
+    for i, layer in enumerate(config.layers):
+        at, has_mlp = f"l{i}.", layer.ff is not None
+        layers.append(PreNormLayerWeights(
+            idx=i, mixer=_mixer_of(layer.mixer, at, get), norm1=get(at + "norm1"), norm2=get(at + "norm2") if has_mlp else None,
+            mlp=ReGLUWeights(*(get(f"{at}mlp.{name}") for name in ("gate", "up", "down"))) if has_mlp else None))
+    return DokulixCheckpoint(config=config, embed_tokens=get("embed"), final_norm=get("final.norm"), lm_head=get("head"), layers=layers,
+                             loop_steps=None if config.loop is None else get("loop.step"))
+
+
+# configuration -> (names and shapes, containers)
+HYBRID_LAYOUTS = {FezopelConfig: (fezopel_shapes, assemble_fezopel), DokulixConfig: (dokulix_shapes, assemble_dokulix)}
+
+
+def hybrid_shapes(config, low_rank=lambda name: None) -> dict[str, tuple]:
+    """Every tensor name of the checkpoint and its shape; None where only the tensor knows it (the
+    inner size of the low-rank products, unless ``low_rank(name of the inner matrix)`` tells)."""
+    return HYBRID_LAYOUTS[type(config)][0](config, low_rank)
+
+
+def assemble_hybrid(config, get):
+    """The containers from ``get(tensor name)``."""
+    return HYBRID_LAYOUTS[type(config)][1](config, get)
+
+
+def load_hybrid_checkpoint(path: str | Path, device: str | torch.device = "cuda") -> FezopelCheckpoint | DokulixCheckpoint:
     """A directory with ``config.json`` and safetensors (one file, or shards with an index)."""
     directory = Path(path)
-    config = FezopelConfig.from_json(directory / "config.json")
+    data = json.loads((directory / "config.json").read_text())
+    kind = next((kind for kind in HYBRID_LAYOUTS if kind.ARCHITECTURE == data.get("architecture")), None)
+    if kind is None:
+        raise ValueError(f"{directory}: no bf16-weight design {data.get('architecture')!r}")
+    config = kind.from_dict(data)
     with ExitStack() as stack:
         reader = ShardReader(directory, stack)
         for name, shape in hybrid_shapes(config).items():
@@ -361,7 +417,7 @@ def load_hybrid_checkpoint(path: str | Path, device: str | torch.device = "cuda"
         return assemble_hybrid(config, lambda name: reader.tensor(name).to(device=device, dtype=torch.bfloat16).contiguous())
 
 
-def save_hybrid_checkpoint(config: FezopelConfig, tensors: dict[str, torch.Tensor], path: str | Path) -> None:
+def save_hybrid_checkpoint(config, tensors: dict[str, torch.Tensor], path: str | Path) -> None:
     """Write ``config.json`` and ``model.safetensors`` as ``load_hybrid_checkpoint`` reads them."""
     from safetensors.torch import save_file
     directory = Path(path)

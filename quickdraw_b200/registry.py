@@ -12,19 +12,20 @@ from typing import Callable
 import torch
 
 from .state import DecodeState, HybridState
-from .weights import Checkpoint, FezopelCheckpoint, FezopelConfig
+from .weights import Checkpoint, DokulixCheckpoint, DokulixConfig, FezopelCheckpoint, FezopelConfig
 
 
 @dataclass(frozen=True)
 class Design:
     name: str
-    library: str                                  # build target of its kernels
+    libraries: tuple[str, ...]                    # build targets of its kernels
     checkpoint: type
     matches: Callable[[dict], bool]               # on the parsed config.json
     load: Callable                                # (directory, device) -> checkpoint
     allocate: Callable                            # (config, max_context, device, chunk, dtype) -> state
     dtypes: tuple[torch.dtype, ...]               # activation types it runs in
     chunk_logits: bool                            # whether a chunk returns the logits of its tokens
+    model: Callable | None = None                 # (checkpoint, dtype) -> what advances a state by one token and by a chunk
 
 
 def _load_qwen(path, device):
@@ -39,12 +40,27 @@ def _load_hybrid(path, device):
     return load_hybrid_checkpoint(path, device=device)
 
 
+def _fezopel(ckpt, dtype):
+    from .hybrid import FezopelModel
+    return FezopelModel(ckpt, dtype)
+
+
+def _dokulix(ckpt, dtype):
+    from .hybrid import DokulixModel
+    return DokulixModel(ckpt, dtype)
+
+
+def _hybrid(name: str, libraries, checkpoint: type, config: type, model) -> Design:
+    return Design(name, libraries, checkpoint, lambda data: data.get("architecture") == config.ARCHITECTURE, _load_hybrid,
+                  lambda cfg, max_context, device, chunk, dtype: HybridState(cfg, max_context, device, chunk, dtype),
+                  (torch.bfloat16, torch.float32), True, model)
+
+
 DESIGNS = (
-    Design("qwen3-next", "nvfp4", Checkpoint, lambda data: "text_config" in data, _load_qwen,
+    Design("qwen3-next", ("nvfp4",), Checkpoint, lambda data: "text_config" in data, _load_qwen,
            lambda config, max_context, device, chunk, dtype: DecodeState.allocate(config, max_context, device), (torch.bfloat16,), False),
-    Design("fezopel", "hybrid", FezopelCheckpoint, lambda data: data.get("architecture") == FezopelConfig.ARCHITECTURE, _load_hybrid,
-           lambda config, max_context, device, chunk, dtype: HybridState(config, max_context, device, chunk, dtype),
-           (torch.bfloat16, torch.float32), True),
+    _hybrid("fezopel", ("hybrid", "recurrent"), FezopelCheckpoint, FezopelConfig, _fezopel),
+    _hybrid("dokulix", ("hybrid", "latent"), DokulixCheckpoint, DokulixConfig, _dokulix),
 )
 
 

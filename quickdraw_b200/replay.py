@@ -34,7 +34,7 @@ def main() -> int:
     if dtype not in design.dtypes:
         print(f"{design.name} does not run in {args.dtype}", file=sys.stderr)
         return 3
-    build.build(targets=(design.library,))
+    build.build(targets=design.libraries)
     out = Path(args.out)
     engine = Engine.from_pretrained(args.model, max_context=max(1, args.max_tokens), device="cuda", dtype=dtype)
     live = None

@@ -61,19 +61,20 @@ class DecodeState:
 
 @dataclass
 class LayerHistory:
-    """One layer's views: ``k``, ``v`` [capacity, kv_heads, dim / vdim] (attention), ``rec`` fp32
-    [heads, dim, vdim], ``conv`` [taps, channels] (position p in row p mod taps)."""
+    """One layer's views: ``k``, ``v`` [capacity, kv_heads, dim / vdim] (attention), ``latent`` [capacity, row]
+    (latent attention), ``rec`` fp32 [heads, dim, vdim], ``conv`` [taps, channels] (position p in row p mod taps)."""
     k: torch.Tensor | None = None
     v: torch.Tensor | None = None
+    latent: torch.Tensor | None = None
     rec: torch.Tensor | None = None
     conv: torch.Tensor | None = None
 
 
 class HybridState:
-    """History of one request of a bf16-weight hybrid.  An attention layer keeps the last ``capacity``
-    positions, position p in row p mod capacity: the window plus the rows a prompt chunk of ``chunk``
-    tokens adds before its first token has attended.  Rows are only read for positions of the current
-    request, so a reset leaves them."""
+    """History of one request of a bf16-weight hybrid, one entry of ``layers`` for every layer run (a looped layer
+    has one per pass).  An attention layer keeps the last ``capacity`` positions, position p in row p mod
+    capacity: the span a query sees plus the rows a prompt chunk of ``chunk`` tokens adds before its first
+    token has attended.  Rows are only read for positions of the current request, so a reset leaves them."""
 
     keeps_every_row = False
 
@@ -89,10 +90,12 @@ class HybridState:
             sizes[buffer] += -(-count // 64) * 64            # every view starts on a 128-byte boundary
             return buffer, start, count, shape
 
-        for layer in config.layers:
-            m, plan = layer.mixer, {}
-            if hasattr(m, "window"):
-                capacity = min(max_context, m.window - 1 + chunk)
+        for index, _ in config.runs():
+            m, plan = config.layers[index].mixer, {}
+            capacity = min(max_context, m.span - 1 + chunk) if hasattr(m, "span") else 0
+            if hasattr(m, "kv_rank"):
+                plan["latent"] = take("kv_k", capacity, m.row)
+            elif hasattr(m, "span"):
                 plan["k"] = take("kv_k", capacity, m.kv_heads, m.dim)
                 plan["v"] = take("kv_v", capacity, m.kv_heads, m.vdim)
             else:

@@ -181,6 +181,55 @@ class WindowAttnConfig:
     rotary_base: float
     scale: float
 
+    @property
+    def span(self) -> int:
+        """The most positions a query sees: rows a cache has to keep."""
+        return self.window
+
+
+@dataclass
+class ChunkAttnConfig:
+    """Attention within chunks of ``span`` positions counted from 0, with a penalty slope * distance per head and one
+    added to the softmax's denominator."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    span: int
+    scale: float
+
+    def slopes(self) -> list[float]:
+        return [2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads)]
+
+
+@dataclass
+class LatentAttnConfig:
+    """Sliding-window attention whose queries, keys and values are expanded from latents; ``dim`` columns per head
+    without and ``rot_dim`` with rotary positions, the latter shared by all keys of a token."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    window: int
+    rotary_base: float
+    scale: float
+
+    @property
+    def span(self) -> int:
+        return self.window
+
+    @property
+    def rot_column(self) -> int:
+        """First rotated column of a cache row: behind the latent, on a 16-byte boundary."""
+        return -(-self.kv_rank // 8) * 8
+
+    @property
+    def row(self) -> int:
+        """Elements of a cache row (a multiple of sixteen)."""
+        return -(-(self.rot_column + self.rot_dim) // 16) * 16
+
 
 @dataclass
 class GLAConfig:
@@ -212,6 +261,33 @@ class WindowAttnWeights:
     q_norm: torch.Tensor
     k_norm: torch.Tensor
     sink: torch.Tensor
+
+
+@dataclass
+class ChunkAttnWeights:
+    q: torch.Tensor
+    q_b: torch.Tensor
+    k: torch.Tensor
+    k_b: torch.Tensor
+    v: torch.Tensor
+    v_b: torch.Tensor
+    q_norm: torch.Tensor
+    k_norm: torch.Tensor
+    o: torch.Tensor
+    o_b: torch.Tensor
+
+
+@dataclass
+class LatentAttnWeights:
+    dq: torch.Tensor
+    dq_norm: torch.Tensor
+    uq: torch.Tensor
+    dkv: torch.Tensor
+    dkv_norm: torch.Tensor
+    uk: torch.Tensor
+    uv: torch.Tensor
+    g: torch.Tensor
+    o: torch.Tensor
 
 
 @dataclass
@@ -294,6 +370,10 @@ class FezopelConfig:
 
     ARCHITECTURE = "Fezopel"
 
+    def runs(self) -> list[tuple[int, None]]:
+        """(layer, no pass of a loop), in the order they run."""
+        return [(i, None) for i in range(len(self.layers))]
+
     @classmethod
     def from_json(cls, path: str | Path) -> "FezopelConfig":
         return cls.from_dict(json.loads(Path(path).read_text()))
@@ -354,6 +434,120 @@ class FezopelCheckpoint:
     final_norm: NormWeights
     lm_head: torch.Tensor
     layers: list[HybridLayerWeights]
+
+
+@dataclass
+class ReGLUWeights:
+    """down(relu(gate h) * (up h))."""
+    gate: torch.Tensor
+    up: torch.Tensor
+    down: torch.Tensor
+
+
+@dataclass
+class PreNormLayerWeights:
+    """RMS norms in front of the mixer and the feed-forward, stored as their distance from one."""
+    idx: int
+    mixer: LatentAttnWeights | ChunkAttnWeights
+    norm1: torch.Tensor
+    mlp: ReGLUWeights | None
+    norm2: torch.Tensor | None
+
+
+@dataclass
+class PreNormLayerConfig:
+    mixer: LatentAttnConfig | ChunkAttnConfig
+    ff: int | None
+
+
+@dataclass
+class LoopConfig:
+    """Layers start .. stop - 1 run ``times`` times in a row with the same weights and a history of their own each time."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass
+class DokulixConfig:
+    vocab_size: int
+    hidden_size: int
+    norm_eps: float
+    layers: list[PreNormLayerConfig]
+    loop: LoopConfig | None = None
+
+    ARCHITECTURE = "Dokulix"
+
+    def runs(self) -> list[tuple[int, int | None]]:
+        """(layer, the pass that begins with it or None), in the order they run."""
+        if self.loop is None:
+            return [(i, None) for i in range(len(self.layers))]
+        start, stop = self.loop.start, self.loop.stop
+        looped = [(i, t if i == start else None) for t in range(self.loop.times) for i in range(start, stop)]
+        return [(i, None) for i in range(start)] + looped + [(i, None) for i in range(stop, len(self.layers))]
+
+    @classmethod
+    def from_json(cls, path: str | Path) -> "DokulixConfig":
+        return cls.from_dict(json.loads(Path(path).read_text()))
+
+    @classmethod
+    def from_dict(cls, data: dict) -> "DokulixConfig":
+        if data.get("architecture") != cls.ARCHITECTURE:
+            raise ValueError(f"not a {cls.ARCHITECTURE} configuration: {data.get('architecture')!r}")
+        layers = []
+        for index, entry in enumerate(data["layers"]):
+            m, kind = entry["mixer"], entry["type"]
+            if kind == "latent_attention":
+                mixer = LatentAttnConfig(heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], q_rank=m["q_rank"],
+                                         kv_rank=m["kv_rank"], window=m["mask"]["size"], rotary_base=float(m["rot"]["base"]),
+                                         scale=float(m["scale"]))
+                if m["rot"]["dims"] != mixer.rot_dim or mixer.rot_dim % 2:
+                    raise ValueError(f"layer {index}: {m['rot']['dims']} rotated dimensions of {mixer.rot_dim}")
+            elif kind == "attention":
+                mixer = ChunkAttnConfig(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], span=m["mask"]["size"],
+                                        scale=float(m["scale"]))
+                if mixer.heads % mixer.kv_heads:
+                    raise ValueError(f"layer {index}: {mixer.heads} heads do not divide among {mixer.kv_heads} key/value heads")
+            else:
+                raise ValueError(f"layer {index}: unknown mixer {kind!r}")
+            mlp = entry["mlp"]
+            if mlp is not None and mlp["kind"] != "dense":
+                raise ValueError(f"layer {index}: unknown feed-forward {mlp['kind']!r}")
+            layers.append(PreNormLayerConfig(mixer=mixer, ff=None if mlp is None else mlp["ff"]))
+        loop = data.get("loop")
+        if loop is not None:
+            loop = LoopConfig(start=loop["start"], stop=loop["stop"], times=loop["times"])
+            if not 0 <= loop.start < loop.stop <= len(layers) or loop.times < 0:
+                raise ValueError(f"loop over layers {loop.start} .. {loop.stop} of {len(layers)}, {loop.times} times")
+        return cls(vocab_size=data["vocab"], hidden_size=data["width"], norm_eps=float(data["norm"]["eps"]), layers=layers, loop=loop)
+
+    def to_dict(self) -> dict:
+        """The ``config.json`` this configuration reads from."""
+        layers = []
+        for layer in self.layers:
+            m = layer.mixer
+            entry = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "mask": {"size": m.span}, "scale": m.scale}
+            if isinstance(m, LatentAttnConfig):
+                kind = "latent_attention"
+                entry |= {"rot_dim": m.rot_dim, "q_rank": m.q_rank, "kv_rank": m.kv_rank,
+                          "rot": {"base": m.rotary_base, "dims": m.rot_dim}}
+            else:
+                kind = "attention"
+                entry |= {"kv_heads": m.kv_heads}
+            layers.append({"type": kind, "mixer": entry, "mlp": None if layer.ff is None else {"kind": "dense", "ff": layer.ff}})
+        loop = None if self.loop is None else {"start": self.loop.start, "stop": self.loop.stop, "times": self.loop.times}
+        return {"architecture": self.ARCHITECTURE, "vocab": self.vocab_size, "width": self.hidden_size,
+                "norm": {"eps": self.norm_eps}, "loop": loop, "layers": layers}
+
+
+@dataclass
+class DokulixCheckpoint:
+    config: DokulixConfig
+    embed_tokens: torch.Tensor
+    final_norm: torch.Tensor
+    lm_head: torch.Tensor
+    layers: list[PreNormLayerWeights]
+    loop_steps: torch.Tensor | None          # [times, width]: added to the stream in front of every pass
 
 
 CONTAINERS = {cls.__name__: cls for cls in (

@@ -360,12 +360,12 @@ def test_prompts_portions_and_decoding_give_the_oracle_s_logits(cuda_device, nam
 
 
 def test_the_stream_after_every_layer(cuda_device):
-    from quickdraw_b200.hybrid import HybridModel
+    from quickdraw_b200.hybrid import FezopelModel
     cfg, tensors, ckpt = build("mixed")
     tokens = cases.prompt(cfg, 30)
     _, want = O.forward(cfg.to_dict(), tensors, tokens)
     record = []
-    HybridModel(ckpt, F32).run(torch.tensor(tokens, device="cuda"), 0, HybridState(cfg, 64, "cuda", dtype=F32), [29], record)
+    FezopelModel(ckpt, F32).run(torch.tensor(tokens, device="cuda"), 0, HybridState(cfg, 64, "cuda", dtype=F32), [29], record)
     for got, layer in zip(record, want):
         assert error(got, layer) < 1e-5
 

@@ -107,25 +107,50 @@ def declarations():
 def test_hybrid_bindings_follow_the_header():
     kinds = {ctypes.c_void_p: "pointer", ctypes.c_int: "int", ctypes.c_float: "float", ctypes.c_longlong: "long long"}
     found = declarations()
-    assert {name for _, name, _ in found} | {"qd_set_chained_launches"} == set(_lib.HYBRID_SIGNATURES)
+    signatures = {name: kinds for names in _lib.HYBRID_LIBRARIES.values() for name, kinds in names.items()}
+    assert {name for _, name, _ in found} | {"qd_set_chained_launches"} == set(signatures)
     for result, name, params in found:
         declared = ["pointer" if "*" in p else re.sub(r"\s+\w+$", "", p.strip()) for p in params.split(",")]
-        assert [kinds[t] for t in _lib.HYBRID_SIGNATURES[name]] == declared, name
+        assert [kinds[t] for t in signatures[name]] == declared, name
         assert (name in _lib.HYBRID_LONG_RESULTS) == (result == "long long"), name
 
 
-def test_hybrid_library_exports_what_the_header_declares():
-    handle = _lib.hybrid_lib()
-    for name in _lib.HYBRID_SIGNATURES:
-        assert hasattr(handle, name), name
-    assert handle.qd_error_string(4) == b"shape not covered by this kernel"
+def test_structures_follow_the_header():
+    """Field by field: names, order and types (pointers first, so that there is no padding between them)."""
+    kinds = {ctypes.c_void_p: "pointer", ctypes.c_int: "int", ctypes.c_float: "float", ctypes.c_longlong: "long long"}
+    text = re.sub(r"/\*.*?\*/", "", HEADER.read_text(), flags=re.S)
+    found = re.findall(r"typedef struct (\w+) \{(.*?)\} \1;", text, flags=re.S)
+    assert {name for name, _ in found} == set(_lib.STRUCTURES)
+    for name, body in found:
+        declared = []
+        for line in filter(None, (part.strip() for part in body.split(";"))):
+            kind, names = re.match(r"(const void\*|void\*|const float\*|float\*|const int\*|unsigned int\*|long long|float|int)\s+(.*)", line, re.S).groups()
+            declared += [(field.strip(), "pointer" if kind.endswith("*") else kind) for field in names.split(",")]
+        assert [(field, kinds[kind]) for field, kind in _lib.STRUCTURES[name]._fields_] == declared, name
+
+
+def test_hybrid_libraries_export_what_the_header_declares():
+    for target, names in _lib.HYBRID_LIBRARIES.items():
+        handle = _lib.hybrid_lib(target)
+        for name in names:
+            assert hasattr(handle, name), name
+        assert handle.qd_error_string(4) == b"shape not covered by this kernel"
+
+
+def test_every_source_belongs_to_one_library():
+    from quickdraw_b200 import build
+    owned = [path.stem for target in build.TARGETS for path in build.sources(target) if path.stem not in build.COMMON]
+    everything = sorted(path.stem for path in build.CSRC.glob("*.cu"))
+    assert sorted(owned + [name for name in build.COMMON]) == everything
+    assert {t for design in registry.DESIGNS for t in design.libraries} == set(build.TARGETS)
 
 
 def test_missing_hybrid_library_fails_loudly(monkeypatch, tmp_path):
-    monkeypatch.setattr(_lib, "_hybrid", None)
-    monkeypatch.setattr(_lib, "HYBRID_PATH", tmp_path / "libquickdraw_b200_hybrid.so")
-    with pytest.raises(_lib.LibraryMissing, match="build hybrid"):
-        _lib.hybrid_lib()
+    monkeypatch.setattr(_lib, "_hybrid", {})
+    monkeypatch.setattr(_lib, "LIB_PATH", tmp_path / "libquickdraw_b200.so")
+    for target in _lib.HYBRID_LIBRARIES:
+        with pytest.raises(_lib.LibraryMissing, match=f"build {target}"):
+            _lib.hybrid_lib(target)
 
 
 class AsIfOnGpu(torch.Tensor):
@@ -138,12 +163,9 @@ def recorder(monkeypatch):
     seen = []
 
     def record(name, *args):
-        assert len(args) == len(_lib.HYBRID_SIGNATURES[name]), (name, len(args), len(_lib.HYBRID_SIGNATURES[name]))
+        declared = _lib.HYBRID_LIBRARIES[_lib.HYBRID_OWNER[name]][name]
+        assert len(args) == len(declared), (name, len(args), len(declared))
         seen.append((name, args))
-
-    class FakeLibrary:
-        def __getattr__(self, name):
-            return lambda *args: 4096
 
     class Properties:
         multi_processor_count = 148
@@ -151,7 +173,7 @@ def recorder(monkeypatch):
     for module in (hybrid, mixers):
         monkeypatch.setattr(module, "call_hybrid", record)
         monkeypatch.setattr(module, "stream_of", lambda t: None)
-    monkeypatch.setattr(mixers, "hybrid_lib", lambda: FakeLibrary())
+    monkeypatch.setattr(mixers, "size_hybrid", lambda name, *args: 4096)
     monkeypatch.setattr(torch.cuda, "get_device_properties", lambda device: Properties)
     return seen
 
@@ -161,14 +183,14 @@ def recorder(monkeypatch):
 def test_drivers_pass_the_declared_number_of_arguments(recorder, name, tokens):
     cfg = cases.MODELS[name]()
     ckpt = synthetic.make_fezopel(cfg)
-    model, state = hybrid.HybridModel(ckpt), HybridState(cfg, 64, "cpu")
+    model, state = hybrid.FezopelModel(ckpt), HybridState(cfg, 64, "cpu")
     ids = torch.arange(tokens).as_subclass(AsIfOnGpu)
     logits = model.run(ids, 3, state, [0, tokens - 1])
     assert logits.shape == (2, cfg.vocab_size) and logits.dtype == torch.float32
     names = [n for n, _ in recorder]
     assert names.count("qd_sublayer_close") == sum(1 + (layer.ff is not None) for layer in cfg.layers)
     windowed = sum(isinstance(layer.mixer, WindowAttnConfig) for layer in cfg.layers)
-    assert names.count("qd_window_attention" if tokens > 1 else "qd_window_attention_step") == windowed
+    assert names.count("qd_attention" if tokens > 1 else "qd_attention_step") == windowed
     recorder.clear()
     assert model.run(ids, 3, state) is None                       # nothing wanted: it ends behind the last mixer
     assert [n for n, _ in recorder].count("qd_layer_norm_rows") == 0
@@ -180,7 +202,7 @@ def test_drivers_pass_the_declared_number_of_arguments(recorder, name, tokens):
 
 def test_stacked_matrices_start_on_multiples_of_eight_rows():
     parts = {"a": torch.randn(5, 4), "b": torch.randn(8, 4), "c": torch.randn(1, 4)}
-    matrix, at = hybrid.stack_rows(parts)
+    matrix, at = mixers.stack_rows(parts)
     assert at == {"a": 0, "b": 8, "c": 16} and matrix.shape == (24, 4)
     for name, part in parts.items():
         assert torch.equal(matrix[at[name]:at[name] + part.shape[0]], part)
@@ -274,7 +296,7 @@ def replayed(monkeypatch, capsys, tmp_path, steps, dtype="bfloat16"):
                                       "--max-tokens", "16"])
     monkeypatch.setattr(sys, "stdin", io.StringIO("".join(json.dumps(s) + "\n" for s in steps)))
     code = replay.main()
-    assert built == [("hybrid",)] and engines[0].dtype == getattr(torch, dtype)
+    assert built == [("hybrid", "recurrent")] and engines[0].dtype == getattr(torch, dtype)
     return code, capsys.readouterr().out.split("\n"), cfg.vocab_size
 
 
