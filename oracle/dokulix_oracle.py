@@ -80,31 +80,38 @@ def masked_attention(q, k, v, scale, sees, slopes=None, extra_one=False):
     return out
 
 
-def latent_attention_mixer(h, w, prefix, m, eps):
+def latent_heads(dq, dkv, w, prefix, m, eps):
+    """Heads [T, H, vdim] from the rows of the two down projections."""
     heads, dim, rot_dim, vdim, rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
-    tokens, positions = h.shape[0], torch.arange(h.shape[0])
-    compressed = rms_norm(h @ w[prefix + "dq"].T, w[prefix + "dq.norm"], eps)
-    q = (compressed @ w[prefix + "uq"].T).view(tokens, heads, dim + rot_dim)
+    tokens, positions = dq.shape[0], torch.arange(dq.shape[0])
+    q = (rms_norm(dq, w[prefix + "dq.norm"], eps) @ w[prefix + "uq"].T).view(tokens, heads, dim + rot_dim)
     q = torch.cat([q[..., :dim], rotate_half(q[..., dim:], positions, m["rot"]["base"], m["rot"]["dims"])], -1)
-    down = h @ w[prefix + "dkv"].T
-    latent = rms_norm(down[:, :rank], w[prefix + "dkv.norm"], eps)
-    shared = rotate_half(down[:, rank:], positions, m["rot"]["base"], m["rot"]["dims"])
+    latent = rms_norm(dkv[:, :rank], w[prefix + "dkv.norm"], eps)
+    shared = rotate_half(dkv[:, rank:], positions, m["rot"]["base"], m["rot"]["dims"])
     keys = (latent @ w[prefix + "uk"].T).view(tokens, heads, dim)
     k = torch.cat([keys, shared[:, None].expand(tokens, heads, rot_dim)], -1)
     v = (latent @ w[prefix + "uv"].T).view(tokens, heads, vdim)
     size = m["mask"]["size"]
-    out = masked_attention(q, k, v, m["scale"], lambda i, j: sees_window(i, j, size)).reshape(tokens, heads * vdim)
+    return masked_attention(q, k, v, m["scale"], lambda i, j: sees_window(i, j, size))
+
+
+def latent_attention_mixer(h, w, prefix, m, eps):
+    out = latent_heads(h @ w[prefix + "dq"].T, h @ w[prefix + "dkv"].T, w, prefix, m, eps).flatten(1)
     return (out * torch.sigmoid(h @ w[prefix + "g"].T)) @ w[prefix + "o"].T
 
 
-def attention_mixer(h, w, prefix, m, eps):
-    heads, kv, dim, vdim, tokens = m["heads"], m["kv_heads"], m["dim"], m["vdim"], h.shape[0]
-    q, k, v = (h @ w[prefix + n].T + w[prefix + n + ".b"] for n in "qkv")
+def chunk_heads(q, k, v, w, prefix, m, eps):
+    """Heads [T, H, vdim] from the projections (biases added)."""
+    heads, kv, dim, vdim, tokens = m["heads"], m["kv_heads"], m["dim"], m["vdim"], q.shape[0]
     q = rms_norm(q.view(tokens, heads, dim), w[prefix + "q.norm"], eps)
     k = rms_norm(k.view(tokens, kv, dim), w[prefix + "k.norm"], eps)
     size = m["mask"]["size"]
-    out = masked_attention(q, k, v.view(tokens, kv, vdim), m["scale"], lambda i, j: sees_chunk(i, j, size), distance_slopes(heads), True)
-    return out.reshape(tokens, heads * vdim) @ w[prefix + "o"].T + w[prefix + "o.b"]
+    return masked_attention(q, k, v.view(tokens, kv, vdim), m["scale"], lambda i, j: sees_chunk(i, j, size), distance_slopes(heads), True)
+
+
+def attention_mixer(h, w, prefix, m, eps):
+    q, k, v = (h @ w[prefix + n].T + w[prefix + n + ".b"] for n in "qkv")
+    return chunk_heads(q, k, v, w, prefix, m, eps).flatten(1) @ w[prefix + "o"].T + w[prefix + "o.b"]
 
 
 MIXERS = {"latent_attention": latent_attention_mixer, "attention": attention_mixer}

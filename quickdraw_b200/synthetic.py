@@ -18,8 +18,9 @@ import zlib
 
 import torch
 
-from .weights import (ChannelDeltaConfig, Checkpoint, FezopelCheckpoint, FezopelConfig, FP8Linear, FullAttnWeights, GDNWeights, GLAConfig,
-                      HybridLayerConfig, LayerWeights, ModelConfig, MoEWeights, NVFP4Linear, WindowAttnConfig)
+from .weights import (ChannelDeltaConfig, Checkpoint, ChunkAttnConfig, DokulixCheckpoint, DokulixConfig, FezopelCheckpoint, FezopelConfig,
+                      FP8Linear, FullAttnWeights, GDNWeights, GLAConfig, HybridLayerConfig, LatentAttnConfig, LayerWeights, LoopConfig,
+                      ModelConfig, MoEWeights, NVFP4Linear, PreNormLayerConfig, WindowAttnConfig)
 
 BF16 = torch.bfloat16
 
@@ -246,3 +247,40 @@ def fezopel_tensors(config: FezopelConfig, seed: int = 0, device="cpu", rank: in
 def make_fezopel(config: FezopelConfig, seed: int = 0, device="cpu", rank: int = 16) -> FezopelCheckpoint:
     from .loader import assemble_hybrid
     return assemble_hybrid(config, fezopel_tensors(config, seed, device, rank).__getitem__)
+
+
+def dokulix_config(num_layers: int = 12, vocab_size: int = 32768, *, hidden: int = 2048, ff: int | None = None, window: int = 1024,
+                   chunk: int = 1024, heads: int = 16, kv_heads: int = 4, dim: int = 128, rot_dim: int = 64, q_rank: int | None = None,
+                   kv_rank: int = 512, loop: LoopConfig | None = None) -> DokulixConfig:
+    """Layers of the size of a real model: two of latent attention, then one of chunked attention."""
+    latent = LatentAttnConfig(heads=heads, dim=dim, rot_dim=rot_dim, vdim=dim, q_rank=q_rank or 3 * hidden // 4, kv_rank=kv_rank, window=window,
+                              rotary_base=1.0e6, scale=(dim + rot_dim) ** -0.5)
+    attn = ChunkAttnConfig(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, span=chunk, scale=dim ** -0.5)
+    return DokulixConfig(vocab_size=vocab_size, hidden_size=hidden, norm_eps=1e-6, loop=loop,
+                         layers=[PreNormLayerConfig(attn if i % 3 == 2 else latent, ff or 4 * hidden) for i in range(num_layers)])
+
+
+def dokulix_tensors(config: DokulixConfig, seed: int = 0, device="cpu") -> dict[str, torch.Tensor]:
+    """Random tensors under the checkpoint's names: matrices with unit gain, norm weights near their neutral value."""
+    from .loader import hybrid_shapes
+    src, out = Source(seed, device), {}
+    for name, shape in hybrid_shapes(config).items():
+        leaf = name.rsplit(".", 1)[-1]
+        if name == "embed":
+            out[name] = src.normal(name, *shape)
+        elif name == "loop.step":
+            out[name] = src.normal(name, *shape, std=0.3)
+        elif leaf == "b":
+            out[name] = src.normal(name, *shape, std=0.3)
+        elif leaf in ("norm1", "norm2") or name == "final.norm":
+            out[name] = src.normal(name, *shape, std=0.1)
+        elif leaf == "norm":
+            out[name] = src.normal(name, *shape, std=0.1, mean=1.0)
+        else:
+            out[name] = src.normal(name, *shape, std=shape[-1] ** -0.5)
+    return out
+
+
+def make_dokulix(config: DokulixConfig, seed: int = 0, device="cpu") -> DokulixCheckpoint:
+    from .loader import assemble_hybrid
+    return assemble_hybrid(config, dokulix_tensors(config, seed, device).__getitem__)

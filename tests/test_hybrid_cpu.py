@@ -17,6 +17,7 @@ from quickdraw_b200.loader import hybrid_shapes, load_hybrid_checkpoint, save_hy
 from quickdraw_b200.state import DecodeState, HybridState
 from quickdraw_b200.weights import FezopelConfig, WindowAttnConfig
 from tests import hybrid_cases as cases
+from tests.recording import AsIfOnGpu, recorder  # noqa: F401 (a fixture)
 
 ROOT = Path(__file__).resolve().parents[1]
 HEADER = ROOT / "include" / "quickdraw_b200_hybrid.h"
@@ -151,31 +152,6 @@ def test_missing_hybrid_library_fails_loudly(monkeypatch, tmp_path):
     for target in _lib.HYBRID_LIBRARIES:
         with pytest.raises(_lib.LibraryMissing, match=f"build {target}"):
             _lib.hybrid_lib(target)
-
-
-class AsIfOnGpu(torch.Tensor):
-    is_cuda = property(lambda self: True)
-
-
-@pytest.fixture
-def recorder(monkeypatch):
-    """The drivers on CPU tensors with the library replaced by a recorder of (name, arguments)."""
-    seen = []
-
-    def record(name, *args):
-        declared = _lib.HYBRID_LIBRARIES[_lib.HYBRID_OWNER[name]][name]
-        assert len(args) == len(declared), (name, len(args), len(declared))
-        seen.append((name, args))
-
-    class Properties:
-        multi_processor_count = 148
-
-    for module in (hybrid, mixers):
-        monkeypatch.setattr(module, "call_hybrid", record)
-        monkeypatch.setattr(module, "stream_of", lambda t: None)
-    monkeypatch.setattr(mixers, "size_hybrid", lambda name, *args: 4096)
-    monkeypatch.setattr(torch.cuda, "get_device_properties", lambda device: Properties)
-    return seen
 
 
 @pytest.mark.parametrize("tokens", [1, 2, 40])
