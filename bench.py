@@ -725,10 +725,10 @@ def main():
     ap.add_argument("--vocab", type=int, default=151936, help="vocabulary (151936 in the headline workload)")
     ap.add_argument("--matvec-rows", type=int, default=0, help="rows of the matvec roofline matrices (default 131072)")
     ap.add_argument("--context", type=int, default=2048, help="KV-cache capacity of the decode engine")
-    ap.add_argument("--model", choices=("qwen3-next", "fezopel"), default="qwen3-next",
-                    help="fezopel: kernels and models of the bf16-weight hybrid design beside the like ones of the default model")
+    ap.add_argument("--model", choices=("qwen3-next", "fezopel", "dokulix"), default="qwen3-next",
+                    help="fezopel, dokulix: kernels and models of a bf16-weight design beside the like ones of the closest other model")
     args = ap.parse_args()
-    if args.model == "fezopel":
+    if args.model != "qwen3-next":
         from quickdraw_b200 import hybrid_bench
         hbm, _ = measured_peaks()
         tensor, _ = measured_tensor_peak()

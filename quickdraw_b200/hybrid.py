@@ -83,6 +83,10 @@ class HybridModel:
         call_hybrid("qd_greedy", ptr(out), out.numel(), ptr(self._keys), ptr(self._counter), ptr(self.next_token), stream_of(out))
         return out
 
+    def products(self) -> list[torch.Tensor]:
+        """The matrices a token is multiplied with, logits aside (a looped layer's once per pass)."""
+        raise NotImplementedError
+
     def check(self) -> int:
         """Status word of the tensor-core products (0 = clean)."""
         return int(self.status.item())
@@ -96,6 +100,9 @@ class FezopelModel(HybridModel):
             self.mix.append(_Sublayer(mixer.projections, layer.mixer.o, layer.around_mixer))
             self.mlp.append(None if layer.mlp is None else
                             _Sublayer({"up": layer.mlp.up}, layer.mlp.down, layer.around_mlp, gelu_columns=cfg.ff))
+
+    def products(self):
+        return [m for sub in self.mix + self.mlp if sub is not None for m in (sub.matrix, sub.out)]
 
     def _project(self, sub: _Sublayer, normed):
         out = self._rows(normed.shape[0], sub.matrix.shape[0])
@@ -184,6 +191,10 @@ class DokulixModel(HybridModel):
             step = self.steps[r + 1] if r + 1 < len(self.runs) else None
             self.closing.append(bias if step is None else step.float() if bias is None else bias + step.float())
         self.folded = c.hidden_size % 8 == 0          # whether one token's products can take the stream itself
+
+    def products(self):
+        parts = [(self.parts[i], self.mixers[i]) for i, _ in self.runs]
+        return [m for part, mixer in parts for m in (part.matrix, part.out, *mixer.inner, part.glu, part.down) if m is not None]
 
     def _stream(self, count, *, source=None, token_ids=None, index=None, y=None, step=None, out=None, norm=None, normed=None):
         """Stream rows: embedding rows of the tokens or rows of ``source``, + ``y``, + ``step``; their norm."""

@@ -1,6 +1,6 @@
-"""Throughput of the Fezopel design on random weights at sizes of real models' layers, beside the
-NVFP4 hybrid MoE model of this package at equal width, depth and vocabulary, and every kernel of the
-design beside the like kernel of that model: ``python bench.py --model fezopel``.
+"""Throughput of the bf16-weight designs on random weights at sizes of real models' layers, beside the closest
+model of this package at equal width, depth and vocabulary, and every kernel of the design beside the like kernel
+of that model: ``python bench.py --model fezopel`` (beside the NVFP4 hybrid MoE), ``--model dokulix`` (beside Fezopel).
 
 Kernels are timed inside CUDA graphs over operand sets that together exceed L2 (no host time in the
 numbers); a fraction is algorithmic bytes or floating-point operations per second over the measured
@@ -11,22 +11,25 @@ from __future__ import annotations
 
 import json
 import os
+from ctypes import byref
 
 import torch
 
 from . import synthetic
-from ._lib import call, call_hybrid, hybrid_lib, lib, ptr, stream_of
+from ._lib import HYBRID_LIBRARIES, call, call_hybrid, hybrid_lib, lib, ptr, stream_of
 from .engine import Engine
-from .mixers import BF16, F32, ChannelDelta, GatedLinearAttention, WindowAttention, linear
+from .mixers import BF16, F32, ChannelDelta, ChunkAttention, GatedLinearAttention, LatentAttention, WindowAttention, column, linear
 from .state import LayerHistory
-from .weights import ChannelDeltaConfig, ChannelDeltaWeights, GLAConfig, GLAWeights, WindowAttnConfig, WindowAttnWeights
+from .weights import (ChannelDeltaConfig, ChannelDeltaWeights, ChunkAttnConfig, ChunkAttnWeights, GLAConfig, GLAWeights, LatentAttnConfig,
+                      LatentAttnWeights, LoopConfig, WindowAttnConfig, WindowAttnWeights)
 
 L2_BYTES = 160e6
 
 
 def graph_time(calls, reps: int = 5, chained: bool = True) -> float:
     """Seconds per call: ``calls`` (closures on different operands) captured into one graph, best of ``reps`` replays."""
-    old, old_hybrid = lib().qd_set_chained_launches(int(chained)), hybrid_lib().qd_set_chained_launches(int(chained))
+    libraries = [lib(), *map(hybrid_lib, HYBRID_LIBRARIES)]
+    old = [library.qd_set_chained_launches(int(chained)) for library in libraries]
     try:
         for fn in calls[:2]:
             fn()
@@ -36,8 +39,8 @@ def graph_time(calls, reps: int = 5, chained: bool = True) -> float:
             for fn in calls:
                 fn()
     finally:
-        lib().qd_set_chained_launches(old)
-        hybrid_lib().qd_set_chained_launches(old_hybrid)
+        for library, before in zip(libraries, old):
+            library.qd_set_chained_launches(before)
     graph.replay()
     best = float("inf")
     for _ in range(reps):
@@ -256,22 +259,141 @@ class Cases:
         self.pair(f"sublayer_close_kernel {tokens} x {width}, {older} earlier results", (own, nbytes), "seq_add_norm", (like, tokens * width * 8))
 
 
+class LatentCases(Cases):
+    """Kernels of the Dokulix design beside those of Fezopel."""
+
+    def product_forms(self, tokens, rows, width):
+        flops = 2.0 * tokens * rows * width
+        x, w = self.rnd(tokens, width), self.rnd(rows, width, std=width ** -0.5)
+        out, half, bias = self.rnd(tokens, rows), self.rnd(tokens, rows // 2), self.rnd(rows, dtype=F32)
+        plain = lambda: linear(x, 0, width, w, out, tokens=tokens, status=self.status)
+        glu = lambda: linear(x, 0, width, w, half, tokens=tokens, status=self.status, glu=True)
+        biased = lambda: linear(x, 0, width, w, out, tokens=tokens, status=self.status, bias=bias)
+        for name, own in (("gated unit", glu), ("bias", biased)):
+            self.pair(f"linear_umma_kernel, {name}, {tokens} x [{rows}, {width}]", ([own] * 8, 0, flops), "linear_umma_kernel", ([plain] * 8, 0, flops))
+
+    def matvec_forms(self, rows, width):
+        nbytes = rows * width * 2
+        x, stream, out, half = self.rnd(1, width), self.rnd(1, width, dtype=F32), self.rnd(1, rows), self.rnd(1, rows // 2)
+        held, norm = self.rnd(1, rows, dtype=F32), self.rnd(width)
+        ws = [self.rnd(rows, width, std=width ** -0.5) for _ in range(sets_for(nbytes))]
+        one = dict(tokens=1, status=self.status)
+        plain = [lambda w=w: linear(x, 0, width, w, out, **one) for w in ws]
+        forms = {"norm": [lambda w=w: linear(stream, 0, width, w, out, norm=norm, norm_offset=1.0, eps=1e-6, **one) for w in ws],
+                 "norm, gated unit": [lambda w=w: linear(stream, 0, width, w, half, norm=norm, norm_offset=1.0, eps=1e-6, glu=True, **one) for w in ws],
+                 "added to the stream": [lambda w=w: linear(x, 0, width, w, held, add=True, **one) for w in ws]}
+        for name, own in forms.items():
+            self.pair(f"linear_rows_kernel, {name}, 1 x [{rows}, {width}]", (own, nbytes), "linear_rows_kernel", (plain, nbytes))
+
+    def _window(self, heads, kv, d, window):
+        m = WindowAttnConfig(heads=heads, kv_heads=kv, dim=d, vdim=d, window=window, rotary_dims=d, rotary_base=1e6, scale=d ** -0.5)
+        weights = WindowAttnWeights(q=None, k=None, v=None, g=None, o=None, q_norm=self.rnd(heads * d), k_norm=self.rnd(kv * d), sink=self.rnd(heads))
+        return WindowAttention(weights, m, 1e-6, self.device), {"q": heads * d, "k": kv * d, "v": kv * d, "g": heads}
+
+    def _chunked(self, heads, kv, d, span):
+        m = ChunkAttnConfig(heads=heads, kv_heads=kv, dim=d, vdim=d, span=span, scale=d ** -0.5)
+        weights = ChunkAttnWeights(q=None, k=None, v=None, o=None, q_b=None, k_b=None, v_b=None, o_b=None, q_norm=self.rnd(d), k_norm=self.rnd(d))
+        return ChunkAttention(weights, m, 1e-6, self.device), {"q": heads * d, "k": kv * d, "v": kv * d}
+
+    def _latent(self, heads, d, rot, rank, window):
+        m = LatentAttnConfig(heads=heads, dim=d, rot_dim=rot, vdim=d, q_rank=1536, kv_rank=rank, window=window, rotary_base=1e6, scale=(d + rot) ** -0.5)
+        w = lambda *shape: self.rnd(*shape, std=shape[-1] ** -0.5)
+        weights = LatentAttnWeights(dq=None, dkv=None, g=None, o=None, dq_norm=self.rnd(m.q_rank), dkv_norm=self.rnd(rank),
+                                    uq=w(heads * (d + rot), m.q_rank), uk=w(heads * d, rank), uv=w(heads * d, rank))
+        return LatentAttention(weights, m, 1e-6, self.device), {"dq": m.q_rank, "dkv": rank + rot, "g": heads * d}
+
+    def attentions(self, tokens, heads, kv, d, rot, rank, span):
+        """Prompt chunks from position 0."""
+        seen, within = sum(min(span, i + 1) for i in range(tokens)), sum(i % span + 1 for i in range(tokens))
+        kv_rows = lambda g: LayerHistory(k=self.rnd(span + tokens, g, d), v=self.rnd(span + tokens, g, d))
+
+        def like(g):
+            mixer, widths = self._window(heads, g, d, span)
+            proj, at = self._laid_out(widths, tokens)
+            return [lambda h=kv_rows(g): mixer.chunk(proj, at, h, 0, self.status)] * 4, 0, 4.0 * seen * heads * d
+        mixer, widths = self._chunked(heads, kv, d, span)
+        proj, at = self._laid_out(widths, tokens)
+        hist = kv_rows(kv)
+        self.pair(f"attn_prepare + attn_flash, {tokens} tokens, chunks of {span}, {heads}/{kv} heads of {d}",
+                  ([lambda: mixer.chunk(proj, at, hist, 0, self.status)] * 4, 0, 4.0 * within * heads * d), f"the same, window {span}", like(kv))
+        latent, widths = self._latent(heads, d, rot, rank, span)
+        rows, at_latent = self._laid_out(widths, tokens)
+        cache = LayerHistory(latent=self.rnd(span + tokens, latent.m.row))
+        latent.chunk(rows, at_latent, cache, 0, self.status)              # binds the arguments of the launches below
+        q_rank = latent.m.q_rank
+        prepare = lambda: latent._prepare(rows)
+        prepare_like, widths = self._window(heads, heads, d, 1)
+        proj_like, at_like = self._laid_out(widths, tokens)
+        ring = LayerHistory(k=self.rnd(tokens, heads, d), v=self.rnd(tokens, heads, d))
+        near = lambda: prepare_like.chunk(proj_like, at_like, ring, 0, self.status)
+        self.pair(f"latent_prepare_kernel {tokens} tokens", ([prepare] * 4, tokens * (2 * q_rank + rank + rot + latent.m.row) * 2),
+                  "attn_prepare + attn_flash, window of one", ([near] * 4, tokens * heads * d * 2 * 8))
+        queries = self.rnd(tokens, heads * (d + rot))
+        rotate = lambda: call_hybrid("qd_rotate_half", ptr(queries), ptr(latent.freq), None, 0, tokens, heads, d + rot, rot, 0, stream_of(queries))
+        self.pair(f"rotate_half_kernel {tokens} tokens, {heads} heads, {rot} of {d + rot} columns", ([rotate] * 4, tokens * heads * rot * 4),
+                  "attn_prepare + attn_flash, window of one", ([near] * 4, tokens * heads * d * 2 * 8))
+        # the attention itself on expanded rows: everything but the products, the norm and the rotation
+        a, expanded, out = latent.args, self.rnd(span + tokens, latent.expand.shape[0]), self.rnd(tokens, heads * d)
+        a.q_rows, a.out, a.gate, a.ld_gate = ptr(queries), ptr(out), ptr(rows), rows.shape[1]
+        a.k_cache, a.v_cache = ptr(expanded), column(expanded, latent.expand_at["v"])
+        core = lambda: call_hybrid("qd_attention", byref(a), stream_of(queries))
+        self.pair(f"attn_flash on expanded latents, {tokens} tokens, window {span}, {heads} heads of {d} + {rot}",
+                  ([core] * 4, 0, 2.0 * seen * heads * (2 * d + rot)), f"attn_prepare + attn_flash, {heads}/{heads} heads of {d}", like(heads))
+
+    def attention_steps(self, heads, kv, d, rot, rank, span):
+        pos = torch.tensor(span - 1, dtype=torch.int32, device=self.device)
+        nbytes = 2 * span * kv * d * 2
+        caches = [LayerHistory(k=self.rnd(span, kv, d), v=self.rnd(span, kv, d)) for _ in range(sets_for(nbytes))]
+
+        def steps(mixer, widths, histories):
+            proj, at = self._laid_out(widths, 1)
+            return [lambda h=h: mixer.step(proj, at, h, pos, self.status) for h in histories]
+        like = (steps(*self._window(heads, kv, d, span), caches), nbytes)
+        self.pair(f"attn_step_kernel, chunk of {span}, {heads}/{kv} heads of {d}", (steps(*self._chunked(heads, kv, d, span), caches), nbytes),
+                  f"attn_step_kernel, window {span}", like)
+        mixer, widths = self._latent(heads, d, rot, rank, span)
+        own_bytes = span * mixer.m.row * 2 + mixer.expand.nbytes
+        sets = sets_for(own_bytes)
+        mixers = [mixer] + [self._latent(heads, d, rot, rank, span)[0] for _ in range(sets - 1)]
+        rows, at = self._laid_out(widths, 1)
+        calls = []
+        for one in mixers:
+            history = LayerHistory(latent=self.rnd(span, mixer.m.row))
+            query, out = self.rnd(1, heads * (d + rot)), self.rnd(1, heads * d)
+            one._bind(rows, at, history, pos)
+            one.latent.q, one.latent.out, one.kept = ptr(query), ptr(out), (history, query, out)
+            calls.append(lambda one=one: call_hybrid("qd_latent_step", byref(one.latent), stream_of(rows)))
+        self.pair(f"latent absorb + mma + values kernels, window {span}, {heads} heads of {d} + {rot}, rank {rank}", (calls, own_bytes),
+                  f"attn_step_kernel, window {span}, {heads}/{kv} heads of {d}", like)
+
+    def stream_norm(self, tokens, width):
+        y, normed, vec = self.rnd(tokens, width), self.rnd(tokens, width), self.rnd(width)
+        streams = [self.rnd(tokens, width, dtype=F32) for _ in range(sets_for(tokens * width * 8) if tokens > 64 else 8)]
+        own = [lambda r=r: call_hybrid("qd_stream_norm", None, None, 0, ptr(r), None, ptr(y), None, ptr(r), ptr(vec), 1.0, ptr(normed), tokens, width, 1e-6,
+                                       0, stream_of(y)) for r in streams]
+        gate = self.rnd(tokens, width)
+        like = [lambda r=r: call_hybrid("qd_sublayer_close", ptr(y), ptr(gate), width, ptr(vec), ptr(vec), ptr(vec), ptr(r), ptr(r), None, 0, None, -1,
+                                        ptr(vec), ptr(vec), ptr(normed), tokens, width, 1e-6, 0, stream_of(y)) for r in streams]
+        self.pair(f"stream_norm_kernel {tokens} x {width}", (own, tokens * width * 12), "sublayer_close_kernel, no earlier results",
+                  (like, tokens * width * 14))
+
+
 def step_bytes(engine, position: int) -> float:
-    """Algorithmic bytes of one token: every matrix once, recurrent states read and written, the visible window."""
+    """Algorithmic bytes of one token: every matrix once per use, recurrent states read and written, the visible rows."""
     model, c = engine.fused, engine.ckpt.config
-    total = sum(sub.matrix.nbytes + sub.out.nbytes for sub in model.mix + [m for m in model.mlp if m]) + engine.ckpt.lm_head.nbytes
-    for layer, history in zip(c.layers, engine.state.layers):
+    total = sum(m.nbytes for m in model.products()) + engine.ckpt.lm_head.nbytes
+    for (index, _), history in zip(c.runs(), engine.state.layers):
+        m = c.layers[index].mixer
         if history.rec is not None:
             total += 2 * history.rec.nbytes
-        else:
-            m = layer.mixer
-            total += min(m.window, position + 1) * m.kv_heads * (m.dim + m.vdim) * 2
+            continue
+        visible = position % m.span + 1 if isinstance(m, ChunkAttnConfig) else min(m.span, position + 1)
+        total += visible * (m.row if history.latent is not None else m.kv_heads * (m.dim + m.vdim)) * 2
     return total
 
 
 def matmul_flops(engine, tokens: int) -> float:
-    model = engine.fused
-    return 2.0 * tokens * sum(sub.matrix.numel() + sub.out.numel() for sub in model.mix + [m for m in model.mlp if m])
+    return 2.0 * tokens * sum(m.numel() for m in engine.fused.products())
 
 
 def timed(fn, reps: int = 3) -> float:
@@ -321,13 +443,7 @@ def model_leg(ckpt, prompts, decode_steps: int, hbm: float, tensor: float, hybri
     return out
 
 
-def run(args, peaks: dict, clocks) -> None:
-    device = torch.device("cuda:0")
-    torch.cuda.set_device(device)
-    hbm, tensor = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
-    torch.manual_seed(0)
-    clocks.mark_begin()
-    cases = Cases(device, peaks["hbm_gbs"], peaks["bf16_tflops"])
+def fezopel_cases(cases: Cases) -> None:
     cases.products(8192, 8192, 2048)
     cases.products(512, 8192, 2048)
     cases.matvec(12288, 2048)
@@ -340,18 +456,59 @@ def run(args, peaks: dict, clocks) -> None:
     cases.attention_step(16, 2, 256, 8192)
     cases.residual(2048, 2048, 6)
     cases.residual(1, 2048, 6)
-    assert int(cases.status.item()) == 0
-    torch.cuda.empty_cache()
+
+
+def dokulix_cases(cases: LatentCases) -> None:
+    cases.product_forms(2048, 16384, 2048)
+    cases.matvec_forms(16384, 2048)
+    cases.matvec_forms(2048, 8192)
+    cases.attentions(2048, 16, 4, 128, 64, 512, 1024)
+    cases.attentions(8192, 16, 4, 128, 64, 512, 4096)
+    cases.attention_steps(16, 4, 128, 64, 512, 1024)
+    cases.attention_steps(16, 4, 128, 64, 512, 8192)
+    cases.stream_norm(2048, 2048)
+    cases.stream_norm(1, 2048)
+
+
+def fezopel_models(device, leg) -> dict:
     models = {}
     for hidden, depth in ((2048, 12), (4096, 12)):
         cfg = synthetic.fezopel_config(depth, 32768, hidden=hidden, heads=hidden // 128, kv_heads=max(2, hidden // 512))
-        models[f"fezopel {depth} x {hidden}"] = model_leg(synthetic.make_fezopel(cfg, 0, device), (512, 2048, 8192), 64, hbm, tensor, True)
+        models[f"fezopel {depth} x {hidden}"] = leg(synthetic.make_fezopel(cfg, 0, device), True)
         torch.cuda.empty_cache()
-    like = synthetic.model_config(num_layers=12, vocab_size=32768)
-    models["nvfp4 hybrid MoE 12 x 2048"] = model_leg(synthetic.make_checkpoint(like, seed=0, device=device), (512, 2048, 8192), 64, hbm, tensor, False)
+    return models
+
+
+def dokulix_models(device, leg) -> dict:
+    models = {}
+    for hidden, depth, loop in ((2048, 12, None), (4096, 12, None), (2048, 12, LoopConfig(3, 9, 2))):
+        cfg = synthetic.dokulix_config(depth, 32768, hidden=hidden, heads=hidden // 128, kv_heads=max(2, hidden // 512), loop=loop)
+        name = f"dokulix {depth} x {hidden}" + ("" if loop is None else f", layers {loop.start} - {loop.stop - 1} {loop.times} times")
+        models[name] = leg(synthetic.make_dokulix(cfg, 0, device), True)
+        torch.cuda.empty_cache()
+    return models
+
+
+def run(args, peaks: dict, clocks) -> None:
+    device = torch.device("cuda:0")
+    torch.cuda.set_device(device)
+    hbm, tensor = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    torch.manual_seed(0)
+    clocks.mark_begin()
+    own = args.model == "fezopel"
+    cases = (Cases if own else LatentCases)(device, peaks["hbm_gbs"], peaks["bf16_tflops"])
+    (fezopel_cases if own else dokulix_cases)(cases)
+    assert int(cases.status.item()) == 0
+    torch.cuda.empty_cache()
+    leg = lambda ckpt, hybrid: model_leg(ckpt, (512, 2048, 8192), 64, hbm, tensor, hybrid)
+    models = {} if own else dokulix_models(device, leg)
+    models |= fezopel_models(device, leg)
+    if own:
+        like = synthetic.model_config(num_layers=12, vocab_size=32768)
+        models["nvfp4 hybrid MoE 12 x 2048"] = leg(synthetic.make_checkpoint(like, seed=0, device=device), False)
     clocks.mark_end()
-    first = models["fezopel 12 x 2048"]
-    line = {"metric": "decode_tok_s", "model": "fezopel", "value": first["decode"]["tok_s"], "unit": "tok/s", "higher_is_better": True, "n_gpus": 1,
+    first = models[f"{args.model} 12 x 2048"]
+    line = {"metric": "decode_tok_s", "model": args.model, "value": first["decode"]["tok_s"], "unit": "tok/s", "higher_is_better": True, "n_gpus": 1,
             "dtype": "bf16", "data": "synthetic (random weights)", "vs_baseline": None, "ms_per_step": first["decode"]["ms_per_token"],
             "config": {"l2": "kernel legs rotate over operands beyond L2 or exceed it; a decode step streams its weights"},
             "models": models, "kernels": cases.rows, "peaks": peaks, "clocks": None, "cpus": os.cpu_count()}

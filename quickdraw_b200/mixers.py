@@ -81,6 +81,7 @@ def step_covers(m) -> bool:
 
 class GroupedAttention:
     """Grouped-query attention over a bounded span of positions; ``constants`` are fields of ``qd_attention_args``."""
+    inner = ()                                                  # matrices between the input and the output projections
     KEYS_PER_SPLIT, MAX_SPLITS = 32, 64
 
     def __init__(self, m, eps: float, device, tensors: dict, **constants):
@@ -151,6 +152,7 @@ class LatentAttention:
         self.projections = {"dq": weights.dq, "dkv": weights.dkv, "g": weights.g}
         self.out_columns = m.heads * m.vdim
         self.expand, self.expand_at = stack_rows({"k": weights.uk, "v": weights.uv})
+        self.inner = (weights.uq, self.expand)
         sms = torch.cuda.get_device_properties(device).multi_processor_count
         blocks = -(-m.heads // self.HEADS_PER_BLOCK)
         self.splits = max(1, min(-(-m.span // self.KEYS_PER_SPLIT), -(-sms // blocks), self.MAX_SPLITS))
