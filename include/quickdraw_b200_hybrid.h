@@ -155,7 +155,7 @@ typedef struct qd_latent_args {
     long long ld, ld_cache;
     float scale, eps;
     int span, capacity, position, tokens, heads, dim, rot, vdim, q_rank, kv_rank, rot_column;
-    int splits;                         /* one token: blocks per 16 heads, at most 32 */
+    int splits;                         /* one token: blocks per 16 heads, at most 64 */
     int dtype;
 } qd_latent_args;
 

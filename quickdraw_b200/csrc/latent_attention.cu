@@ -21,7 +21,7 @@ namespace {
 
 typedef qd_latent_args Latent;
 constexpr int kTile = 32, kThreads = 256, kWarps = kThreads / 32;
-constexpr int kMaxSplits = 32;
+constexpr int kMaxSplits = 64;
 
 QD_DEVINL int position_of(const Latent& p) { return p.position_ptr ? *p.position_ptr : p.position; }
 QD_DEVINL const bf16* weights(const void* p) { return reinterpret_cast<const bf16*>(p); }
@@ -413,9 +413,14 @@ __global__ void __launch_bounds__(kThreads) latent_values_kernel(const __grid_co
     grid_dependency_wait();
     const Splits plan = split_plan(p, position_of(p));
     if (warp == 0) {
-        const float2 s = lane < plan.active ? __ldcg(split_stats(p) + (size_t)h * p.splits + lane) : make_float2(-INFINITY, 0.f);
-        const float w = expf(s.x - warp_max(s.x));
-        factor[lane] = w / warp_sum(w * s.y);
+        float2 s[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+            s[i] = i * 32 + lane < plan.active ? __ldcg(split_stats(p) + (size_t)h * p.splits + i * 32 + lane) : make_float2(-INFINITY, 0.f);
+        const float top = warp_max(fmaxf(s[0].x, s[1].x)), a = expf(s[0].x - top), b = expf(s[1].x - top);
+        const float total = warp_sum(fmaf(a, s[0].y, b * s[1].y));
+        factor[lane] = a / total;
+        factor[32 + lane] = b / total;
     }
     __syncthreads();
     const int columns = value_columns(p.kv_rank), quads = columns / 4;

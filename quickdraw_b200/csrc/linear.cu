@@ -241,6 +241,9 @@ linear_umma_kernel(const __grid_constant__ LinearParams p, const __grid_constant
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int t0 = blockIdx.x * HALVES * 128, n0 = blockIdx.y * TN;
     const int steps = (p.width + kStepK - 1) / kStepK;
+    __shared__ __align__(16) float bias[TN];
+    if (p.f.bias)
+        for (int i = tid; i < TN; i += Tile::kThreads) bias[i] = n0 + i < p.rows ? p.f.bias[n0 + i] : 0.f;
     const int halves = (HALVES == 2 && p.tokens - t0 > 128) ? 2 : 1;       // a half without tokens is not multiplied
 
     if (tid == 0) {
@@ -316,7 +319,7 @@ linear_umma_kernel(const __grid_constant__ LinearParams p, const __grid_constant
 #pragma unroll
                             for (int q = 0; q < 8; ++q) f[q] = __uint_as_float(v[j + q]);
                             if (p.f.bias) {
-                                const float4 a = load4(p.f.bias + n), b = load4(p.f.bias + n + 4);
+                                const float4 a = load4(bias + c + j), b = load4(bias + c + j + 4);
                                 f[0] += a.x; f[1] += a.y; f[2] += a.z; f[3] += a.w; f[4] += b.x; f[5] += b.y; f[6] += b.z; f[7] += b.w;
                             }
                             if (gelu) {
@@ -419,7 +422,7 @@ int dispatch(const void* x, long long ldx, const void* w, void* y, long long ldy
         return launch_rows<TX, TY, 8>(x, ldx, w, y, ldy, tokens, rows, width, f, norm, stream);
     }
     if (norm.weight) return QD_ERR_UNSUPPORTED;
-    if (sizeof(TX) == 2 && vectors && rows % 8 == 0 && ldy % 8 == 0 && aligned16(y) && aligned16(f.bias)) {
+    if (sizeof(TX) == 2 && vectors && rows % 8 == 0 && ldy % 8 == 0 && aligned16(y)) {
         const LinearParams p = {y, ldy, tokens, rows, width, f, status};
         return umma_dispatch<TY>(x, ldx, w, p, stream);
     }

@@ -84,6 +84,62 @@ __global__ void __launch_bounds__(256) attn_prepare_kernel(const __grid_constant
     for (int i = tid; i < vn; i += 256) ring_v[i] = v[i];
 }
 
+// The same for rows of four-element pieces: a warp per head, no divisions by the head size.
+template <typename T>
+__global__ void __launch_bounds__(256) attn_prepare_vec_kernel(const __grid_constant__ AttnParams p) {
+    chain_enter();
+    extern __shared__ float trig[];                    // cosines, sines
+    __shared__ float red[33];
+    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, half = p.rot / 2;
+    const int position = (p.position_ptr ? *p.position_ptr : p.position) + t;
+    const int qn = p.heads * p.dim, kn = p.kv_heads * p.dim, vn = p.kv_heads * p.vdim;
+    const T* q = reinterpret_cast<const T*>(p.q) + (long long)t * p.ld;
+    const T* k = reinterpret_cast<const T*>(p.k) + (long long)t * p.ld;
+    const T* v = reinterpret_cast<const T*>(p.v) + (long long)t * p.ld;
+    for (int i = tid; i < half; i += 256) rotation(position, p.freq[i], p.freq[half + i], trig[i], trig[half + i]);
+    const auto squares = [](const float4& x, float sum) { return fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, sum)))); };
+    float qr = 1.f, kr = 1.f;
+    if (p.norm == QD_NORM_ROW) {
+        float qq = 0.f, kk = 0.f;
+        for (int i = tid * 4; i < qn; i += 1024) qq = squares(load4(q + i), qq);
+        for (int i = tid * 4; i < kn; i += 1024) kk = squares(load4(k + i), kk);
+        qr = 1.0f / sqrtf(block_sum(qq, red) / (float)qn + p.eps);
+        kr = 1.0f / sqrtf(block_sum(kk, red) / (float)kn + p.eps);
+    }
+    __syncthreads();
+    const size_t slot = position % p.capacity;
+    T* ring_k = reinterpret_cast<T*>(p.k_cache) + slot * p.ld_k;
+    T* ring_v = reinterpret_cast<T*>(p.v_cache) + slot * p.ld_v;
+    T* q_out = reinterpret_cast<T*>(p.q_rows) + (size_t)t * qn;
+    for (int h = tid >> 5; h < p.heads + p.kv_heads; h += 8) {
+        const bool query = h < p.heads;
+        const int at = (query ? h : h - p.heads) * p.dim;
+        const T* src = (query ? q : k) + at;
+        T* dst = (query ? q_out : ring_k) + at;
+        const bf16* w = as_bf16(query ? p.q_norm : p.k_norm) + (p.norm == QD_NORM_ROW ? at : 0);
+        float r = query ? qr : kr;
+        if (p.norm == QD_NORM_HEAD) {
+            float ss = 0.f;
+            for (int d = lane * 4; d < p.dim; d += 128) ss = squares(load4(src + d), ss);
+            r = 1.0f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+        }
+        for (int d = lane * 4; d < p.dim; d += 128) {
+            float4 x = load4(src + d);
+            if (p.norm != QD_NORM_NONE) {
+                const float4 g = load4(w + d);
+                x.x *= r * g.x; x.y *= r * g.y; x.z *= r * g.z; x.w *= r * g.w;
+            }
+            if (d < p.rot) {
+                const int i = d >> 1;
+                x = make_float4(fmaf(x.x, trig[i], -x.y * trig[half + i]), fmaf(x.y, trig[i], x.x * trig[half + i]),
+                                fmaf(x.z, trig[i + 1], -x.w * trig[half + i + 1]), fmaf(x.w, trig[i + 1], x.z * trig[half + i + 1]));
+            }
+            store4(dst + d, x);
+        }
+    }
+    for (int i = tid * 4; i < vn; i += 1024) store4(ring_v + i, load4(v + i));
+}
+
 // ----------------------------------------------------------------------------- any type, any shape
 constexpr int kRowsPerLane = 8;                        // value columns per lane: 256 per block column
 
@@ -185,23 +241,30 @@ __global__ void __launch_bounds__(WARPS * 32) attn_flash_kernel(const __grid_con
     for (int i = tid; i < all / 8; i += kFlashThreads) reinterpret_cast<uint4*>(tiles)[i] = make_uint4(0u, 0u, 0u, 0u);
     __syncthreads();
     const int kp = p.dim / 8, qp = qdim / 8, vp = p.vdim / 8;          // 16-byte pieces
-    for (int i = tid; i < kFlashRows * qp; i += kFlashThreads) {
-        const int r = i / qp, piece = i % qp, row = r0 + r;
+    for (int r = warp; r < kFlashRows; r += WARPS) {
+        const int row = r0 + r;
         const bool ok = row < total;
-        const size_t src = ok ? ((size_t)(row / share) * p.heads + g * share + row % share) * qdim + piece * 8 : 0;
-        copy16_or_zero(qs + r * krow + piece * 8, q + src, ok);
+        const bf16* src = q + (ok ? ((size_t)(row / share) * p.heads + g * share + row % share) * qdim : 0);
+        for (int piece = lane; piece < qp; piece += 32) copy16_or_zero(qs + r * krow + piece * 8, src + piece * 8, ok);
     }
+    const int slot_first = key_first % p.capacity;
     auto stage = [&](int tile) {
         const int j0 = key_first + tile * kFlashKeys;
         bf16* kd = ks + (tile & 1) * kFlashKeys * krow;
         bf16* vd = vs + (tile & 1) * kFlashKeys * kVRow;
-        for (int i = tid; i < kFlashKeys * (qp + vp); i += kFlashThreads) {
-            const int r = i / (qp + vp), piece = i % (qp + vp), j = j0 + r;
+        for (int r = warp; r < kFlashKeys; r += WARPS) {          // a warp per row
+            const int j = j0 + r;
             const bool ok = j <= pos_last;
-            const size_t slot = ok ? j % p.capacity : 0;
-            if (piece < kp) copy16_or_zero(kd + r * krow + piece * 8, kc + slot * p.ld_k + piece * 8, ok);
-            else if (piece < qp) copy16_or_zero(kd + r * krow + piece * 8, common + slot * p.ld_shared + (piece - kp) * 8, ok);
-            else copy16_or_zero(vd + r * kVRow + (piece - qp) * 8, vc + slot * p.ld_v + (piece - qp) * 8, ok);
+            int slot = ok ? slot_first + (j - key_first) : 0;
+            if (slot >= p.capacity) slot -= p.capacity;           // what a block sees fits the ring
+            const bf16* own = kc + slot * p.ld_k;
+            const bf16* shared_row = common + slot * p.ld_shared - p.dim;
+            const bf16* value = vc + slot * p.ld_v;
+            for (int piece = lane; piece < qp + vp; piece += 32) {
+                if (piece < kp) copy16_or_zero(kd + r * krow + piece * 8, own + piece * 8, ok);
+                else if (piece < qp) copy16_or_zero(kd + r * krow + piece * 8, shared_row + piece * 8, ok);
+                else copy16_or_zero(vd + r * kVRow + (piece - qp) * 8, value + (piece - qp) * 8, ok);
+            }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -640,7 +703,11 @@ int chunk(const AttnParams& p, cudaStream_t s) {
     if (p.q) {
         const size_t shared = (size_t)(p.rot + p.heads + p.kv_heads + 1) * 4;
         if (!allow_smem(attn_prepare_kernel<T>, shared)) return QD_ERR_UNSUPPORTED;
-        const int rc = qd_launch(attn_prepare_kernel<T>, dim3(p.tokens), dim3(256), shared, s, 1, p);
+        const bool quads = p.dim % 4 == 0 && p.vdim % 4 == 0 && p.rot % 4 == 0 && p.ld % 4 == 0 && p.ld_k % 4 == 0 && p.ld_v % 4 == 0 && aligned16(p.q) &&
+                           aligned16(p.k) && aligned16(p.v) && aligned16(p.q_norm) && aligned16(p.k_norm) && aligned16(p.k_cache) &&
+                           aligned16(p.v_cache) && aligned16(p.q_rows);
+        const int rc = quads ? qd_launch(attn_prepare_vec_kernel<T>, dim3(p.tokens), dim3(256), (size_t)(p.rot + 1) * 4, s, 1, p)
+                             : qd_launch(attn_prepare_kernel<T>, dim3(p.tokens), dim3(256), shared, s, 1, p);
         if (rc != QD_OK) return rc;
     }
     const bool rows16 = sizeof(T) == 2 && p.dim % 8 == 0 && p.vdim % 8 == 0 && p.shared_dim % 8 == 0 && p.ld_k % 8 == 0 && p.ld_v % 8 == 0 &&

@@ -145,7 +145,7 @@ class ChunkAttention(GroupedAttention):
 class LatentAttention:
     """Latent attention in a sliding window with a gate per value column.  The cache holds latents.  A chunk expands the
     visible ones into keys and values; one token works on the latents (the expansions move to its query and to its result)."""
-    KEYS_PER_SPLIT, MAX_SPLITS, HEADS_PER_BLOCK = 32, 32, 16
+    KEYS_PER_SPLIT, MAX_SPLITS, HEADS_PER_BLOCK = 32, 64, 16
 
     def __init__(self, weights: LatentAttnWeights, m: LatentAttnConfig, eps: float, device):
         self.w, self.m, self.eps, self.freq = weights, m, eps, frequencies(m.rotary_base, m.rot_dim, device)
