@@ -134,7 +134,8 @@ int qd_attention(const qd_attention_args* args, void* stream);
 /* Floats of `partial` (16-byte aligned). */
 long long qd_attention_step_floats(int heads, int vdim, int splits);
 
-/* One token in one launch (q given, shared_dim 0, capacity >= span). */
+/* One token in one launch (q given, shared_dim 0, capacity >= span); with q_rows in two where a group of heads exceeds
+ * what one launch holds. */
 int qd_attention_step(const qd_attention_args* args, void* stream);
 
 /* Latent attention over the last `span` positions (libquickdraw_b200_latent.so).  The cache row of position p is

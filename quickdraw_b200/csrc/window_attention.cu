@@ -729,6 +729,7 @@ int step(const AttnParams& a, cudaStream_t s) {
     AttnStep sp = {a, 2};
     const auto smem = [&] { return step_smem<T>(a.heads / a.kv_heads, a.dim, a.vdim, a.rot, sp.buffers); };
     if (smem() > 220 * 1024) sp.buffers = 1;
+    if (smem() > kMaxSmem) return a.q_rows ? chunk<T>(a, s) : QD_ERR_UNSUPPORTED;      // very many heads to a key row
     if (!allow_smem(attn_step_kernel<T>, smem())) return QD_ERR_UNSUPPORTED;
     return qd_launch(attn_step_kernel<T>, dim3(a.kv_heads, a.splits), dim3(kStepThreads), smem(), s, 1, sp);
 }

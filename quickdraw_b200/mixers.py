@@ -105,18 +105,17 @@ class GroupedAttention:
         a.position_ptr, a.position = place(position)
         a.tokens, a.dtype, a.splits = proj.shape[0], DTYPE_CODE[proj.dtype], self.splits
         out = torch.empty((a.tokens, self.out_columns), dtype=proj.dtype, device=proj.device)
-        a.out = ptr(out)
-        return out
+        queries = torch.empty((a.tokens, self.m.heads * self.m.dim), dtype=proj.dtype, device=proj.device)
+        a.out, a.q_rows = ptr(out), ptr(queries)
+        return out, queries                                     # the queries live until the launch
 
     def chunk(self, proj, at, history: LayerHistory, position, status):
-        out = self._bind(proj, at, history, position)
-        queries = torch.empty((proj.shape[0], self.m.heads * self.m.dim), dtype=proj.dtype, device=proj.device)
-        self.args.q_rows = ptr(queries)
+        out, queries = self._bind(proj, at, history, position)
         call_hybrid("qd_attention", byref(self.args), stream_of(proj))
         return out
 
     def step(self, proj, at, history: LayerHistory, position, status):
-        out = self._bind(proj, at, history, position)
+        out, queries = self._bind(proj, at, history, position)
         call_hybrid("qd_attention_step", byref(self.args), stream_of(proj))
         return out
 

@@ -260,6 +260,16 @@ def test_chunked_decoding_with_long_splits(M, name, splits, dtype):
     assert error(got[180:], want()[180:]) < (2e-5 if dtype == F32 else 2e-2)
 
 
+@pytest.mark.parametrize("dtype", [F32, BF16])
+def test_more_heads_to_a_key_than_one_launch_holds(M, dtype):
+    m, tokens = cases.chunked(heads=70, kv_heads=1, dim=256, vdim=256, span=14, scale=0.08), 32
+    w, eps, proj, at, want = chunk_case(m, tokens, dtype, sharp=1.5)
+    mixer = M.ChunkAttention(on_gpu(w), m, eps, torch.device("cuda"))
+    history = LayerHistory(k=nan_rows(dtype, 30, 1, 256), v=nan_rows(dtype, 30, 1, 256))
+    got = drive(mixer, proj.cuda(), at, history, [17] + [1] * 15)
+    assert error(got, want()) < (2e-5 if dtype == F32 else 2e-2)
+
+
 @pytest.mark.parametrize("norm,sink,gate,mask", [(0, 0, 0, 1), (1, 1, 2, 1), (2, 0, 1, 0), (0, 2, 2, 0), (2, 1, 0, 1)])
 @pytest.mark.parametrize("vdim", [24, 21])
 @pytest.mark.parametrize("dtype", [F32, BF16])
